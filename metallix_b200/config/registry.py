@@ -16,6 +16,7 @@ from dataclasses import dataclass
 from typing import Any, Dict, Mapping, Optional, Type
 
 from .dimorax import DimoraxConfig
+from .kokolorn import KokolornConfig
 from .mekazen import MekazenConfig
 from .qwen3 import ConfigError, Qwen3Config
 from .sadosun import SadosunConfig
@@ -140,3 +141,6 @@ register(SADOSUN)
 DIMORAX = ModelFamily(architecture=DimoraxConfig.ARCHITECTURE, model_type=DimoraxConfig.MODEL_TYPE,
                       kind="dimorax", config_class=DimoraxConfig)
 register(DIMORAX)
+KOKOLORN = ModelFamily(architecture=KokolornConfig.ARCHITECTURE, model_type=KokolornConfig.MODEL_TYPE,
+                       kind="kokolorn", config_class=KokolornConfig)
+register(KOKOLORN)

@@ -67,6 +67,8 @@ class LayerRun:
     layer: int
     cache: Optional[int] = None
     write_cache: bool = True
+    join: Optional[int] = None      # which of ModelSpec.joins acts on the residual stream right before this run
+    turn: int = 0                   # ... and for which time, for a join with parameters per turn
 
     def cache_entry(self) -> int:
         return self.layer if self.cache is None else self.cache
@@ -131,6 +133,8 @@ class ModelSpec:
     # [tokens, s, hidden], all equal to the embedding at the start and summed at
     # the end, which blocks of a hyper-connection arrangement read and write.
     streams: int = 0
+    # What may happen to the residual stream ahead of a layer run (``LayerRun.join``).
+    joins: Tuple[PartSpec, ...] = ()
 
     def num_cache_entries(self) -> int:
         return max(run.cache_entry() for run in self.order) + 1
@@ -142,6 +146,8 @@ class ModelSpec:
         for run in self.order:
             if not 0 <= run.layer < len(self.layers):
                 raise ValueError(f"order names layer {run.layer}, the model has {len(self.layers)}")
+            if run.join is not None and not (0 <= run.join < len(self.joins) and self.streams == 0):
+                raise ValueError(f"order names join {run.join}, the model has {len(self.joins)} and {self.streams} streams")
             entry = run.cache_entry()
             if entry < 0:
                 raise ValueError(f"order names cache entry {entry}")

@@ -60,7 +60,7 @@ paged_attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ cac
                               int max_pages, const int* __restrict__ row_token,
                               const int* __restrict__ row_request, const int* __restrict__ positions,
                               int heads, int kv_heads, int page_tokens, int num_pages, int max_splits,
-                              int window, int chunk, float scale, float softcap, int* status) {
+                              int window, int chunk, float scale, float softcap, ScoreBias bias, int* status) {
   constexpr int E = Vec16<T>::kElems;  // elements per 16-byte piece
   constexpr int LPK = HD / E;          // 16-byte pieces (and lanes) per key row
   constexpr int KPW = 32 / LPK;        // key rows a warp reads at once
@@ -149,7 +149,11 @@ paged_attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ cac
 #pragma unroll
       for (int offset = LPK / 2; offset > 0; offset >>= 1)
         dots[h] += __shfl_xor_sync(0xffffffffu, dots[h], offset);
-      if (sub == 0 && kk < count) s_score[h * kSplitKeys + kk] = capped_score(dots[h] * scale, softcap);
+      if (sub == 0 && kk < count) {
+        float s = capped_score(dots[h] * scale, softcap);
+        if (bias.table != nullptr && h < group) s += bias_at(bias.row(kv * group + h), pos - begin - kk, bias.far);
+        s_score[h * kSplitKeys + kk] = s;
+      }
     }
   }
   __syncthreads();
@@ -239,6 +243,15 @@ __device__ __forceinline__ float decode_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
+// The biases of a thread's eight keys (zeros without a table): key nb * 8 + j of its own lies `back` - nb * 8 - j
+// positions back. Asked for ahead of the wait for the keys: a table is no kernel's output.
+__device__ __forceinline__ void decode_biases(float (&near)[4][2], ScoreBias bias, int head, bool live, int back) {
+#pragma unroll
+  for (int nb = 0; nb < 4; ++nb)
+#pragma unroll
+    for (int j = 0; j < 2; ++j)
+      near[nb][j] = bias.table != nullptr && live ? bias_at(bias.row(head), back - nb * 8 - j, bias.far) : 0.0f;
+}
 // Key rows lie in shared memory as they lie in the cache, each followed by 16
 // bytes of padding: eight consecutive rows then start in eight different bank
 // groups, so ldmatrix meets no conflict, and a row is one bulk copy.
@@ -253,7 +266,7 @@ paged_attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __n
                                   int max_pages, const int* __restrict__ row_token,
                                   const int* __restrict__ row_request, const int* __restrict__ positions,
                                   int heads, int kv_heads, int page_tokens, int num_pages, int max_splits,
-                                  int window, int chunk, float scale, float softcap, int* status) {
+                                  int window, int chunk, float scale, float softcap, ScoreBias bias, int* status) {
   constexpr int ROW_BYTES = HD * 2;
   constexpr int TILE_BYTES = kSplitKeys * (ROW_BYTES + 16);
   extern __shared__ __align__(128) unsigned char mma_shared[];
@@ -343,6 +356,8 @@ paged_attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __n
       qa2[ks] = g < group ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 8 + 2 * t) : 0u;
     }
   }
+  float near[4][2];
+  decode_biases(near, bias, kv * group + g, g < group, pos - begin - warp * 32 - 2 * t);
   const bool keys_landed = barrier_wait(&barriers[0], 0, status);
   __syncthreads();  // also orders the zero rows written by other threads
 
@@ -372,7 +387,7 @@ paged_attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __n
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int kk = key_base + nb * 8 + 2 * t + j;
-      sc[nb][j] = kk < count ? capped_score(sc[nb][j] * scale, softcap) * kLog2E : -INFINITY;
+      sc[nb][j] = kk < count ? (capped_score(sc[nb][j] * scale, softcap) + near[nb][j]) * kLog2E : -INFINITY;
       m_w = fmaxf(m_w, sc[nb][j]);
     }
   }
@@ -467,7 +482,7 @@ paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache,
                                   int max_pages, const int* __restrict__ row_token,
                                   const int* __restrict__ row_request, const int* __restrict__ positions,
                                   int heads, int kv_heads, int page_tokens, int num_pages, int max_splits,
-                                  int window, int chunk, float scale, float softcap, int* status) {
+                                  int window, int chunk, float scale, float softcap, ScoreBias bias, int* status) {
   constexpr int HALVES = HD / kTmaColumns;                 // 64-value halves of a row
   constexpr int TILE_BYTES = kSplitKeys * HD * 2;
   extern __shared__ unsigned char tma_decode_raw[];
@@ -547,6 +562,8 @@ paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache,
       qa2[ks] = g < group ? *reinterpret_cast<const uint32_t*>(qrow + ks * 16 + 8 + 2 * t) : 0u;
     }
   }
+  float near[4][2];
+  decode_biases(near, bias, kv * group + g, g < group, pos - key0 - warp * 32 - 2 * t);
   const bool keys_landed = barrier_wait(&barriers[0], 0, status);
 
   // ---- scores of this warp's 32 keys
@@ -576,7 +593,7 @@ paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache,
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int kk = key_base + nb * 8 + 2 * t + j;
-      sc[nb][j] = kk >= lo && kk <= hi ? capped_score(sc[nb][j] * scale, softcap) * kLog2E : -INFINITY;
+      sc[nb][j] = kk >= lo && kk <= hi ? (capped_score(sc[nb][j] * scale, softcap) + near[nb][j]) * kLog2E : -INFINITY;
       m_w = fmaxf(m_w, sc[nb][j]);
     }
   }
@@ -687,7 +704,7 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
                                        int max_pages, const int* __restrict__ row_token,
                                        const int* __restrict__ row_request, const int* __restrict__ positions,
                                        int heads, int kv_heads, int page_tokens, int num_pages, int max_splits,
-                                       int window, int chunk, float scale, float softcap, int* status) {
+                                       int window, int chunk, float scale, float softcap, ScoreBias bias, int* status) {
   constexpr int HALVES = HD / kTmaColumns;                 // 64-value halves of a row
   constexpr int TILE_BYTES = kSplitKeys * HD * 2;
   extern __shared__ unsigned char tma_decode_raw[];
@@ -787,6 +804,8 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
     const int key0 = tile * kSplitKeys;
     const int lo = max(first_key - key0, 0), hi = min(pos - key0, kSplitKeys - 1);   // the tile's rows that count
     const bool has_keys = key_base <= hi && key_base + 31 >= lo;
+    float near[4][2];
+    decode_biases(near, bias, kv * group + g, g < group, pos - key0 - warp * 32 - 2 * t);
     const bool keys_landed = barrier_wait(&barriers[0], parity, status);
 
     // ---- scores of this warp's 32 keys
@@ -813,7 +832,7 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int kk = key_base + nb * 8 + 2 * t + j;
-        sc[nb][j] = kk >= lo && kk <= hi ? capped_score(sc[nb][j] * scale, softcap) * kLog2E : -INFINITY;
+        sc[nb][j] = kk >= lo && kk <= hi ? (capped_score(sc[nb][j] * scale, softcap) + near[nb][j]) * kLog2E : -INFINITY;
         m_t = fmaxf(m_t, sc[nb][j]);
       }
     }
@@ -1014,6 +1033,8 @@ struct DecodeProject {
   int has_sink = 0;
   float sink_score = 0.0f;
   const float* sink_heads = nullptr;   // one score per query head instead (float32)
+  // A bias per head and distance on the scores (no table: none).
+  ScoreBias bias = {nullptr, 0};
 };
 
 template <typename T, int HD, int G>
@@ -1036,7 +1057,7 @@ static int launch_decode(const void* q, const void* cache, void* out, float* par
   kernel<<<grid, kDecodeThreads, shared, stream>>>(
       static_cast<const T*>(q), static_cast<const T*>(cache), partial, block_tables, max_pages,
       row_token, row_request, positions, heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk,
-      scale, project.softcap, status);
+      scale, project.softcap, project.bias, status);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return static_cast<int>(e);
   return static_cast<int>(launch_chained(paged_attention_merge_kernel<T>, dim3(rows, heads), dim3(HD <= 64 ? 64 : (HD <= 128 ? 128 : 256)), 0,
@@ -1101,7 +1122,7 @@ static int launch_decode_mma(const void* q, const void* cache, void* out, float*
       if (attribute != cudaSuccess) return static_cast<int>(attribute);
       e = launch_chained(kernel, dim3(slots, kv_heads, rows), dim3(kDecodeThreads), shared, stream, map_cache,
                          static_cast<const __nv_bfloat16*>(q), partial, block_tables, max_pages, row_token, row_request,
-                         positions, heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, project.softcap, status);
+                         positions, heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, project.softcap, project.bias, status);
       if (e != cudaSuccess) return static_cast<int>(e);
       return finish(slots);
     }
@@ -1110,7 +1131,7 @@ static int launch_decode_mma(const void* q, const void* cache, void* out, float*
     if (attribute != cudaSuccess) return static_cast<int>(attribute);
     e = launch_chained(kernel, grid, dim3(kDecodeThreads), shared, stream, map_cache,
                        static_cast<const __nv_bfloat16*>(q), partial, block_tables, max_pages, row_token, row_request,
-                       positions, heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, project.softcap, status);
+                       positions, heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, project.softcap, project.bias, status);
   } else {
     const int shared = 2 * kSplitKeys * (HD * 2 + 16);
     auto kernel = paged_attention_decode_mma_kernel<HD>;
@@ -1119,7 +1140,7 @@ static int launch_decode_mma(const void* q, const void* cache, void* out, float*
     e = launch_chained(kernel, grid, dim3(kDecodeThreads), shared, stream,
                        static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(cache),
                        partial, block_tables, max_pages, row_token, row_request, positions, heads,
-                       kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, project.softcap, status);
+                       kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, project.softcap, project.bias, status);
   }
   if (e != cudaSuccess) return static_cast<int>(e);
   return finish(0);
@@ -1160,8 +1181,10 @@ MXB_API int mxb_paged_attention_decode(const void* q, const void* cache, void* o
                                        int heads, int kv_heads, int head_dim, int page_tokens,
                                        int num_pages, int max_splits, int window, int chunk, float scale,
                                        int dtype, const void* gate, long long gate_stride, float softcap, int has_sink,
-                                       float sink_score, const float* sink_heads, int* status, cudaStream_t stream) {
+                                       float sink_score, const float* sink_heads, const float* bias_table, int bias_far,
+                                       int* status, cudaStream_t stream) {
   if (rows <= 0) return 0;
+  if (bias_table != nullptr && bias_far < 0) return static_cast<int>(cudaErrorInvalidValue);
   if (!mxb_paged_attention_decode_supported(head_dim, heads, kv_heads, dtype) || max_splits <= 0)
     return static_cast<int>(cudaErrorInvalidValue);
   const int group = heads / kv_heads;
@@ -1172,6 +1195,7 @@ MXB_API int mxb_paged_attention_decode(const void* q, const void* cache, void* o
   project.has_sink = has_sink;
   project.sink_score = sink_score;
   project.sink_heads = sink_heads;
+  project.bias = ScoreBias{bias_table, bias_far};
 #define ARGS q, cache, out, partial, block_tables, max_pages, row_token, row_request, positions, rows, \
              heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, status, stream, project
 #define BY_GROUP(T, HD)                                        \
@@ -1210,8 +1234,9 @@ MXB_API int mxb_paged_attention_decode_project(const void* q, const void* cache,
                                                int heads, int kv_heads, int head_dim, int page_tokens, int num_pages,
                                                int max_splits, int window, int chunk, float scale, const void* w, long long ldw,
                                                int hidden, float* summands, const void* gate, long long gate_stride,
-                                               float softcap, int has_sink, float sink_score, const float* sink_heads, int* status,
-                                               cudaStream_t stream) {
+                                               float softcap, int has_sink, float sink_score, const float* sink_heads,
+                                               const float* bias_table, int bias_far, int* status, cudaStream_t stream) {
+  if (bias_table != nullptr && bias_far < 0) return static_cast<int>(cudaErrorInvalidValue);
   if (rows <= 0 || hidden <= 0 || max_splits <= 0) return static_cast<int>(cudaErrorInvalidValue);
   if (!mxb_paged_attention_decode_project_supported(head_dim, heads, kv_heads, kBF16, tokens, w, ldw))
     return static_cast<int>(cudaErrorInvalidValue);
@@ -1227,6 +1252,7 @@ MXB_API int mxb_paged_attention_decode_project(const void* q, const void* cache,
   project.has_sink = has_sink;
   project.sink_score = sink_score;
   project.sink_heads = sink_heads;
+  project.bias = ScoreBias{bias_table, bias_far};
   void* out = nullptr;
 #define ARGS q, cache, out, partial, block_tables, max_pages, row_token, row_request, positions, rows, \
              heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, status, stream, project
@@ -1298,7 +1324,7 @@ MXB_API int mxb_paged_attention_decode_noalloc(const void* q, const void* cache,
   if (e != cudaSuccess) return static_cast<int>(e);
   return mxb_paged_attention_decode(q, cache, out, scratch, block_tables, max_pages, row_token,
                                     row_request, positions, rows, heads, kv_heads, head_dim, page_tokens,
-                                    num_pages, splits, window, 0, scale, dtype, nullptr, 0, 0.0f, 0, 0.0f, nullptr, status, stream);
+                                    num_pages, splits, window, 0, scale, dtype, nullptr, 0, 0.0f, 0, 0.0f, nullptr, nullptr, 0, status, stream);
 }
 
 MXB_TIMELINE_EXPORT(mxb_timeline_attention)

@@ -75,7 +75,7 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
                      const int* __restrict__ tile_length, const int* __restrict__ positions, int heads,
                      int kv_heads, int page_tokens, int num_pages, int window, int chunk, float scale, float softcap,
                      const __nv_bfloat16* __restrict__ gate, long long gate_stride, int has_sink, float sink_log2, const float* __restrict__ sink_heads,
-                     int* status) {
+                     ScoreBias bias, int* status) {
   constexpr int CHUNKS = HD / 8;                      // 16-byte chunks per row
   constexpr int TILE_BYTES = kFlashKeys * HD * 2;
   extern __shared__ __align__(128) unsigned char shared[];
@@ -200,6 +200,20 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
         for (int j = 0; j < 4; ++j) s[nb][j] = outer * tanhf(s[nb][j] * inner);
       }
     }
+    // ---- a bias per head and distance, if any, kept over scale as well
+    if (bias.table != nullptr) {
+      const float* table = bias.row(head);
+      const float over = 1.0f / scale;
+#pragma unroll
+      for (int nb = 0; nb < kFlashKeys / 8; ++nb) {
+#pragma unroll
+        for (int j = 0; j < 2; ++j) {
+          const int key = kt * kFlashKeys + nb * 8 + 2 * t + j;
+          s[nb][j] = fmaf(bias_at(table, pos_lo - key, bias.far), over, s[nb][j]);
+          s[nb][2 + j] = fmaf(bias_at(table, pos_hi - key, bias.far), over, s[nb][2 + j]);
+        }
+      }
+    }
     // ---- mask, running maximum and sum (float32). m_* hold the running
     // maximum already multiplied by scale * log2(e).
     const int key0 = kt * kFlashKeys;
@@ -306,7 +320,8 @@ static int launch_flash(const void* q, const void* cache, void* out, const int* 
                         const int* tile_request, const int* tile_start, const int* tile_length,
                         const int* positions, int tiles, int heads, int kv_heads, int page_tokens,
                         int num_pages, int window, int chunk, float scale, const void* gate, long long gate_stride,
-                        float softcap, int has_sink, float sink_score, const float* sink_heads, int* status, cudaStream_t stream) {
+                        float softcap, int has_sink, float sink_score, const float* sink_heads, ScoreBias bias, int* status,
+                        cudaStream_t stream) {
   const int shared = 4 * kFlashKeys * HD * 2;
   auto kernel = flash_prefill_kernel<HD>;
   cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, shared);
@@ -316,7 +331,7 @@ static int launch_flash(const void* q, const void* cache, void* out, const int* 
       static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(cache),
       static_cast<__nv_bfloat16*>(out), block_tables, max_pages, tile_request, tile_start, tile_length,
       positions, heads, kv_heads, page_tokens, num_pages, window, chunk, scale, softcap,
-      static_cast<const __nv_bfloat16*>(gate), gate_stride, has_sink, sink_score * 1.4426950408889634f, sink_heads, status);
+      static_cast<const __nv_bfloat16*>(gate), gate_stride, has_sink, sink_score * 1.4426950408889634f, sink_heads, bias, status);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -339,14 +354,17 @@ MXB_API int mxb_flash_prefill(const void* q, const void* cache, void* out, const
                               const int* tile_length, const int* positions, int tiles, int heads,
                               int kv_heads, int head_dim, int page_tokens, int num_pages, int window, int chunk,
                               float scale, int dtype, const void* gate, long long gate_stride, float softcap,
-                              int has_sink, float sink_score, const float* sink_heads, int* status, cudaStream_t stream) {
+                              int has_sink, float sink_score, const float* sink_heads, const float* bias_table,
+                              int bias_far, int* status, cudaStream_t stream) {
   if (tiles <= 0) return 0;
   if (!mxb_flash_prefill_supported(head_dim, heads, kv_heads, dtype)) return static_cast<int>(cudaErrorInvalidValue);
+  if (bias_table != nullptr && bias_far < 0) return static_cast<int>(cudaErrorInvalidValue);
+  const ScoreBias bias = {bias_table, bias_far};
   if (head_dim == 64)
     return launch_flash<64>(q, cache, out, block_tables, max_pages, tile_request, tile_start, tile_length,
                             positions, tiles, heads, kv_heads, page_tokens, num_pages, window, chunk, scale, gate, gate_stride, softcap, has_sink,
-                            sink_score, sink_heads, status, stream);
+                            sink_score, sink_heads, bias, status, stream);
   return launch_flash<128>(q, cache, out, block_tables, max_pages, tile_request, tile_start, tile_length,
                            positions, tiles, heads, kv_heads, page_tokens, num_pages, window, chunk, scale, gate, gate_stride, softcap, has_sink,
-                            sink_score, sink_heads, status, stream);
+                            sink_score, sink_heads, bias, status, stream);
 }

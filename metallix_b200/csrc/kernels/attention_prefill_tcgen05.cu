@@ -77,7 +77,8 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
                              const int* __restrict__ tile_length, const int* __restrict__ positions, int heads,
                              int kv_heads, int page_tokens, int num_pages, int window, int chunk, float scale, float softcap,
                              int shared_bytes, float* __restrict__ partial, const __nv_bfloat16* __restrict__ gate,
-                             long long gate_stride, int has_sink, float sink_log2, const float* __restrict__ sink_heads, int* status) {
+                             long long gate_stride, int has_sink, float sink_log2, const float* __restrict__ sink_heads,
+                             ScoreBias bias, int bias_bytes, int* status) {
   using Config = FaConfig<HD>;
   constexpr int MAX_STAGES = Config::kKeyStages;
   constexpr int HALVES = Config::kHalves;
@@ -87,7 +88,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
   extern __shared__ unsigned char fa_shared_raw[];
   const int slack = (1024 - (shared_address(fa_shared_raw) & 1023)) & 1023;
   const int VS = Config::kValueStages;
-  const int fitting = (shared_bytes - slack - Config::kSmallBytes) / Config::kTileBytes - 1 - VS;
+  const int fitting = (shared_bytes - slack - Config::kSmallBytes - bias_bytes) / Config::kTileBytes - 1 - VS;
   const int KS = fitting < MAX_STAGES ? fitting : MAX_STAGES;
   if (KS < 1) {  // the launcher asks for more than that
     if (threadIdx.x == 0) atomicOr(status, kStatusWaitTimeout);
@@ -111,6 +112,8 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
   volatile int& failed = *reinterpret_cast<volatile int*>(&tmem_base_slot + 1);
   // [tile parity][part][row]: the threads of a row exchange maxima (and, at the end, sums)
   float (*row_max)[kFaParts][kFaRows] = reinterpret_cast<float (*)[kFaParts][kFaRows]>(small + 512);
+  // This head's biases by distance, where they fit (bias_bytes > 0); else they are read where they lie.
+  float* near_bias = reinterpret_cast<float*>(small + Config::kSmallBytes);
   static_assert((1 + 4 * MAX_STAGES + 8 + 4 + 1) * 8 + 8 <= 512, "the barriers do not fit their area");
 
   const int head = blockIdx.x, tile = blockIdx.y;  // heads of one tile run side by side and share its keys in L2
@@ -149,6 +152,8 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
     barrier_init_fence();
     failed = 0;
   }
+  if (bias_bytes > 0)
+    for (int i = threadIdx.x; i <= bias.far; i += kFaThreads) near_bias[i] = bias.row(head)[i];
   if (warp == 1) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n"
                  ::"r"(shared_address(&tmem_base_slot)), "r"(kFaTmemColumns) : "memory");
@@ -302,6 +307,8 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
     const float scale_log2 = scale * 1.4426950408889634f;
     const uint32_t tmem_lane = tmem_base + (static_cast<uint32_t>(lane_base) << 16);
     uint64_t* meet = &row_ready[warp & 3];
+    const float* bias_row = bias.table == nullptr ? nullptr : (bias_bytes > 0 ? near_bias : bias.row(head));
+    const float over_scale = 1.0f / scale;
     float acc[PART_HD];
 #pragma unroll
     for (int i = 0; i < PART_HD; ++i) acc[i] = 0.0f;
@@ -334,6 +341,18 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
         const float inner = scale / softcap, outer = softcap / scale;
 #pragma unroll
         for (int j = 0; j < PART_KEYS; ++j) raw[j] = __float_as_uint(outer * tanhf(__uint_as_float(raw[j]) * inner));
+      }
+      if (bias.table != nullptr) {   // over scale as well; keys from bias.far positions back on share one number
+        const int back = pos - key0;
+        if (back - (PART_KEYS - 1) >= bias.far) {
+          const float far = bias_row[bias.far] * over_scale;
+#pragma unroll
+          for (int j = 0; j < PART_KEYS; ++j) raw[j] = __float_as_uint(__uint_as_float(raw[j]) + far);
+        } else {
+#pragma unroll
+          for (int j = 0; j < PART_KEYS; ++j)
+            raw[j] = __float_as_uint(fmaf(bias_at(bias_row, back - j, bias.far), over_scale, __uint_as_float(raw[j])));
+        }
       }
       if (all_seen) {
 #pragma unroll
@@ -483,7 +502,7 @@ static int launch_flash_tc(const void* q, const void* cache, void* out, const in
                            const int* positions, int tokens, int tiles, int heads, int kv_heads, int page_tokens,
                            int num_pages, int window, int chunk, float scale, int key_shares, float* partial,
                            const void* gate, long long gate_stride, float softcap, int has_sink, float sink_score, const float* sink_heads,
-                           int* status, cudaStream_t stream) {
+                           ScoreBias bias, int* status, cudaStream_t stream) {
   using Config = FaConfig<HD>;
   const float sink_log2 = sink_score * 1.4426950408889634f;
   CUtensorMap map_q, map_cache;
@@ -500,7 +519,10 @@ static int launch_flash_tc(const void* q, const void* cache, void* out, const in
     cudaGetDevice(&device);
     cudaDeviceGetAttribute(&shared_limit, cudaDevAttrMaxSharedMemoryPerBlockOptin, device);
   }
-  const int shared_bytes = Config::kSharedBytes < shared_limit ? Config::kSharedBytes : shared_limit;
+  const int staged = bias.table != nullptr && bias.far < 1 << 20 ? ((bias.far + 1) * 4 + 15) / 16 * 16 : 0;
+  const int bias_bytes = staged > 0 && Config::kSharedBytes + staged <= shared_limit ? staged : 0;
+  const int wanted = Config::kSharedBytes + bias_bytes;
+  const int shared_bytes = wanted < shared_limit ? wanted : shared_limit;
   cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, shared_bytes);
   if (e != cudaSuccess) return static_cast<int>(e);
   const bool shared_out = key_shares > 1;
@@ -508,7 +530,8 @@ static int launch_flash_tc(const void* q, const void* cache, void* out, const in
   kernel<<<grid, kFaThreads, shared_bytes, stream>>>(
       map_q, map_cache, static_cast<__nv_bfloat16*>(out), block_tables, max_pages, tile_request, tile_start,
       tile_length, positions, heads, kv_heads, page_tokens, num_pages, window, chunk, scale, softcap, shared_bytes,
-      shared_out ? partial : nullptr, static_cast<const __nv_bfloat16*>(gate), gate_stride, has_sink, sink_log2, sink_heads, status);
+      shared_out ? partial : nullptr, static_cast<const __nv_bfloat16*>(gate), gate_stride, has_sink, sink_log2, sink_heads,
+      bias, bias_bytes, status);
   e = cudaGetLastError();
   if (e != cudaSuccess || !shared_out) return static_cast<int>(e);
   flash_prefill_merge_kernel<HD><<<dim3(heads, tiles, kMergeGroups), HD, 0, stream>>>(
@@ -541,7 +564,8 @@ MXB_API int mxb_flash_prefill_tcgen05(const void* q, const void* cache, void* ou
                                       int heads, int kv_heads, int head_dim, int page_tokens, int num_pages,
                                       int window, int chunk, float scale, int dtype, int key_shares, float* partial,
                                       const void* gate, long long gate_stride, float softcap, int has_sink,
-                                      float sink_score, const float* sink_heads, int* status, cudaStream_t stream) {
+                                      float sink_score, const float* sink_heads, const float* bias_table, int bias_far,
+                                      int* status, cudaStream_t stream) {
   if (tiles <= 0) return 0;
   if (key_shares < 1 || key_shares > kMergeShares || (key_shares > 1 && partial == nullptr))
     return static_cast<int>(cudaErrorInvalidValue);
@@ -550,11 +574,13 @@ MXB_API int mxb_flash_prefill_tcgen05(const void* q, const void* cache, void* ou
   if ((reinterpret_cast<uintptr_t>(q) & 15) || (reinterpret_cast<uintptr_t>(cache) & 15) ||
       (reinterpret_cast<uintptr_t>(out) & 15) || (reinterpret_cast<uintptr_t>(gate) & 15) || ((gate_stride * 2) & 15))
     return static_cast<int>(cudaErrorInvalidValue);
+  if (bias_table != nullptr && bias_far < 0) return static_cast<int>(cudaErrorInvalidValue);
+  const ScoreBias bias = {bias_table, bias_far};
   if (head_dim == 64)
     return launch_flash_tc<64>(q, cache, out, block_tables, max_pages, tile_request, tile_start, tile_length,
                                positions, tokens, tiles, heads, kv_heads, page_tokens, num_pages, window, chunk, scale,
-                               key_shares, partial, gate, gate_stride, softcap, has_sink, sink_score, sink_heads, status, stream);
+                               key_shares, partial, gate, gate_stride, softcap, has_sink, sink_score, sink_heads, bias, status, stream);
   return launch_flash_tc<128>(q, cache, out, block_tables, max_pages, tile_request, tile_start, tile_length,
                               positions, tokens, tiles, heads, kv_heads, page_tokens, num_pages, window, chunk, scale,
-                              key_shares, partial, gate, gate_stride, softcap, has_sink, sink_score, sink_heads, status, stream);
+                              key_shares, partial, gate, gate_stride, softcap, has_sink, sink_score, sink_heads, bias, status, stream);
 }

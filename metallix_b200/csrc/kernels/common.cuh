@@ -72,15 +72,36 @@ __device__ __forceinline__ float sigmoid_of(float g) { return 1.0f / (1.0f + exp
 
 // The activation of a gated feed-forward, act(gate) * up: silu(z) = z / (1 + e^-z), or the tanh form of
 // gelu, 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))).
-enum GateActivation : int { kActSilu = 0, kActGeluTanh = 1 };
+// A third, with clamped halves: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(1.702 g) (u + 1).
+enum GateActivation : int { kActSilu = 0, kActGeluTanh = 1, kActClamped = 2 };
+constexpr float kClampedSlope = 1.702f;
 __device__ __forceinline__ float gate_activation(float z, int activation) {
   if (activation == kActGeluTanh) return 0.5f * z * (1.0f + tanhf(0.7978845608028654f * fmaf(0.044715f * z * z, z, z)));
   return __fdividef(z, 1.0f + __expf(-z));
+}
+// What a gated feed-forward hands on from one gate and one up value (rounded to bfloat16 by whoever stores it).
+__device__ __forceinline__ float gated_product(float gate, float up, int activation, float limit) {
+  if (activation == kActClamped) {
+    gate = fminf(gate, limit);
+    up = fminf(fmaxf(up, -limit), limit);
+    return __fdividef(gate, 1.0f + __expf(-kClampedSlope * gate)) * (up + 1.0f);
+  }
+  return gate_activation(gate, activation) * up;
 }
 
 // A cap c on a scaled score ahead of the softmax: s <- c tanh(s / c), which keeps small scores and
 // bounds all of them to (-c, c); c = 0 leaves the score as it is.
 __device__ __forceinline__ float capped_score(float s, float cap) { return cap > 0.0f ? cap * tanhf(s / cap) : s; }
+
+// A bias per head and distance that joins a scaled (and capped) score ahead of the softmax: `table` is float32
+// [heads, far + 1], entry n for a key n positions back, the last entry for every key at least `far` back.
+// A null table: none.
+struct ScoreBias {
+  const float* table;
+  int far;
+  __device__ __forceinline__ const float* row(int head) const { return table + static_cast<size_t>(head) * (far + 1); }
+};
+__device__ __forceinline__ float bias_at(const float* row, int distance, int far) { return row[min(max(distance, 0), far)]; }
 
 // The first key a query at position `pos` sees. Two rules, either or both:
 // a sliding window keeps the last `window` positions (keys > pos - window), a

@@ -1,5 +1,7 @@
-// The gated delta rule with one decay per head and key channel, state per
-// request in the cache's slots, float32 throughout.
+// Matrix-state recurrences over the tokens of a request, the state kept per
+// request in the cache's slots, float32 throughout: the gated delta rule with
+// one decay per head and key channel, the same with one decay per head, and
+// the state-space dual (Mamba-2), which writes without looking first.
 //
 // Per head, with key width D and value width V, a request carries a matrix
 // S [D, V]. A token brings q, k (D values each, from one of G groups that
@@ -9,6 +11,12 @@
 //   qn = q / sqrt(sum q^2 + 1e-6) * D^-1/2,   kn = k / sqrt(sum k^2 + 1e-6)
 //   beta = sigmoid(b),   g_d = exp(-a_h * softplus(s_d + bias_d))
 //   S <- g (rows) * S;  u = beta (v - S^T kn);  S <- S + kn u^T;  o = S^T qn
+//
+// With one decay per head, g is one number, exp(-a_h softplus(s + bias)), from
+// one pre-activation per head. The dual takes q = C, k = B and v = x as they
+// come, dt = softplus(s + bias) in place of beta, g = exp(-a_h dt), and
+//
+//   S <- g S + k (dt v)^T;   o = S^T q + skip_h v
 //
 // Every value column of S goes its own way: column j needs only v_j and what
 // all columns share (qn, kn, g, beta). A block owns some of the columns of
@@ -27,6 +35,7 @@
 
 namespace mxb {
 
+enum DeltaMode : int { kDeltaChannel = 0, kDeltaHead = 1, kDeltaDual = 2 };
 constexpr int kDeltaMaxWarps = 8;     // tokens of a batch: one warp prepares each (a block of fewer warps takes fewer)
 
 // Where channel d of a shared vector lies: every lane's quarter starts 4 floats further than a
@@ -34,20 +43,25 @@ constexpr int kDeltaMaxWarps = 8;     // tokens of a batch: one warp prepares ea
 template <int DPT>
 __device__ __forceinline__ int delta_slot(int d) { return d + (d / DPT) * 4; }
 
+__device__ __forceinline__ float delta_softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
+
 // LANES lanes share a value column, each with DPT of its key channels; COLS neighbouring columns a thread.
-template <typename T, int DPT, int LANES, int COLS>
+// MODE: see DeltaMode; `step_pre` is float32 [.., heads * dim] with a decay per channel, else of T with one value per head.
+template <typename T, int DPT, int LANES, int COLS, int MODE>
 __global__ void __launch_bounds__(512)
 delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off, int v_off,
                   const T* __restrict__ beta_pre, long long ldb, int b_off,
-                  const float* __restrict__ step_pre, long long lds, const float* __restrict__ step_bias,
-                  const float* __restrict__ rate, float* __restrict__ state, long long slot_stride, int num_slots,
+                  const void* __restrict__ step_pre, long long lds, const float* __restrict__ step_bias,
+                  const float* __restrict__ rate, const float* __restrict__ skip, float* __restrict__ state, long long slot_stride, int num_slots,
                   const int* __restrict__ row_start, const int* __restrict__ row_length,
                   const int* __restrict__ request_slots, float* __restrict__ out, int heads, int groups, int dim,
                   int vdim, int* status) {
   constexpr int PITCH = LANES * (DPT + 4);
   constexpr int NL = (LANES * DPT + 31) / 32;   // channels a lane prepares for its warp's token
-  __shared__ __align__(16) float s_q[kDeltaMaxWarps][PITCH], s_k[kDeltaMaxWarps][PITCH], s_g[kDeltaMaxWarps][PITCH];
-  __shared__ float s_beta[kDeltaMaxWarps], s_qk[kDeltaMaxWarps];
+  constexpr bool PER_CHANNEL = MODE == kDeltaChannel;
+  __shared__ __align__(16) float s_q[kDeltaMaxWarps][PITCH], s_k[kDeltaMaxWarps][PITCH];
+  __shared__ __align__(16) float s_g[PER_CHANNEL ? kDeltaMaxWarps : 1][PER_CHANNEL ? PITCH : 4];
+  __shared__ float s_beta[kDeltaMaxWarps], s_qk[kDeltaMaxWarps], s_decay[kDeltaMaxWarps];
   const int row = blockIdx.x, head = blockIdx.y;
   const int length = row_length[row];
   if (length <= 0) return;   // a padding row owns no state
@@ -69,14 +83,16 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
   const float head_rate = rate[head];
   // zeros in the shared vectors' padding channels (dim .. 4 * DPT), once: they are never written again
   for (int i = threadIdx.x; i < kDeltaMaxWarps * PITCH; i += blockDim.x) {
-    (&s_q[0][0])[i] = 0.0f; (&s_k[0][0])[i] = 0.0f; (&s_g[0][0])[i] = 0.0f;
+    (&s_q[0][0])[i] = 0.0f; (&s_k[0][0])[i] = 0.0f;
+    if (PER_CHANNEL) (&s_g[0][0])[i] = 0.0f;
   }
   float bias[NL];
 #pragma unroll
   for (int i = 0; i < NL; ++i) {
     const int d = lane + 32 * i;
-    bias[i] = d < dim ? step_bias[head * dim + d] : 0.0f;
+    bias[i] = !PER_CHANNEL ? step_bias[head] : (d < dim ? step_bias[head * dim + d] : 0.0f);
   }
+  const float head_skip = MODE == kDeltaDual ? skip[head] : 0.0f;
   // this thread's quarter of its columns of S
   float s[COLS][DPT];
   // In memory a column's channels lie side by side ([heads, vdim, dim]): a lane's share is one run of DPT values.
@@ -97,15 +113,16 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
       const long long t = first + base + warp;
       const T* q_row = qkv + t * ld + q_off + group * dim;
       const T* k_row = qkv + t * ld + k_off + group * dim;
-      const float* step_row = step_pre + t * lds + head * dim;
+      const float* step_row = static_cast<const float*>(step_pre) + t * lds + head * dim;   // with a decay per channel
 #pragma unroll
       for (int i = 0; i < NL; ++i) {
         const int d = lane + 32 * i;
         raw_q[i] = d < dim ? to_float(q_row[d]) : 0.0f;
         raw_k[i] = d < dim ? to_float(k_row[d]) : 0.0f;
-        raw_step[i] = d < dim ? step_row[d] : 0.0f;
+        if (PER_CHANNEL) raw_step[i] = d < dim ? step_row[d] : 0.0f;
       }
-      raw_beta = to_float(beta_pre[t * ldb + b_off + head]);
+      if (!PER_CHANNEL) raw_step[0] = to_float(static_cast<const T*>(step_pre)[t * lds + head]);
+      if (MODE != kDeltaDual) raw_beta = to_float(beta_pre[t * ldb + b_off + head]);
     }
 #pragma unroll
     for (int j = 0; j < kDeltaMaxWarps; ++j)
@@ -125,22 +142,27 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
       for (int i = 0; i < NL; ++i) {
         qq = fmaf(raw_q[i], raw_q[i], qq); kk = fmaf(raw_k[i], raw_k[i], kk); qk = fmaf(raw_q[i], raw_k[i], qk);
       }
-      qq = warp_sum(qq); kk = warp_sum(kk); qk = warp_sum(qk);
-      const float q_unit = rsqrtf(qq + 1e-6f) * q_scale, k_unit = rsqrtf(kk + 1e-6f);
+      qk = warp_sum(qk);
+      float q_unit = 1.0f, k_unit = 1.0f;
+      if (MODE != kDeltaDual) {
+        qq = warp_sum(qq); kk = warp_sum(kk);
+        q_unit = rsqrtf(qq + 1e-6f) * q_scale;
+        k_unit = rsqrtf(kk + 1e-6f);
+      }
 #pragma unroll
       for (int i = 0; i < NL; ++i) {
         const int d = lane + 32 * i;
         if (d < dim) {
-          const float z = raw_step[i] + bias[i];
-          const float softplus = z > 20.0f ? z : log1pf(expf(z));
           const int at = delta_slot<DPT>(d);
           s_q[warp][at] = raw_q[i] * q_unit;
           s_k[warp][at] = raw_k[i] * k_unit;
-          s_g[warp][at] = expf(-head_rate * softplus);
+          if (PER_CHANNEL) s_g[warp][at] = expf(-head_rate * delta_softplus(raw_step[i] + bias[i]));
         }
       }
       if (lane == 0) {
-        s_beta[warp] = sigmoid_of(raw_beta);
+        const float step = PER_CHANNEL ? 0.0f : delta_softplus(raw_step[0] + bias[0]);
+        if (!PER_CHANNEL) s_decay[warp] = expf(-head_rate * step);
+        s_beta[warp] = MODE == kDeltaDual ? step : sigmoid_of(raw_beta);
         s_qk[warp] = qk * q_unit * k_unit;
       }
     }
@@ -156,7 +178,8 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
       if (j >= batch) break;
       const float4* q4 = reinterpret_cast<const float4*>(&s_q[j][part * (DPT + 4)]);
       const float4* k4 = reinterpret_cast<const float4*>(&s_k[j][part * (DPT + 4)]);
-      const float4* g4 = reinterpret_cast<const float4*>(&s_g[j][part * (DPT + 4)]);
+      const float4* g4 = reinterpret_cast<const float4*>(&s_g[PER_CHANNEL ? j : 0][PER_CHANNEL ? part * (DPT + 4) : 0]);
+      const float decay = PER_CHANNEL ? 0.0f : s_decay[j];
       // Shared memory's read rate paces the walk: what is read once (decay, key, query) serves all of the
       // thread's columns, and the key stays in registers for the write where there is room for it.
       constexpr bool KEEP = DPT * COLS <= 32;
@@ -165,13 +188,15 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
       for (int c = 0; c < COLS; ++c) k_dot[c] = q_dot[c] = 0.0f;
 #pragma unroll
       for (int i = 0; i < DPT; i += 4) {
-        const float4 g = g4[i / 4], k = k4[i / 4], q = q4[i / 4];
+        const float4 g = PER_CHANNEL ? g4[i / 4] : make_float4(decay, decay, decay, decay), k = k4[i / 4], q = q4[i / 4];
         if (KEEP) { kept[i] = k.x; kept[i + 1] = k.y; kept[i + 2] = k.z; kept[i + 3] = k.w; }
 #pragma unroll
         for (int c = 0; c < COLS; ++c) {
           s[c][i] *= g.x; s[c][i + 1] *= g.y; s[c][i + 2] *= g.z; s[c][i + 3] *= g.w;
-          k_dot[c] = fmaf(k.x, s[c][i], k_dot[c]); k_dot[c] = fmaf(k.y, s[c][i + 1], k_dot[c]);
-          k_dot[c] = fmaf(k.z, s[c][i + 2], k_dot[c]); k_dot[c] = fmaf(k.w, s[c][i + 3], k_dot[c]);
+          if (MODE != kDeltaDual) {
+            k_dot[c] = fmaf(k.x, s[c][i], k_dot[c]); k_dot[c] = fmaf(k.y, s[c][i + 1], k_dot[c]);
+            k_dot[c] = fmaf(k.z, s[c][i + 2], k_dot[c]); k_dot[c] = fmaf(k.w, s[c][i + 3], k_dot[c]);
+          }
           q_dot[c] = fmaf(q.x, s[c][i], q_dot[c]); q_dot[c] = fmaf(q.y, s[c][i + 1], q_dot[c]);
           q_dot[c] = fmaf(q.z, s[c][i + 2], q_dot[c]); q_dot[c] = fmaf(q.w, s[c][i + 3], q_dot[c]);
         }
@@ -181,7 +206,7 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
       for (int c = 0; c < COLS; ++c) {
 #pragma unroll
         for (int offset = 1; offset < LANES; offset <<= 1) {   // over the lanes that share the column
-          k_dot[c] += __shfl_xor_sync(0xffffffffu, k_dot[c], offset);
+          if (MODE != kDeltaDual) k_dot[c] += __shfl_xor_sync(0xffffffffu, k_dot[c], offset);
           q_dot[c] += __shfl_xor_sync(0xffffffffu, q_dot[c], offset);
         }
         u[c] = s_beta[j] * (v[j][c] - k_dot[c]);
@@ -202,7 +227,7 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
         for (int c = 0; c < COLS; ++c)
           if (live[c])
             out[(static_cast<long long>(first + base + j)) * (static_cast<long long>(heads) * vdim) + head * vdim + column + c] =
-                fmaf(s_qk[j], u[c], q_dot[c]);
+                fmaf(s_qk[j], u[c], q_dot[c]) + (MODE == kDeltaDual ? head_skip * v[j][c] : 0.0f);
       }
     }
   }
@@ -230,13 +255,19 @@ MXB_API int mxb_delta_rule_max_dim() { return 256; }
 // values apart, advanced in place. Row r brings row_length[r]
 // tokens (0: a padding row, nothing is read or written) from packed token row_start[r] on and owns slot
 // request_slots[r]. out: float32 [tokens, heads * vdim]. longest: the most tokens any row brings, 0 if unknown.
+// mode 0: the above. mode 1: one decay per head; step_pre is [tokens, lds] of `dtype` with one pre-activation per
+// head, step_bias [heads]. mode 2, the state-space dual: as mode 1, with q, k and v taken as they come (C, B, x),
+// softplus(step) in place of sigmoid(beta), no look at the state before the write, and skip (float32 [heads]) times v
+// added to what is read; beta_pre is not read.
 MXB_API int mxb_delta_rule(const void* qkv, long long ld, int q_off, int k_off, int v_off, const void* beta_pre,
-                           long long ldb, int b_off, const float* step_pre, long long lds, const float* step_bias,
-                           const float* rate, float* state, long long slot_stride, int num_slots,
+                           long long ldb, int b_off, const void* step_pre, long long lds, const float* step_bias,
+                           const float* rate, const float* skip, int mode, float* state, long long slot_stride, int num_slots,
                            const int* row_start, const int* row_length, const int* request_slots, float* out,
                            int rows, int heads, int groups, int dim, int vdim, int dtype, int longest, int* status,
                            cudaStream_t stream) {
   if (rows <= 0) return 0;
+  if (mode < kDeltaChannel || mode > kDeltaDual || (mode == kDeltaDual) != (skip != nullptr))
+    return static_cast<int>(cudaErrorInvalidValue);
   if (heads <= 0 || groups <= 0 || heads % groups != 0 || dim <= 0 || dim > mxb_delta_rule_max_dim() || vdim <= 0)
     return static_cast<int>(cudaErrorInvalidValue);
   // Lanes a column and channels a lane by the key width; a block has up to 512 threads and as many columns as
@@ -254,20 +285,25 @@ MXB_API int mxb_delta_rule(const void* qkv, long long ld, int q_off, int k_off, 
     columns /= 2;
   columns = ((columns + step - 1) / step) * step;
   const dim3 grid(rows, heads, (vdim + columns - 1) / columns), block(columns * lanes);
-#define LAUNCH(T, DPT, LANES)                                                                                       \
-  delta_rule_kernel<T, DPT, LANES, 1><<<grid, block, 0, stream>>>(static_cast<const T*>(qkv), ld, q_off, k_off,      \
-      v_off, static_cast<const T*>(beta_pre), ldb, b_off, step_pre, lds, step_bias, rate, state, slot_stride,       \
+#define LAUNCH_MODE(T, DPT, LANES, MODE)                                                                            \
+  delta_rule_kernel<T, DPT, LANES, 1, MODE><<<grid, block, 0, stream>>>(static_cast<const T*>(qkv), ld, q_off, k_off,      \
+      v_off, static_cast<const T*>(beta_pre), ldb, b_off, step_pre, lds, step_bias, rate, skip, state, slot_stride, \
       num_slots, row_start, row_length, request_slots, out, heads, groups, dim, vdim, status)
+#define LAUNCH(T, DPT, LANES)                                        \
+  if (mode == kDeltaChannel) LAUNCH_MODE(T, DPT, LANES, kDeltaChannel);   \
+  else if (mode == kDeltaHead) LAUNCH_MODE(T, DPT, LANES, kDeltaHead);    \
+  else LAUNCH_MODE(T, DPT, LANES, kDeltaDual)
 #define BY_DIM(T)                                                   \
-  if (lanes == 4 && per_lane == 4) LAUNCH(T, 4, 4);                 \
-  else if (lanes == 4) LAUNCH(T, 8, 4);                             \
-  else if (lanes == 8) LAUNCH(T, 8, 8);                             \
-  else if (per_lane == 8) LAUNCH(T, 8, 16);                         \
-  else LAUNCH(T, 16, 16);
+  if (lanes == 4 && per_lane == 4) { LAUNCH(T, 4, 4); }             \
+  else if (lanes == 4) { LAUNCH(T, 8, 4); }                         \
+  else if (lanes == 8) { LAUNCH(T, 8, 8); }                         \
+  else if (per_lane == 8) { LAUNCH(T, 8, 16); }                     \
+  else { LAUNCH(T, 16, 16); }
   if (dtype == kF32) { BY_DIM(float) }
   else if (dtype == kBF16) { BY_DIM(__nv_bfloat16) }
   else return static_cast<int>(cudaErrorInvalidValue);
 #undef BY_DIM
 #undef LAUNCH
+#undef LAUNCH_MODE
   return static_cast<int>(cudaGetLastError());
 }

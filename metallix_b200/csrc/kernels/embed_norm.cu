@@ -57,12 +57,12 @@ __global__ void rmsnorm_kernel(TOut* __restrict__ y, const TIn* __restrict__ x,
 template <typename TDelta, typename TOut>
 __global__ void add_rmsnorm_kernel(float* __restrict__ x, const TDelta* __restrict__ delta,
                                    TOut* __restrict__ y, const float* __restrict__ w, int size,
-                                   float eps) {
+                                   size_t delta_stride, float eps) {
   __shared__ float scratch[33];
   const size_t base = static_cast<size_t>(blockIdx.x) * size;
   float sum = 0.0f;
   for (int i = threadIdx.x; i < size; i += blockDim.x) {
-    const float v = x[base + i] + to_float(delta[base + i]);
+    const float v = x[base + i] + to_float(delta[blockIdx.x * delta_stride + i]);
     x[base + i] = v;
     sum += v * v;
   }
@@ -95,7 +95,7 @@ __device__ __forceinline__ void store4(__nv_bfloat16* p, float4 v) {
 template <typename TDelta, typename TOut, bool ADD>
 __global__ void add_rmsnorm_vec4_kernel(float* __restrict__ x, const TDelta* __restrict__ delta,
                                         TOut* __restrict__ y, const float* __restrict__ w,
-                                        const int* __restrict__ rows_index, int size, float eps) {
+                                        const int* __restrict__ rows_index, int size, size_t delta_stride, float eps) {
   __shared__ float scratch[33];
   chain_release();
   const size_t src = rows_index ? static_cast<size_t>(rows_index[blockIdx.x]) : static_cast<size_t>(blockIdx.x);
@@ -113,7 +113,7 @@ __global__ void add_rmsnorm_vec4_kernel(float* __restrict__ x, const TDelta* __r
   for (int i = first; i < size; i += blockDim.x * 4) {
     float4 v = load4(row + i);
     if (ADD) {
-      const float4 d = load4(delta + src * size + i);
+      const float4 d = load4(delta + src * delta_stride + i);
       v.x += d.x; v.y += d.y; v.z += d.z; v.w += d.w;
       store4(row + i, v);
     }
@@ -205,15 +205,15 @@ add_summands_rmsnorm_kernel(float* __restrict__ x, const float* __restrict__ sum
 
 static bool aligned16(const void* p) { return reinterpret_cast<uintptr_t>(p) % 16 == 0; }
 
-// x[r, :] += delta[r, :] alone (the last residual sum of a model).
+// x[r, :] += delta[r, :] alone (the last residual sum of a model); delta may be shorter than x and starts over then.
 template <typename TDelta>
-__global__ void add_kernel(float* __restrict__ x, const TDelta* __restrict__ delta, size_t count) {
+__global__ void add_kernel(float* __restrict__ x, const TDelta* __restrict__ delta, size_t count, size_t period) {
   chain_release();
   chain_wait();
   x = behind_wait(x);
   delta = behind_wait(delta);
   const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
-  if (i < count) x[i] += to_float(delta[i]);
+  if (i < count) x[i] += to_float(delta[period == count ? i : i % period]);
 }
 
 static int norm_threads(int size) {
@@ -247,10 +247,10 @@ MXB_API int mxb_rmsnorm(void* y, int y_dtype, const void* x, int x_dtype, const 
     float* xs = const_cast<float*>(static_cast<const float*>(x));  // read only: ADD is false
     if (y_dtype == kF32)
       return static_cast<int>(launch_chained(add_rmsnorm_vec4_kernel<float, float, false>, dim3(rows), dim3(vec_threads), 0,
-                                             stream, xs, static_cast<const float*>(nullptr), static_cast<float*>(y), w, rows_index, size, eps));
+                                             stream, xs, static_cast<const float*>(nullptr), static_cast<float*>(y), w, rows_index, size, size_t{0}, eps));
     if (y_dtype == kBF16)
       return static_cast<int>(launch_chained(add_rmsnorm_vec4_kernel<float, __nv_bfloat16, false>, dim3(rows), dim3(vec_threads), 0,
-                                             stream, xs, static_cast<const float*>(nullptr), static_cast<__nv_bfloat16*>(y), w, rows_index, size, eps));
+                                             stream, xs, static_cast<const float*>(nullptr), static_cast<__nv_bfloat16*>(y), w, rows_index, size, size_t{0}, eps));
     return static_cast<int>(cudaErrorInvalidValue);
   }
   const int threads = norm_threads(size);
@@ -266,13 +266,14 @@ MXB_API int mxb_rmsnorm(void* y, int y_dtype, const void* x, int x_dtype, const 
 }
 
 MXB_API int mxb_add_rmsnorm(float* x, const void* delta, int delta_dtype, void* y, int y_dtype,
-                            const float* w, int rows, int size, float eps, cudaStream_t stream) {
+                            const float* w, int rows, int size, int one_delta, float eps, cudaStream_t stream) {
   if (rows <= 0) return 0;
+  const size_t delta_stride = one_delta ? 0 : size;   // one row of deltas for every row of x, or one each
   if (size % 4 == 0 && aligned16(x) && aligned16(y) && aligned16(w) && aligned16(delta) &&
       (delta_dtype == kF32 || size % 8 == 0)) {
     const int vec_threads = norm_threads(size / 4);
 #define VEC(TD, TO) return static_cast<int>(launch_chained(add_rmsnorm_vec4_kernel<TD, TO, true>, dim3(rows), dim3(vec_threads), \
-        0, stream, x, static_cast<const TD*>(delta), static_cast<TO*>(y), w, static_cast<const int*>(nullptr), size, eps))
+        0, stream, x, static_cast<const TD*>(delta), static_cast<TO*>(y), w, static_cast<const int*>(nullptr), size, delta_stride, eps))
     if (delta_dtype == kF32 && y_dtype == kF32) VEC(float, float);
     if (delta_dtype == kBF16 && y_dtype == kBF16) VEC(__nv_bfloat16, __nv_bfloat16);
     if (delta_dtype == kF32 && y_dtype == kBF16) VEC(float, __nv_bfloat16);
@@ -282,7 +283,7 @@ MXB_API int mxb_add_rmsnorm(float* x, const void* delta, int delta_dtype, void* 
   }
   const int threads = norm_threads(size);
 #define LAUNCH(TD, TO) add_rmsnorm_kernel<TD, TO><<<rows, threads, 0, stream>>>( \
-      x, static_cast<const TD*>(delta), static_cast<TO*>(y), w, size, eps)
+      x, static_cast<const TD*>(delta), static_cast<TO*>(y), w, size, delta_stride, eps)
   if (delta_dtype == kF32 && y_dtype == kF32) LAUNCH(float, float);
   else if (delta_dtype == kBF16 && y_dtype == kBF16) LAUNCH(__nv_bfloat16, __nv_bfloat16);
   else if (delta_dtype == kF32 && y_dtype == kBF16) LAUNCH(float, __nv_bfloat16);
@@ -311,16 +312,17 @@ MXB_API int mxb_add_summands_rmsnorm(float* x, const float* summands, int parts,
   return static_cast<int>(e);
 }
 
-MXB_API int mxb_add(float* x, const void* delta, int delta_dtype, long long count,
+MXB_API int mxb_add(float* x, const void* delta, int delta_dtype, long long count, long long period,
                     cudaStream_t stream) {
   if (count <= 0) return 0;
+  if (period <= 0) return static_cast<int>(cudaErrorInvalidValue);
   const int threads = 256;
   const unsigned blocks = static_cast<unsigned>((count + threads - 1) / threads);
   if (delta_dtype == kF32)
     return static_cast<int>(launch_chained(add_kernel<float>, dim3(blocks), dim3(threads), 0, stream, x,
-                                           static_cast<const float*>(delta), static_cast<size_t>(count)));
+                                           static_cast<const float*>(delta), static_cast<size_t>(count), static_cast<size_t>(period)));
   return static_cast<int>(launch_chained(add_kernel<__nv_bfloat16>, dim3(blocks), dim3(threads), 0, stream, x,
-                                         static_cast<const __nv_bfloat16*>(delta), static_cast<size_t>(count)));
+                                         static_cast<const __nv_bfloat16*>(delta), static_cast<size_t>(count), static_cast<size_t>(period)));
 }
 
 // Turns the overlap of consecutive kernels (programmatic dependent launch) on

@@ -65,12 +65,19 @@ gemm_simple_kernel(TOut* __restrict__ c, const TIn* __restrict__ a, const TIn* _
   }
 }
 
+// min(gate, limit) sigmoid(1.702 min(gate, limit)) (clamp(up, -limit, limit) + 1), with the full exponential.
+__device__ __forceinline__ float clamped_product(float gate, float up, float limit) {
+  gate = fminf(gate, limit);
+  up = fminf(fmaxf(up, -limit), limit);
+  return gate / (1.0f + expf(-kClampedSlope * gate)) * (up + 1.0f);
+}
+
 // out[t, i] = act(gate_up[t, i]) * gate_up[t, inter + i], float32 inside (act: silu, or the tanh form of gelu):
 // sigmoid(g) * g * u as the reference writes it
 // (crates/models/qwen/src/forward.rs:1913-1917).
 template <typename T>
 __global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ gate_up, int inter,
-                                size_t count, int activation) {
+                                size_t count, int activation, float limit) {
   const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= count) return;
   const size_t t = i / inter, col = i - t * inter;
@@ -80,13 +87,17 @@ __global__ void silu_mul_kernel(T* __restrict__ out, const T* __restrict__ gate_
     out[i] = from_float<T>(0.5f * g * (1.0f + tanhf(0.7978845608028654f * (g + 0.044715f * g * g * g))) * u);
     return;
   }
+  if (activation == kActClamped) {
+    out[i] = from_float<T>(clamped_product(g, u, limit));
+    return;
+  }
   const float sig = 1.0f / (1.0f + expf(-g));
   out[i] = from_float<T>(sig * g * u);
 }
 
 // Eight bfloat16 values per thread (16-byte loads and stores).
 __global__ void silu_mul_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ gate_up,
-                                       int inter, size_t groups, int activation) {
+                                       int inter, size_t groups, int activation, float limit) {
   const size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x;
   if (i >= groups) return;
   const int per_row = inter / 8;
@@ -103,6 +114,9 @@ __global__ void silu_mul_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __
     if (activation == kActGeluTanh) {
       r0 = 0.5f * g0 * (1.0f + tanhf(0.7978845608028654f * (g0 + 0.044715f * g0 * g0 * g0))) * u0;
       r1 = 0.5f * g1 * (1.0f + tanhf(0.7978845608028654f * (g1 + 0.044715f * g1 * g1 * g1))) * u1;
+    } else if (activation == kActClamped) {
+      r0 = clamped_product(g0, u0, limit);
+      r1 = clamped_product(g1, u1, limit);
     } else {
       r0 = (1.0f / (1.0f + expf(-g0))) * g0 * u0;
       r1 = (1.0f / (1.0f + expf(-g1))) * g1 * u1;
@@ -133,21 +147,21 @@ MXB_API int mxb_gemm_simple(void* c, int c_dtype, const void* a, const void* w, 
 }
 
 MXB_API int mxb_silu_mul(void* out, const void* gate_up, int dtype, long long tokens, int inter, int activation,
-                         cudaStream_t stream) {
+                         float limit, cudaStream_t stream) {
   const size_t count = static_cast<size_t>(tokens) * inter;
   if (count == 0) return 0;
   if (dtype == kBF16 && inter % 8 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0 &&
       reinterpret_cast<uintptr_t>(gate_up) % 16 == 0) {
     const size_t groups = count / 8;
     silu_mul_bf16x8_kernel<<<static_cast<unsigned>((groups + 255) / 256), 256, 0, stream>>>(
-        static_cast<__nv_bfloat16*>(out), static_cast<const __nv_bfloat16*>(gate_up), inter, groups, activation);
+        static_cast<__nv_bfloat16*>(out), static_cast<const __nv_bfloat16*>(gate_up), inter, groups, activation, limit);
     return static_cast<int>(cudaGetLastError());
   }
   const unsigned blocks = static_cast<unsigned>((count + 255) / 256);
   if (dtype == kF32)
-    silu_mul_kernel<float><<<blocks, 256, 0, stream>>>(static_cast<float*>(out), static_cast<const float*>(gate_up), inter, count, activation);
+    silu_mul_kernel<float><<<blocks, 256, 0, stream>>>(static_cast<float*>(out), static_cast<const float*>(gate_up), inter, count, activation, limit);
   else if (dtype == kBF16)
-    silu_mul_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>(static_cast<__nv_bfloat16*>(out), static_cast<const __nv_bfloat16*>(gate_up), inter, count, activation);
+    silu_mul_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>(static_cast<__nv_bfloat16*>(out), static_cast<const __nv_bfloat16*>(gate_up), inter, count, activation, limit);
   else
     return static_cast<int>(cudaErrorInvalidValue);
   return static_cast<int>(cudaGetLastError());

@@ -22,9 +22,9 @@ constexpr int kTcM = 128;     // rows of a tile
 constexpr int kTcK = 64;      // k per stage: 64 bfloat16 = one 128-byte swizzle row
 constexpr int kTcThreads = 192;
 
-enum TcEpilogue : int { kTcStoreBf16 = 0, kTcStoreF32 = 1, kTcSwiGLU = 2, kTcReluSquared = 3, kTcGeGLU = 4 };
-// the epilogues that take a tile of gate rows beside a tile of up rows: act(gate) * up (silu, or the tanh form of gelu)
-__host__ __device__ constexpr bool tc_gated(int epilogue) { return epilogue == kTcSwiGLU || epilogue == kTcGeGLU; }
+enum TcEpilogue : int { kTcStoreBf16 = 0, kTcStoreF32 = 1, kTcSwiGLU = 2, kTcReluSquared = 3, kTcGeGLU = 4, kTcClampedGLU = 5 };
+// the epilogues that take a tile of gate rows beside a tile of up rows: act(gate) * up (silu, or the tanh form of gelu), or the product of clamped halves
+__host__ __device__ constexpr bool tc_gated(int epilogue) { return epilogue == kTcSwiGLU || epilogue == kTcGeGLU || epilogue == kTcClampedGLU; }
 
 template <int BN, int STAGES_> struct TcConfig {
   static constexpr int kStageBytes = (kTcM + BN) * kTcK * 2;
@@ -51,7 +51,7 @@ template <int BN, int EPI, int STAGES_>
 __global__ void __launch_bounds__(kTcThreads)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                     void* __restrict__ out, int m, int n, int k, long long ldo, const int* __restrict__ tile_group,
-                    int group_rows, int* status) {
+                    int group_rows, float limit, int* status) {
   using Config = TcConfig<BN, STAGES_>;
   constexpr int STAGES = Config::kStages;
   constexpr int OUT_COLUMNS = tc_gated(EPI) ? BN / 2 : BN;  // output columns of a tile
@@ -177,7 +177,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             // gate and up take the rounding to bfloat16 they would get on their way through memory
             const float gate = to_float(from_float<__nv_bfloat16>(__uint_as_float(acc[i])));
             const float u = to_float(from_float<__nv_bfloat16>(__uint_as_float(up[i])));
-            values[i] = gate_activation(gate, EPI == kTcGeGLU ? kActGeluTanh : kActSilu) * u;  // rounded to bfloat16 anyway
+            values[i] = gated_product(gate, u, EPI == kTcGeGLU ? kActGeluTanh : (EPI == kTcClampedGLU ? kActClamped : kActSilu), limit);  // rounded to bfloat16 anyway
           }
         } else if (EPI == kTcReluSquared) {
 #pragma unroll
@@ -246,7 +246,8 @@ int g_tc_bn = 0, g_tc_deep = -1;  // tuning overrides: tile width, deep (1) or s
 
 template <int BN, int EPI, int STAGES_>
 static int launch_tc_staged(const CUtensorMap& map_a, const CUtensorMap& map_b, void* out, int m, int n, int k,
-                            long long ldo, const int* tile_group, int group_rows, int* status, cudaStream_t stream) {
+                            long long ldo, const int* tile_group, int group_rows, float limit, int* status,
+                            cudaStream_t stream) {
   using Config = TcConfig<BN, STAGES_>;
   auto kernel = gemm_tcgen05_kernel<BN, EPI, STAGES_>;
   cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, Config::kSharedBytes);
@@ -261,7 +262,7 @@ static int launch_tc_staged(const CUtensorMap& map_a, const CUtensorMap& map_b, 
   }
   dim3 grid(tiles < sm_count ? tiles : sm_count);  // one block per SM walks over the tiles
   kernel<<<grid, kTcThreads, Config::kSharedBytes, stream>>>(map_a, map_b, out, m, n, k, ldo, tile_group, group_rows,
-                                                             status);
+                                                             limit, status);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -270,12 +271,12 @@ static int launch_tc_staged(const CUtensorMap& map_a, const CUtensorMap& map_b, 
 template <int BN, int EPI>
 static int launch_tc(const CUtensorMap& map_a, const CUtensorMap& map_b, void* out, int m, int n, int k,
                      long long ldo, int* status, cudaStream_t stream, const int* tile_group = nullptr,
-                     int group_rows = 0) {
+                     int group_rows = 0, float limit = 0.0f) {
   constexpr int deep = BN >= 256 ? 4 : (BN >= 128 ? 6 : 8);
   const bool shallow = g_tc_deep == 0;
   if (shallow)
-    return launch_tc_staged<BN, EPI, deep / 2>(map_a, map_b, out, m, n, k, ldo, tile_group, group_rows, status, stream);
-  return launch_tc_staged<BN, EPI, deep>(map_a, map_b, out, m, n, k, ldo, tile_group, group_rows, status, stream);
+    return launch_tc_staged<BN, EPI, deep / 2>(map_a, map_b, out, m, n, k, ldo, tile_group, group_rows, limit, status, stream);
+  return launch_tc_staged<BN, EPI, deep>(map_a, map_b, out, m, n, k, ldo, tile_group, group_rows, limit, status, stream);
 }
 
 }  // namespace mxb
@@ -290,9 +291,9 @@ MXB_API int mxb_gemm_tcgen05_supported(int m, int n, int k, long long lda, long 
 
 // epilogue: 0 bfloat16 out[m, n], 1 float32 out[m, n], 2 SwiGLU: w is
 // [2 * n, k] (gate rows, then up rows) and out is bfloat16 [m, n]; 4 the same
-// with the tanh form of gelu in place of silu.
+// with the tanh form of gelu in place of silu; 5 min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, -limit, limit) + 1).
 MXB_API int mxb_gemm_tcgen05(void* out, const void* a, const void* w, int m, int n, int k, long long lda,
-                             long long ldw, long long ldo, int epilogue, int* status, cudaStream_t stream) {
+                             long long ldw, long long ldo, int epilogue, float limit, int* status, cudaStream_t stream) {
   if (!mxb_gemm_tcgen05_supported(m, n, k, lda, ldw)) return static_cast<int>(cudaErrorInvalidValue);
   if ((reinterpret_cast<uintptr_t>(a) & 15) || (reinterpret_cast<uintptr_t>(w) & 15)) return static_cast<int>(cudaErrorInvalidValue);
   const int w_rows = tc_gated(epilogue) ? 2 * n : n;
@@ -323,6 +324,11 @@ MXB_API int mxb_gemm_tcgen05(void* out, const void* a, const void* w, int m, int
     if (bn == 256) return launch_tc<256, kTcGeGLU>(map_a, map_b, out, m, n, k, ldo, status, stream);
     if (bn == 128) return launch_tc<128, kTcGeGLU>(map_a, map_b, out, m, n, k, ldo, status, stream);
     return launch_tc<64, kTcGeGLU>(map_a, map_b, out, m, n, k, ldo, status, stream);
+  }
+  if (epilogue == kTcClampedGLU) {
+    if (bn == 256) return launch_tc<256, kTcClampedGLU>(map_a, map_b, out, m, n, k, ldo, status, stream, nullptr, 0, limit);
+    if (bn == 128) return launch_tc<128, kTcClampedGLU>(map_a, map_b, out, m, n, k, ldo, status, stream, nullptr, 0, limit);
+    return launch_tc<64, kTcClampedGLU>(map_a, map_b, out, m, n, k, ldo, status, stream, nullptr, 0, limit);
   }
   if (epilogue == kTcStoreF32) {
     if (bn == 256) return launch_tc<256, kTcStoreF32>(map_a, map_b, out, m, n, k, ldo, status, stream);

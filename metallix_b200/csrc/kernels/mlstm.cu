@@ -414,11 +414,11 @@ mlstm_chunk_kernel(const T* __restrict__ proj, long long ld, int q_off, int k_of
   if (threadIdx.x == 0) m_state[0] = s_m0[0];
 }
 
-// y[t, h, :] = x[t, h, :] * rsqrt(mean_v(x^2) + eps) * w[h, :] * sigmoid(g[t, h, :]); one warp per (t, h).
+// y[t, h, :] = x[t, h, :] * rsqrt(mean_v(x^2) + eps) * w[h, :] * sigmoid(g[t, h, :]) (silu: g sigmoid(g)); one warp per (t, h).
 template <typename TGate, typename TOut>
 __global__ void __launch_bounds__(128)
 head_norm_gate_kernel(const float* __restrict__ x, const float* __restrict__ w, const TGate* __restrict__ gate,
-                      long long ldg, TOut* __restrict__ y, int pairs, int heads, int vdim, float eps) {
+                      long long ldg, TOut* __restrict__ y, int pairs, int heads, int vdim, int silu, float eps) {
   chain_release();
   const int pair = blockIdx.x * 4 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (pair >= pairs) return;
@@ -432,7 +432,10 @@ head_norm_gate_kernel(const float* __restrict__ x, const float* __restrict__ w, 
   TOut* dst = y + static_cast<long long>(pair) * vdim;
   for (int j = lane; j < vdim; j += 32) {
     float v = row[j] * scale * w[h * vdim + j];
-    if (g != nullptr) v *= sigmoid_of(to_float(g[j]));
+    if (g != nullptr) {
+      const float z = to_float(g[j]);
+      v *= silu ? z * sigmoid_of(z) : sigmoid_of(z);
+    }
     dst[j] = from_float<TOut>(v);
   }
 }
@@ -519,13 +522,13 @@ MXB_API int mxb_mlstm_scan(const void* proj, long long ld, int q_off, int k_off,
 }
 
 MXB_API int mxb_head_norm_gate(const float* x, const float* w, const void* gate, long long ldg, int gate_dtype, void* y,
-                               int out_dtype, int tokens, int heads, int vdim, float eps, cudaStream_t stream) {
+                               int out_dtype, int tokens, int heads, int vdim, int silu, float eps, cudaStream_t stream) {
   const int pairs = tokens * heads;
   if (pairs <= 0) return 0;
   const dim3 grid((pairs + 3) / 4);
 #define LAUNCH(TG, TO)                                                                                         \
   head_norm_gate_kernel<TG, TO><<<grid, 128, 0, stream>>>(x, w, static_cast<const TG*>(gate), ldg,              \
-                                                          static_cast<TO*>(y), pairs, heads, vdim, eps)
+                                                          static_cast<TO*>(y), pairs, heads, vdim, silu, eps)
   if (gate_dtype == kF32 && out_dtype == kF32) LAUNCH(float, float);
   else if (gate_dtype == kF32 && out_dtype == kBF16) LAUNCH(float, __nv_bfloat16);
   else if (gate_dtype == kBF16 && out_dtype == kF32) LAUNCH(__nv_bfloat16, float);

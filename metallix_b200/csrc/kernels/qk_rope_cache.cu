@@ -12,6 +12,9 @@
 // together, weights of that width) instead of head by head; the second has a
 // kernel of its own below, one block per token.
 //
+// Queries may further be multiplied by a factor of their position, read from a
+// table (`q_factors`, float32, one per position).
+//
 // Cache layout of one layer: [pages, 2 (K, V), kv_heads, page_tokens, head_dim];
 // position p of a request lives in page table[p / page_tokens] at row
 // p % page_tokens, which the caller passes flattened as slot = page *
@@ -19,6 +22,17 @@
 #include "common.cuh"
 
 namespace mxb {
+
+// What a query at position `pos` is multiplied by: 1 without a table.
+__device__ __forceinline__ float query_factor(const float* __restrict__ q_factors, int factor_positions, int pos,
+                                              bool reports, int* status) {
+  if (q_factors == nullptr) return 1.0f;
+  if (pos < 0 || pos >= factor_positions) {
+    if (reports) atomicOr(status, kStatusBadSlot);
+    pos = 0;
+  }
+  return q_factors[pos];
+}
 
 template <typename T>
 __global__ void qk_norm_rope_cache_kernel(
@@ -30,7 +44,7 @@ __global__ void qk_norm_rope_cache_kernel(
     const float* __restrict__ q_weight, const float* __restrict__ k_weight,  // null: no norm
     const float* __restrict__ cos_table, const float* __restrict__ sin_table,  // null: no rotation
     int table_positions, int rotary_dim, int interleaved, int heads, int kv_heads, int head_dim, int page_tokens,
-    int num_pages, float eps, int* status) {
+    int num_pages, float eps, const float* __restrict__ q_factors, int factor_positions, int* status) {
   extern __shared__ float head[];  // head_dim values
   __shared__ float scratch[33];
   const int t = blockIdx.x;
@@ -85,6 +99,7 @@ __global__ void qk_norm_rope_cache_kernel(
     if (threadIdx.x == 0) atomicOr(status, kStatusBadSlot);
     pos = 0;
   }
+  const float factor = is_q ? query_factor(q_factors, factor_positions, positions[t], threadIdx.x == 0, status) : 1.0f;
   for (int i = threadIdx.x; i < head_dim; i += blockDim.x) {
     float out = head[i];
     if (rotate && i < rotary_dim) {
@@ -97,7 +112,7 @@ __global__ void qk_norm_rope_cache_kernel(
       const float s = sin_table[static_cast<size_t>(pos) * half + j];
       out = first ? head[i] * c - head[partner] * s : head[i] * c + head[partner] * s;
     }
-    dst[i] = from_float<T>(out);
+    dst[i] = from_float<T>(out * factor);
   }
 }
 
@@ -119,7 +134,8 @@ qk_norm_rope_cache_warp_kernel(
     T* __restrict__ cache, const int* __restrict__ slots, const int* __restrict__ positions,
     const float* __restrict__ q_weight, const float* __restrict__ k_weight,
     const float* __restrict__ cos_table, const float* __restrict__ sin_table, int table_positions,
-    int tokens, int heads, int kv_heads, int page_tokens, int num_pages, float eps, int* status) {
+    int tokens, int heads, int kv_heads, int page_tokens, int num_pages, float eps,
+    const float* __restrict__ q_factors, int factor_positions, int* status) {
   constexpr int V = 16 / static_cast<int>(sizeof(T));
   constexpr int HALF = HD / 2;
   constexpr int LANES = HALF / V;          // lanes of a head
@@ -200,6 +216,7 @@ qk_norm_rope_cache_warp_kernel(
       }
     }
   }
+  const float factor = active && is_q ? query_factor(q_factors, factor_positions, positions[t], sub == 0, status) : 1.0f;
   chain_wait();
   src = behind_wait(src);  // written by the kernel ahead of this one
   Values in_lo = {}, in_hi = {};
@@ -245,8 +262,8 @@ qk_norm_rope_cache_warp_kernel(
   Values out_lo, out_hi;
 #pragma unroll
   for (int j = 0; j < V; ++j) {
-    out_lo.v[j] = from_float<T>(x[j]);
-    out_hi.v[j] = from_float<T>(x[V + j]);
+    out_lo.v[j] = from_float<T>(x[j] * factor);
+    out_hi.v[j] = from_float<T>(x[V + j] * factor);
   }
   reinterpret_cast<Values*>(dst)[sub] = out_lo;
   reinterpret_cast<Values*>(dst + HALF)[sub] = out_hi;
@@ -272,7 +289,7 @@ qk_rownorm_rope_cache_kernel(
     const float* __restrict__ q_weight, const float* __restrict__ k_weight,
     const float* __restrict__ cos_table, const float* __restrict__ sin_table, int table_positions,
     int rotary_dim, int interleaved, int heads, int kv_heads, int head_dim, int page_tokens, int num_pages,
-    float eps, int* status) {
+    float eps, const float* __restrict__ q_factors, int factor_positions, int* status) {
   __shared__ float scratch[66];
   using Values = Pack<T, V>;
   chain_release();
@@ -355,6 +372,7 @@ qk_rownorm_rope_cache_kernel(
     k_sum = scratch[65];
   }
   const int half = rotary_dim >> 1;
+  const float factor = query_factor(q_factors, factor_positions, positions[t], threadIdx.x == 0, status);
 
   auto finish = [&](const T* row, int width, float sum, const float* weight, bool is_q) {
     const float scale = weight != nullptr ? rsqrtf(sum / static_cast<float>(width) + eps) : 1.0f;
@@ -407,7 +425,7 @@ qk_rownorm_rope_cache_kernel(
       }
       Values out;
 #pragma unroll
-      for (int j = 0; j < V; ++j) out.v[j] = from_float<T>(x[j]);
+      for (int j = 0; j < V; ++j) out.v[j] = from_float<T>(is_q ? x[j] * factor : x[j]);
       if (is_q) *reinterpret_cast<Values*>(q_out + static_cast<size_t>(t) * width + i) = out;
       else *reinterpret_cast<Values*>(key_page + h * head_stride + d0) = out;
     };
@@ -426,7 +444,8 @@ MXB_API int mxb_qk_norm_rope_cache(
     long long v_stride, void* q_out, void* cache, const int* slots, const int* positions,
     const float* q_weight, const float* k_weight, const float* cos_table, const float* sin_table,
     int table_positions, int rotary_dim, int interleaved, int norm_scope, int tokens, int heads, int kv_heads,
-    int head_dim, int page_tokens, int num_pages, float eps, int dtype, int* status, cudaStream_t stream) {
+    int head_dim, int page_tokens, int num_pages, float eps, int dtype, const float* q_factors, int factor_positions,
+    int* status, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (rotary_dim < 0 || rotary_dim > head_dim || (rotary_dim & 1)) return static_cast<int>(cudaErrorInvalidValue);
   if (dtype != kF32 && dtype != kBF16) return static_cast<int>(cudaErrorInvalidValue);
@@ -452,7 +471,7 @@ MXB_API int mxb_qk_norm_rope_cache(
       if (launch_status == cudaSuccess) launch_status = launch_chained(kernel, dim3(tokens), dim3(256), shared, stream, \
         static_cast<const T*>(q_in), static_cast<const T*>(k_in), static_cast<const T*>(v_in), q_stride, k_stride, v_stride, \
         static_cast<T*>(q_out), static_cast<T*>(cache), slots, positions, q_weight, k_weight, cos_table, sin_table, \
-        table_positions, rotary_dim, interleaved, heads, kv_heads, head_dim, page_tokens, num_pages, eps, status); } while (0)
+        table_positions, rotary_dim, interleaved, heads, kv_heads, head_dim, page_tokens, num_pages, eps, q_factors, factor_positions, status); } while (0)
     if (dtype == kF32) { if (wide) ROW_LAUNCH(float, 4); else ROW_LAUNCH(float, 1); }
     else { if (wide) ROW_LAUNCH(__nv_bfloat16, 8); else ROW_LAUNCH(__nv_bfloat16, 1); }
 #undef ROW_LAUNCH
@@ -471,7 +490,7 @@ MXB_API int mxb_qk_norm_rope_cache(
 #define WARP_LAUNCH(T, HD) launch_status = launch_chained(qk_norm_rope_cache_warp_kernel<T, HD>, dim3(blocks), dim3(256), 0, stream, \
         static_cast<const T*>(q_in), static_cast<const T*>(k_in), static_cast<const T*>(v_in), q_stride, k_stride, \
         v_stride, static_cast<T*>(q_out), static_cast<T*>(cache), slots, positions, q_weight, k_weight, cos_table, \
-        sin_table, table_positions, tokens, heads, kv_heads, page_tokens, num_pages, eps, status)
+        sin_table, table_positions, tokens, heads, kv_heads, page_tokens, num_pages, eps, q_factors, factor_positions, status)
     if (dtype == kF32) {
       if (head_dim == 64) WARP_LAUNCH(float, 64); else if (head_dim == 128) WARP_LAUNCH(float, 128); else WARP_LAUNCH(float, 256);
     } else {
@@ -489,14 +508,14 @@ MXB_API int mxb_qk_norm_rope_cache(
         static_cast<const float*>(q_in), static_cast<const float*>(k_in), static_cast<const float*>(v_in),
         q_stride, k_stride, v_stride, static_cast<float*>(q_out), static_cast<float*>(cache), slots,
         positions, q_weight, k_weight, cos_table, sin_table, table_positions, rotary_dim, interleaved, heads,
-        kv_heads, head_dim, page_tokens, num_pages, eps, status);
+        kv_heads, head_dim, page_tokens, num_pages, eps, q_factors, factor_positions, status);
   else if (dtype == kBF16)
     qk_norm_rope_cache_kernel<__nv_bfloat16><<<grid, threads, shared, stream>>>(
         static_cast<const __nv_bfloat16*>(q_in), static_cast<const __nv_bfloat16*>(k_in),
         static_cast<const __nv_bfloat16*>(v_in), q_stride, k_stride, v_stride,
         static_cast<__nv_bfloat16*>(q_out), static_cast<__nv_bfloat16*>(cache), slots, positions,
         q_weight, k_weight, cos_table, sin_table, table_positions, rotary_dim, interleaved, heads, kv_heads,
-        head_dim, page_tokens, num_pages, eps, status);
+        head_dim, page_tokens, num_pages, eps, q_factors, factor_positions, status);
   else
     return static_cast<int>(cudaErrorInvalidValue);
   return static_cast<int>(cudaGetLastError());

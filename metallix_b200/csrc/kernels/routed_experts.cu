@@ -4,7 +4,8 @@
 // outputs (or, as a switch, s = sigmoid(z) for each output on its own; the
 // outputs may also form equal groups of neighbours of which only the best few,
 // by the sum of a group's two largest s + correction, can be chosen from; and
-// the weights may be multiplied by a constant); the `top` outputs with the largest s + correction are chosen (ties
+// the weights may be multiplied by a constant; or, as a third form, s = z + correction itself decides and
+// weighs: the largest are chosen and their weights are the softmax over the chosen alone); the `top` outputs with the largest s + correction are chosen (ties
 // go to the lower index); their weights are their s, divided by the sum of
 // the chosen s (+ 1e-20). The sum s + correction is formed and compared in
 // double precision: where the correction is the same for several outputs and
@@ -35,12 +36,13 @@
 
 namespace mxb {
 
+enum RouteScores : int { kScoreSoftmax = 0, kScoreSigmoid = 1, kScoreChosen = 2 };
 constexpr int kRouteThreads = 128;   // four tokens a block, a warp each
 
 __global__ void __launch_bounds__(kRouteThreads)
 route_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int* __restrict__ chosen,
              float* __restrict__ weights, float* __restrict__ dense, float* __restrict__ identity_weight,
-             int tokens, int outputs, int experts, int top, int sigmoid_scores, int group_count, int group_keep,
+             int tokens, int outputs, int experts, int top, int scores, int group_count, int group_keep,
              float weight_scale, long long ld) {
   extern __shared__ double shared[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
@@ -50,7 +52,16 @@ route_kernel(const float* __restrict__ logits, const float* __restrict__ correct
   float* score = reinterpret_cast<float*>(reinterpret_cast<double*>(shared) + static_cast<size_t>(kRouteThreads / 32) * outputs) +
                  static_cast<size_t>(warp) * outputs;                                        // s
   const float* z = logits + static_cast<long long>(t) * ld;   // rows may be further apart than they are long
-  if (sigmoid_scores) {   // every output's score on its own: s = 1 / (1 + e^-z)
+  if (scores == kScoreChosen) {   // z + bias decides; e^(z - peak) over the chosen ones' sum weighs (the peak is always chosen)
+    float peak = -INFINITY;
+    for (int r = lane; r < outputs; r += 32) peak = fmaxf(peak, z[r] + correction[r]);
+    peak = warp_max(peak);
+    for (int r = lane; r < outputs; r += 32) {
+      const float v = z[r] + correction[r];
+      score[r] = expf(v - peak);
+      choice[r] = v;
+    }
+  } else if (scores == kScoreSigmoid) {   // every output's score on its own: s = 1 / (1 + e^-z)
     for (int r = lane; r < outputs; r += 32) {
       const float s = 1.0f / (1.0f + expf(-z[r]));
       score[r] = s;
@@ -342,13 +353,14 @@ using namespace mxb;
 
 // logits: float32 [tokens, outputs]; correction: float32 [outputs]; chosen: int32 [tokens, top];
 // weights: float32 [tokens, top]; dense: float32 [tokens, experts]; identity_weight: float32 [tokens].
-// sigmoid_scores: s = sigmoid(z) instead of softmax(z). group_count > 1: the outputs form that many equal groups of
+// scores: 0 s = softmax(z), 1 s = sigmoid(z), 2 z + correction chooses and the softmax over the chosen weighs. group_count > 1: the outputs form that many equal groups of
 // neighbours, and only outputs of the group_keep best groups can be chosen. weight_scale multiplies the weights.
 MXB_API int mxb_route_experts(const float* logits, const float* correction, int* chosen, float* weights, float* dense,
                               float* identity_weight, int tokens, int outputs, int experts, int top,
-                              int sigmoid_scores, int group_count, int group_keep, float weight_scale,
+                              int scores, int group_count, int group_keep, float weight_scale,
                               long long ld, cudaStream_t stream) {
   if (tokens <= 0) return 0;
+  if (scores < kScoreSoftmax || scores > kScoreChosen) return static_cast<int>(cudaErrorInvalidValue);
   if (outputs <= 0 || experts < 0 || experts > outputs || top <= 0 || top > outputs)
     return static_cast<int>(cudaErrorInvalidValue);
   if (group_count > 1 && (outputs % group_count != 0 || group_keep < 1 || group_keep > group_count ||
@@ -358,7 +370,7 @@ MXB_API int mxb_route_experts(const float* logits, const float* correction, int*
   const size_t shared = (sizeof(float) + (group_count > 1 ? 2 : 1) * sizeof(double)) * outputs * (kRouteThreads / 32);
   if (shared > 48 * 1024) return static_cast<int>(cudaErrorInvalidValue);
   route_kernel<<<ceil_div(tokens, kRouteThreads / 32), kRouteThreads, shared, stream>>>(
-      logits, correction, chosen, weights, dense, identity_weight, tokens, outputs, experts, top, sigmoid_scores,
+      logits, correction, chosen, weights, dense, identity_weight, tokens, outputs, experts, top, scores,
       group_count, group_keep, weight_scale, ld < outputs ? outputs : ld);
   return static_cast<int>(cudaGetLastError());
 }

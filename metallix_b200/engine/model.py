@@ -1,5 +1,5 @@
 """A decoder put together from a ``ModelSpec``: embedding, blocks in the
-spec's order, final norm on the wanted rows only, output head
+spec's order (with what joins the residual stream ahead of a run), final norm on the wanted rows only, output head
 (crates/models/qwen/src/forward.rs:1562-1606)."""
 from __future__ import annotations
 
@@ -22,6 +22,7 @@ class DecoderModel:
         self.spec, self.runtime = spec, runtime
         weights = WeightStore(tensors)
         self.embedding = build_part("embedding", spec.embedding, weights, runtime)
+        self.joins = [build_part("join", join, weights, runtime) for join in spec.joins]
         self.blocks = []
         for layer in spec.layers:
             builder = _BUILDERS.get(("block", layer.block.kind))
@@ -55,9 +56,11 @@ class DecoderModel:
         return needs
 
     def weight_bytes(self) -> int:
-        """Bytes of every weight one step reads once."""
+        """Bytes of every weight one step reads (a layer that runs several times counts each time)."""
         total = self.head.weight_bytes() if not self.head.tied else self.embedding.weight_bytes()
-        for block in self.blocks:
+        for run in self.order:
+            block = self.blocks[run.layer]
+            total += self.joins[run.join].weight_bytes() if run.join is not None else 0
             for part in (block.mixer, getattr(block, "feed_forward", None)):
                 total += part.weight_bytes() if hasattr(part, "weight_bytes") else 0
         return total
@@ -74,9 +77,15 @@ class DecoderModel:
         streams = self.spec.streams
         if streams:   # several copies of the stream: [tokens, streams, hidden]
             residual = open_streams(residual, streams)
+        # the stream as the embedding left it, for joins that read it again: a copy where a layer changes it first
+        first = None
+        if self.joins:
+            first = residual if self.order[0].join is not None else residual.clone()
         pending = None
         for index, run in enumerate(self.order):
             block = self.blocks[run.layer]
+            if run.join is not None:
+                residual, pending = self.joins[run.join].forward(residual, pending, first, run.turn)
             pending = block.forward(residual, pending, ctx, views(run.cache_entry(), run.write_cache))
             if tap is not None:
                 settle(residual, pending)

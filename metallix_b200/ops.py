@@ -29,14 +29,14 @@ _P, _I, _L, _F = ctypes.c_void_p, ctypes.c_int, ctypes.c_longlong, ctypes.c_floa
 _SIGNATURES = {
     "mxb_embed": [_P, _P, _I, _P, _I, _I, _I, _F, _P, _P],
     "mxb_rmsnorm": [_P, _I, _P, _I, _P, _P, _I, _I, _F, _P],
-    "mxb_add_rmsnorm": [_P, _P, _I, _P, _I, _P, _I, _I, _F, _P],
+    "mxb_add_rmsnorm": [_P, _P, _I, _P, _I, _P, _I, _I, _I, _F, _P],
     "mxb_add_summands_rmsnorm": [_P, _P, _I, _P, _I, _P, _I, _I, _F, _P],
-    "mxb_add": [_P, _P, _I, _L, _P],
+    "mxb_add": [_P, _P, _I, _L, _L, _P],
     "mxb_copy_units": [_P, _I, _I, _L, _P, _I, _P, _P],
     "mxb_qk_norm_rope_cache": [_P, _P, _P, _L, _L, _L, _P, _P, _P, _P, _P, _P, _P, _P,
-                               _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _P],
+                               _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P],
     "mxb_paged_attention_tile": [_P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I,
-                                 _F, _I, _P, _L, _I, _I, _F, _I, _I, _F, _P, _P, _P],
+                                 _F, _I, _P, _L, _I, _I, _F, _I, _I, _F, _P, _P, _I, _P, _P],
     "mxb_short_conv": [_P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "mxb_selective_scan": [_P, _L, _P, _L, _P, _P, _P, _P, _L, _P, _P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I,
                            _I, _P, _P],
@@ -50,9 +50,14 @@ _SIGNATURES = {
     "mxb_experts_routed": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
     "mxb_add_gated_rows": [_P, _P, _P, _L, _I, _I, _I, _P],
     "mxb_pair_add_rmsnorm": [_P, _P, _I, _P, _I, _F, _P, _P, _P, _P, _I, _P, _I, _I, _F, _P],
+    "mxb_pair_norm_max_size": [],
+    "mxb_pair_norm": [_P, _P, _I, _I, _P, _I, _P, _P, _P, _P, _F, _F, _F, _F, _P, _I, _P, _I, _I, _F, _P],
+    "mxb_gated_norm_max_part": [],
+    "mxb_gated_norm": [_P, _P, _L, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P],
+    "mxb_join_rows": [_P, _P, _I, _P, _P, _I, _I, _I, _P],
     "mxb_add_bias": [_P, _L, _I, _P, _P, _L, _I, _I, _I, _P],
     "mxb_delta_rule_max_dim": [],
-    "mxb_delta_rule": [_P, _L, _I, _I, _I, _P, _L, _I, _P, _L, _P, _P, _P, _L, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I,
+    "mxb_delta_rule": [_P, _L, _I, _I, _I, _P, _L, _I, _P, _L, _P, _P, _P, _I, _P, _L, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I,
                        _I, _I, _P, _P],
     "mxb_add_cast": [_P, _P, _I, _P, _I, _L, _P],
     "mxb_gelu_gate_rows": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
@@ -61,40 +66,40 @@ _SIGNATURES = {
     "mxb_mlstm_state_values": [_I, _I, _I],
     "mxb_mlstm_scan": [_P, _L, _I, _I, _I, _I, _I, _P, _P, _F, _F, _P, _L, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I,
                        _I, _P, _P],
-    "mxb_head_norm_gate": [_P, _P, _P, _L, _I, _P, _I, _I, _I, _I, _F, _P],
+    "mxb_head_norm_gate": [_P, _P, _P, _L, _I, _P, _I, _I, _I, _I, _I, _F, _P],
     "mxb_latent_cache": [_P, _L, _P, _F, _I, _I, _I, _I, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _P, _P],
     "mxb_latent_heads": [_P, _L, _P, _L, _P, _L, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I,
                          _I, _P, _P],
     "mxb_rotate_into": [_P, _L, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _I, _P, _I, _I, _P, _P],
     "mxb_relu_squared": [_P, _P, _L, _I, _P],
     "mxb_paged_attention_decode": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I,
-                                   _F, _I, _P, _L, _F, _I, _F, _P, _P, _P],
+                                   _F, _I, _P, _L, _F, _I, _F, _P, _P, _I, _P, _P],
     "mxb_postnorm_add_rmsnorm": [_P, _P, _I, _I, _P, _F, _P, _I, _P, _F, _I, _I, _P],
     "mxb_sigmoid_gate": [_P, _P, _P, _L, _L, _L, _I, _I, _I, _P],
     "mxb_softcap": [_P, _F, _L, _P],
     "mxb_paged_attention_decode_supported": [_I, _I, _I, _I],
     "mxb_paged_attention_decode_project_supported": [_I, _I, _I, _I, _I, _P, _L],
     "mxb_paged_attention_decode_project": [_P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I,
-                                           _F, _P, _L, _I, _P, _P, _L, _F, _I, _F, _P, _P, _P],
+                                           _F, _P, _L, _I, _P, _P, _L, _F, _I, _F, _P, _P, _I, _P, _P],
     "mxb_paged_attention_split_keys": [],
     "mxb_set_decode_resident_blocks": [_I, _I],
     "mxb_flash_prefill": [_P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _L, _F, _I, _F,
-                          _P, _P, _P],
+                          _P, _P, _I, _P, _P],
     "mxb_flash_prefill_supported": [_I, _I, _I, _I],
     "mxb_flash_prefill_tile": [],
     "mxb_flash_prefill_tcgen05": [_P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P,
-                                  _P, _L, _F, _I, _F, _P, _P, _P],
+                                  _P, _L, _F, _I, _F, _P, _P, _I, _P, _P],
     "mxb_flash_prefill_tcgen05_supported": [_I, _I, _I, _I, _I],
     "mxb_flash_prefill_tcgen05_tile": [],
     "mxb_gemm_simple": [_P, _I, _P, _P, _I, _I, _I, _I, _L, _L, _L, _P],
-    "mxb_gemm_skinny": [_P, _I, _P, _P, _I, _I, _I, _L, _L, _L, _I, _I, _P],
+    "mxb_gemm_skinny": [_P, _I, _P, _P, _I, _I, _I, _L, _L, _L, _I, _I, _F, _P],
     "mxb_gemm_skinny_supported": [_I, _I, _I, _L, _L],
-    "mxb_gemm_stream": [_P, _I, _P, _P, _I, _I, _I, _L, _L, _L, _I, _I, _P, _P],
+    "mxb_gemm_stream": [_P, _I, _P, _P, _I, _I, _I, _L, _L, _L, _I, _I, _F, _P, _P],
     "mxb_gemm_stream_supported": [_I, _I, _I, _L, _L, _I],
-    "mxb_gemm_tcgen05": [_P, _P, _P, _I, _I, _I, _L, _L, _L, _I, _P, _P],
+    "mxb_gemm_tcgen05": [_P, _P, _P, _I, _I, _I, _L, _L, _L, _I, _F, _P, _P],
     "mxb_gemm_tcgen05_supported": [_I, _I, _I, _L, _L],
     "mxb_gemm_tcgen05_grouped": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _L, _L, _L, _I, _P, _P],
-    "mxb_silu_mul": [_P, _P, _I, _L, _I, _I, _P],
+    "mxb_silu_mul": [_P, _P, _I, _L, _I, _I, _F, _P],
     "mxb_argmax": [_P, _L, _I, _I, _P, _P, _P, _P],
     "mxb_argmax_pieces": [_I, _I],
     "mxb_sample_icdf": [_P, _L, _I, _I, _P, _P, _P, _P, _P, _P, _P, _P, _P],
@@ -310,7 +315,8 @@ def add_rmsnorm(x: torch.Tensor, delta: torch.Tensor, weight: torch.Tensor, eps:
                 out_dtype: torch.dtype, out: Optional[torch.Tensor] = None) -> torch.Tensor:
     """x += delta in float32 (in place), then returns RMSNorm(x) * w. A delta
     of three dimensions, float32 ``[parts, rows, size]``, is a sum its producer
-    left in parts: they are added up in their order first."""
+    left in parts: they are added up in their order first. A delta of one
+    dimension, ``[size]``, joins every row."""
     _check(x, "x", (torch.float32,), 2)
     _check(weight, "weight", (torch.float32,), 1)
     rows, size = x.shape
@@ -325,19 +331,20 @@ def add_rmsnorm(x: torch.Tensor, delta: torch.Tensor, weight: torch.Tensor, eps:
         _call("mxb_add_summands_rmsnorm", x.data_ptr(), delta.data_ptr(), delta.shape[0], out.data_ptr(),
               _CODES[out_dtype], weight.data_ptr(), rows, size, float(eps), _stream())
         return out
-    _check(delta, "delta", tuple(_CODES), 2)
-    _need(delta.shape == x.shape, "delta and x differ in shape")
+    one = delta.dim() == 1
+    _check(delta, "delta", tuple(_CODES), 1 if one else 2)
+    _need(delta.shape == (x.shape[1:] if one else x.shape), "delta and x differ in shape")
     _call("mxb_add_rmsnorm", x.data_ptr(), delta.data_ptr(), _CODES[delta.dtype], out.data_ptr(),
-          _CODES[out_dtype], weight.data_ptr(), rows, size, float(eps), _stream())
+          _CODES[out_dtype], weight.data_ptr(), rows, size, 1 if one else 0, float(eps), _stream())
     return out
 
 
 def add_(x: torch.Tensor, delta: torch.Tensor) -> torch.Tensor:
-    """x += delta, the sum in float32."""
+    """x += delta, the sum in float32. A delta of one dimension joins every row of x."""
     _check(x, "x", (torch.float32,))
     _check(delta, "delta", tuple(_CODES))
-    _need(delta.shape == x.shape, "delta and x differ in shape")
-    _call("mxb_add", x.data_ptr(), delta.data_ptr(), _CODES[delta.dtype], x.numel(), _stream())
+    _need(delta.shape == x.shape or (delta.dim() == 1 and delta.numel() == x.shape[-1]), "delta and x differ in shape")
+    _call("mxb_add", x.data_ptr(), delta.data_ptr(), _CODES[delta.dtype], x.numel(), delta.numel(), _stream())
     return x
 
 
@@ -379,6 +386,58 @@ def pair_add_rmsnorm(x: torch.Tensor, a: Optional[torch.Tensor], b: Optional[tor
     if weight is None:
         return None
     return (first, second) if second_weight is not None else first
+
+
+def pair_norm(x: torch.Tensor, left: torch.Tensor, right: torch.Tensor, left_weight: torch.Tensor,
+              right_weight: torch.Tensor, left_eps: float, right_eps: float, a: float, b: float,
+              left_bias: Optional[torch.Tensor] = None, right_bias: Optional[torch.Tensor] = None,
+              weight: Optional[torch.Tensor] = None, eps: float = 0.0,
+              out_dtype: torch.dtype = torch.float32) -> Optional[torch.Tensor]:
+    """x += a * RMSNorm(left + left_bias) * left_weight + b * RMSNorm(right +
+    right_bias) * right_weight in float32 (in place), then, with ``weight``,
+    returns RMSNorm(x) * weight in ``out_dtype``; the biases are optional.
+    ``left`` and ``right`` are ``[rows, size]`` of either type; ``left`` may be
+    float32 ``[parts, rows, size]``, whose parts are added up first."""
+    _check(x, "x", (torch.float32,), 2)
+    rows, size = x.shape
+    parts = 1
+    if left.dim() == 3:
+        _check(left, "left", (torch.float32,), 3)
+        parts = left.shape[0]
+        _need(left.shape[1:] == x.shape and parts >= 1, "left's summands and x differ in shape")
+    else:
+        _check(left, "left", tuple(_CODES), 2)
+        _need(left.shape == x.shape, "left and x differ in shape")
+    _check(right, "right", tuple(_CODES), 2)
+    _need(right.shape == x.shape, "right and x differ in shape")
+    for name, tensor, needed in (("left_weight", left_weight, True), ("right_weight", right_weight, True),
+                                 ("left_bias", left_bias, False), ("right_bias", right_bias, False), ("weight", weight, False)):
+        if tensor is not None or needed:
+            _check(tensor, name, (torch.float32,), 1)
+            _need(tensor.numel() == size, f"{name} has the wrong size")
+    _need(out_dtype in _CODES, "out_dtype must be float32 or bfloat16")
+    out = torch.empty((rows, size), dtype=out_dtype, device=x.device) if weight is not None else None
+    _call("mxb_pair_norm", x.data_ptr(), left.data_ptr(), _CODES[left.dtype], parts, right.data_ptr(), _CODES[right.dtype],
+          _ptr(left_bias), _ptr(right_bias), left_weight.data_ptr(), right_weight.data_ptr(), float(left_eps),
+          float(right_eps), float(a), float(b), _ptr(out), _CODES[out_dtype], _ptr(weight), rows, size, float(eps), _stream())
+    return out
+
+
+def join_rows(x: torch.Tensor, delta: Optional[torch.Tensor], first: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
+    """``[rows, 2 * size]`` = [x + delta | first] in ``out_dtype`` (the sum in
+    float32; x is left as it is; ``delta`` is optional)."""
+    _check(x, "x", (torch.float32,), 2)
+    _check(first, "first", (torch.float32,), 2)
+    _need(first.shape == x.shape, "x and first differ in shape")
+    if delta is not None:
+        _check(delta, "delta", tuple(_CODES), 2)
+        _need(delta.shape == x.shape, "delta and x differ in shape")
+    _need(out_dtype in _CODES, "out_dtype must be float32 or bfloat16")
+    rows, size = x.shape
+    out = torch.empty((rows, 2 * size), dtype=out_dtype, device=x.device)
+    _call("mxb_join_rows", x.data_ptr(), _ptr(delta), _CODES[delta.dtype] if delta is not None else F32, first.data_ptr(),
+          out.data_ptr(), _CODES[out_dtype], rows, size, _stream())
+    return out
 
 
 def add_bias(x: torch.Tensor, bias: torch.Tensor, out_dtype: torch.dtype) -> torch.Tensor:
@@ -616,6 +675,7 @@ def selective_scan(x: torch.Tensor, step: torch.Tensor, step_bias: torch.Tensor,
 
 
 # ------------------------------------------------------------ routed experts
+ROUTE_SCORES = {"softmax": 0, "sigmoid": 1, "chosen": 2}
 ROUTER_OUTPUTS = 1024   # the most router outputs the routing kernel keeps in shared memory
 
 
@@ -623,7 +683,9 @@ def route_experts(logits: torch.Tensor, correction: torch.Tensor, experts: int, 
                   groups: Optional[tuple] = None, scale: float = 1.0):
     """Scores over all router outputs (``scores``: "softmax" over the row, or
     "sigmoid" of each logit on its own), the ``top`` largest score + correction
-    chosen, weights = the chosen scores over their sum, times ``scale``.
+    chosen, weights = the chosen scores over their sum, times ``scale``. With
+    "chosen" the ``top`` largest logit + correction (a bias of the router's) are
+    chosen and their weights are the softmax over these sums alone.
     ``groups`` = (count, keep): the outputs form ``count`` equal groups of
     neighbours and only outputs of the ``keep`` groups with the largest sum of
     their two largest score + correction can be chosen. ``logits`` is float32
@@ -638,7 +700,7 @@ def route_experts(logits: torch.Tensor, correction: torch.Tensor, experts: int, 
     tokens, outputs = logits.shape
     _need(correction.numel() == outputs and 0 <= experts <= outputs and 0 < top <= outputs
           and outputs <= ROUTER_OUTPUTS, "the router's sizes do not fit")
-    _need(scores in ("softmax", "sigmoid"), f"unknown scores {scores!r}")
+    _need(scores in ROUTE_SCORES, f"unknown scores {scores!r}")
     count, keep = (int(groups[0]), int(groups[1])) if groups else (1, 1)
     if count > 1:
         _need(outputs % count == 0 and 1 <= keep <= count and keep * (outputs // count) >= top
@@ -649,7 +711,7 @@ def route_experts(logits: torch.Tensor, correction: torch.Tensor, experts: int, 
     dense = torch.empty((tokens, experts), dtype=torch.float32, device=device)
     on_identity = torch.empty((tokens,), dtype=torch.float32, device=device)
     _call("mxb_route_experts", logits.data_ptr(), correction.data_ptr(), chosen.data_ptr(), weights.data_ptr(),
-          dense.data_ptr(), on_identity.data_ptr(), tokens, outputs, experts, top, 1 if scores == "sigmoid" else 0,
+          dense.data_ptr(), on_identity.data_ptr(), tokens, outputs, experts, top, ROUTE_SCORES[scores],
           count, keep, float(scale), logits.stride(0), _stream())
     return chosen, weights, dense, on_identity
 
@@ -831,10 +893,11 @@ def mlstm_scan(proj: torch.Tensor, offsets, i_bias: torch.Tensor, f_bias: torch.
 
 
 def head_norm_gate(x: torch.Tensor, weight: torch.Tensor, gate: Optional[torch.Tensor], heads: int, eps: float,
-                   out_dtype: torch.dtype) -> torch.Tensor:
+                   out_dtype: torch.dtype, activation: str = "sigmoid") -> torch.Tensor:
     """Each head of x (float32 ``[tokens, heads * vdim]``) over its root mean
     square, times ``weight`` (all heads' size), times sigmoid(gate) (same shape,
-    rows may be strided)."""
+    rows may be strided), or silu(gate) with ``activation="silu"``."""
+    _need(activation in ("sigmoid", "silu"), f"unknown activation {activation!r}")
     _check(x, "x", (torch.float32,), 2)
     _check(weight, "weight", (torch.float32,), 1)
     tokens, width = x.shape
@@ -847,7 +910,27 @@ def head_norm_gate(x: torch.Tensor, weight: torch.Tensor, gate: Optional[torch.T
     _need(out_dtype in _CODES, "out_dtype must be float32 or bfloat16")
     out = torch.empty((tokens, width), dtype=out_dtype, device=x.device)
     _call("mxb_head_norm_gate", x.data_ptr(), weight.data_ptr(), _ptr(gate), ldg, gate_code, out.data_ptr(),
-          _CODES[out_dtype], tokens, heads, width // heads, float(eps), _stream())
+          _CODES[out_dtype], tokens, heads, width // heads, 1 if activation == "silu" else 0, float(eps), _stream())
+    return out
+
+
+def gated_norm(x: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, parts: int, eps: float, out_dtype: torch.dtype,
+               activation: str = "silu") -> torch.Tensor:
+    """u = x * act(gate) for x float32 ``[tokens, width]``, each of the row's
+    ``parts`` equal parts over its own root mean square, times ``weight``
+    (``[width]``). ``gate`` has x's shape (rows may be strided); act is "silu" or
+    "sigmoid"."""
+    _check(x, "x", (torch.float32,), 2)
+    _check(weight, "weight", (torch.float32,), 1)
+    tokens, width = x.shape
+    _need(parts >= 1 and width % parts == 0 and weight.numel() == width, "x, weight and the parts do not fit")
+    _need(gate.is_cuda and gate.dtype in _CODES and gate.dim() == 2 and gate.stride(1) == 1 and gate.shape == x.shape,
+          "gate must be [tokens, width] with unit column stride")
+    _need(activation in ("silu", "sigmoid") and out_dtype in _CODES, "unknown activation or out_dtype")
+    out = torch.empty((tokens, width), dtype=out_dtype, device=x.device)
+    _call("mxb_gated_norm", x.data_ptr(), gate.data_ptr(), gate.stride(0), _CODES[gate.dtype], weight.data_ptr(),
+          out.data_ptr(), _CODES[out_dtype], tokens, parts, width // parts, 1 if activation == "silu" else 0, float(eps),
+          _stream())
     return out
 
 
@@ -859,7 +942,7 @@ def delta_rule_max_dim() -> int:
 def delta_rule(qkv: torch.Tensor, offsets, beta: torch.Tensor, step: torch.Tensor, step_bias: torch.Tensor,
                rate: torch.Tensor, state: torch.Tensor, row_start: torch.Tensor, row_length: torch.Tensor,
                request_slots: torch.Tensor, heads: int, groups: int, dim: int, vdim: int,
-               longest: int = 0) -> torch.Tensor:
+               longest: int = 0, decay: str = "channel") -> torch.Tensor:
     """The gated delta rule with a decay per head and key channel over a step's
     tokens. ``qkv`` ``[tokens, columns]`` holds, from the column ``offsets``
     (q, k, v) on, groups * dim queries and keys and heads * vdim values (after
@@ -874,17 +957,50 @@ def delta_rule(qkv: torch.Tensor, offsets, beta: torch.Tensor, step: torch.Tenso
     value column's key channels side by side) is advanced in place; request row r brings ``row_length[r]`` tokens from packed token
     ``row_start[r]`` on (0: a padding row) and owns slot ``request_slots[r]``.
     Returns float32 ``[tokens, heads * vdim]``. ``longest``: the most tokens of
-    a row if known (a step of single tokens gets smaller blocks)."""
+    a row if known (a step of single tokens gets smaller blocks). ``decay``
+    "head": one decay per head; ``step`` is then ``[tokens, heads]`` of qkv's type
+    (a view of a wider tensor will do) and ``step_bias`` ``[heads]``."""
+    _need(decay in ("channel", "head"), f"unknown decay {decay!r}")
+    return _matrix_state(1 if decay == "head" else 0, qkv, offsets, beta, step, step_bias, rate, None, state, row_start,
+                         row_length, request_slots, heads, groups, dim, vdim, longest)
+
+
+def state_space_dual(xbc: torch.Tensor, offsets, step: torch.Tensor, step_bias: torch.Tensor, rate: torch.Tensor,
+                     skip: torch.Tensor, state: torch.Tensor, row_start: torch.Tensor, row_length: torch.Tensor,
+                     request_slots: torch.Tensor, heads: int, groups: int, dim: int, vdim: int,
+                     longest: int = 0) -> torch.Tensor:
+    """The state-space dual (Mamba-2) over a step's tokens. ``xbc`` holds, from
+    the column ``offsets`` (C, B, x) on, groups * dim values of C and of B and heads *
+    vdim of x; head h reads group h // (heads / groups). ``step`` ``[tokens, heads]``
+    of xbc's type are the step sizes' pre-activations: dt = softplus(step +
+    step_bias), g = exp(-rate dt); per head S <- g S + dt B x^T, y = S^T C + skip x.
+    ``state`` float32 ``[slots, heads, vdim, dim]`` (a value column's channels side by
+    side) is advanced in place; rows and slots as in ``delta_rule``. Returns
+    float32 ``[tokens, heads * vdim]``."""
+    return _matrix_state(2, xbc, offsets, None, step, step_bias, rate, skip, state, row_start, row_length, request_slots,
+                         heads, groups, dim, vdim, longest)
+
+
+def _matrix_state(mode: int, qkv, offsets, beta, step, step_bias, rate, skip, state, row_start, row_length, request_slots,
+                  heads: int, groups: int, dim: int, vdim: int, longest: int) -> torch.Tensor:
     _need(qkv.is_cuda and qkv.dtype in _CODES and qkv.dim() == 2 and qkv.stride(1) == 1,
           "qkv must be a CUDA [tokens, columns] tensor with unit column stride")
     tokens = qkv.shape[0]
-    _need(beta.is_cuda and beta.dtype == qkv.dtype and beta.dim() == 2 and beta.stride(1) == 1
-          and beta.shape == (tokens, heads), "beta must be [tokens, heads] of qkv's type")
-    _need(step.is_cuda and step.dtype == torch.float32 and step.dim() == 2 and step.stride(1) == 1
-          and step.shape == (tokens, heads * dim), "step must be float32 [tokens, heads * dim]")
+    per_head = lambda tensor: (tensor.is_cuda and tensor.dtype == qkv.dtype and tensor.dim() == 2
+                               and (tensor.stride(1) == 1 or heads == 1) and tensor.shape == (tokens, heads))
+    _need(mode == 2 or per_head(beta), "beta must be [tokens, heads] of qkv's type")
+    if mode == 0:
+        _need(step.is_cuda and step.dtype == torch.float32 and step.dim() == 2 and step.stride(1) == 1
+              and step.shape == (tokens, heads * dim), "step must be float32 [tokens, heads * dim]")
+    else:
+        _need(per_head(step), "step must be [tokens, heads] of qkv's type")
     _check(step_bias, "step_bias", (torch.float32,), 1)
     _check(rate, "rate", (torch.float32,), 1)
-    _need(step_bias.numel() == heads * dim and rate.numel() == heads, "step_bias or rate has the wrong size")
+    _need(step_bias.numel() == (heads * dim if mode == 0 else heads) and rate.numel() == heads,
+          "step_bias or rate has the wrong size")
+    if mode == 2:
+        _check(skip, "skip", (torch.float32,), 1)
+        _need(skip.numel() == heads, "skip has the wrong size")
     _check(state, "state", (torch.float32,), 4)
     _need(state.shape[1:] == (heads, vdim, dim), f"state must be [slots, {heads}, {vdim}, {dim}]")
     _need(heads % groups == 0 and 0 < dim <= delta_rule_max_dim(), "the head layout does not fit")
@@ -896,8 +1012,9 @@ def delta_rule(qkv: torch.Tensor, offsets, beta: torch.Tensor, step: torch.Tenso
     _need(max(q_off + groups * dim, k_off + groups * dim, v_off + heads * vdim) <= qkv.shape[1],
           "the column offsets reach beyond qkv")
     out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=qkv.device)
-    _call("mxb_delta_rule", qkv.data_ptr(), qkv.stride(0), q_off, k_off, v_off, beta.data_ptr(), beta.stride(0), 0,
-          step.data_ptr(), step.stride(0), step_bias.data_ptr(), rate.data_ptr(), state.data_ptr(), state.stride(0),
+    _call("mxb_delta_rule", qkv.data_ptr(), qkv.stride(0), q_off, k_off, v_off, _ptr(beta),
+          beta.stride(0) if beta is not None else 0, 0, step.data_ptr(), step.stride(0), step_bias.data_ptr(),
+          rate.data_ptr(), _ptr(skip), mode, state.data_ptr(), state.stride(0),
           state.shape[0], row_start.data_ptr(), row_length.data_ptr(), request_slots.data_ptr(), out.data_ptr(), rows,
           heads, groups, dim, vdim, _CODES[qkv.dtype], int(longest), status_word(qkv.device).data_ptr(), _stream())
     return out
@@ -1024,7 +1141,7 @@ def qk_norm_rope_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_out:
                        positions: torch.Tensor, q_weight: Optional[torch.Tensor],
                        k_weight: Optional[torch.Tensor], cos: Optional[torch.Tensor],
                        sin: Optional[torch.Tensor], eps: float, interleaved: bool = False,
-                       norm_scope: str = "head") -> None:
+                       norm_scope: str = "head", q_factors: Optional[torch.Tensor] = None) -> None:
     """RMSNorm of q and k (if weights are given; ``norm_scope`` "head": each
     head by itself, weights of head_dim values; "projection": all of a token's
     query heads together and all of its key heads together, weights as wide as
@@ -1033,7 +1150,8 @@ def qk_norm_rope_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_out:
     [tokens, heads, head_dim], k and v written into ``cache``
     [pages, 2, kv_heads, page_tokens, head_dim] at ``slots`` (a negative slot
     skips the token; ``cache=None`` writes nothing). q, k and v are
-    [tokens, heads * head_dim] views whose rows may be strided."""
+    [tokens, heads * head_dim] views whose rows may be strided. ``q_factors``
+    (float32, one per position): what the queries are multiplied by."""
     dtype = q.dtype
     for name, tensor in (("q", q), ("k", k), ("v", v)):
         _need(tensor.is_cuda and tensor.dtype == dtype and tensor.dtype in _CODES and tensor.dim() == 2
@@ -1073,25 +1191,28 @@ def qk_norm_rope_cache(q: torch.Tensor, k: torch.Tensor, v: torch.Tensor, q_out:
         _need(cos.shape == sin.shape, "cos and sin differ in shape")
         table_positions, rotary_dim = cos.shape[0], cos.shape[1] * 2
         _need(rotary_dim <= head_dim, "rotary_dim exceeds head_dim")
+    if q_factors is not None:
+        _check(q_factors, "q_factors", (torch.float32,), 1)
     _call("mxb_qk_norm_rope_cache", q.data_ptr(), k.data_ptr(), v.data_ptr(), q.stride(0), k.stride(0),
           v.stride(0), _ptr(q_out), _ptr(cache), _ptr(slots), positions.data_ptr(), _ptr(q_weight),
           _ptr(k_weight), _ptr(cos), _ptr(sin), table_positions, rotary_dim, 1 if interleaved else 0,
           1 if norm_scope == "projection" else 0, tokens, heads, kv_heads,
-          head_dim, page_tokens, num_pages, float(eps), _CODES[dtype],
+          head_dim, page_tokens, num_pages, float(eps), _CODES[dtype], _ptr(q_factors),
+          q_factors.numel() if q_factors is not None else 0,
           status_word(q.device).data_ptr(), _stream())
 
 
 def norm_rotate_heads(x: torch.Tensor, head_dim: int, positions: torch.Tensor,
                       weight: Optional[torch.Tensor] = None, cos: Optional[torch.Tensor] = None,
                       sin: Optional[torch.Tensor] = None, eps: float = 0.0, interleaved: bool = False,
-                      norm_scope: str = "head") -> torch.Tensor:
+                      norm_scope: str = "head", factors: Optional[torch.Tensor] = None) -> torch.Tensor:
     """RMSNorm (if ``weight``) and rotation (if tables) of x
-    [tokens, n * head_dim]; returns [tokens, n, head_dim]. Writes no cache."""
+    [tokens, n * head_dim], times ``factors[position]`` (if given); returns [tokens, n, head_dim]. Writes no cache."""
     _need(x.dim() == 2 and x.shape[1] % head_dim == 0, "x must be [tokens, n * head_dim]")
     out = torch.empty((x.shape[0], x.shape[1] // head_dim, head_dim), dtype=x.dtype, device=x.device)
     empty = x[:, :0]
     qk_norm_rope_cache(x, empty, empty, out, None, None, positions, weight, None, cos, sin, eps,
-                       interleaved=interleaved, norm_scope=norm_scope)
+                       interleaved=interleaved, norm_scope=norm_scope, q_factors=factors)
     return out
 
 
@@ -1115,12 +1236,25 @@ def _sink(sink, heads: int):
     return 1, float(sink), None
 
 
+def _score_bias(bias, heads: int):
+    """(pointer, far) as the attention kernels take a bias per head and distance:
+    None for none, or a contiguous float32 tensor ``[heads, far + 1]`` whose entry
+    n belongs to a key n positions back and whose last entry to all keys from
+    ``far`` positions back on."""
+    if bias is None:
+        return None, 0
+    _need(isinstance(bias, torch.Tensor) and bias.is_cuda and bias.dtype == torch.float32 and bias.is_contiguous()
+          and bias.dim() == 2 and bias.shape[0] == heads and bias.shape[1] >= 1,
+          f"a bias on the scores must be contiguous float32 [{heads}, distances] on the device")
+    return bias.data_ptr(), bias.shape[1] - 1
+
+
 def paged_attention_tile(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor,
                          block_tables: torch.Tensor, tile_request: torch.Tensor,
                          tile_start: torch.Tensor, tile_length: torch.Tensor,
                          positions: torch.Tensor, scale: float, window: int = 0, chunk: int = 0,
                          gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                         gate_per_head: bool = False, sink=None) -> torch.Tensor:
+                         gate_per_head: bool = False, sink=None, bias=None) -> torch.Tensor:
     """Attention of every query token over its request's cached keys (itself
     included) in float32; q is [tokens, heads, head_dim], out
     [tokens, heads, value_dim] with value_dim at most head_dim (the first
@@ -1134,7 +1268,8 @@ def paged_attention_tile(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor
     ``gate_per_head``; rows may be strided): the output is multiplied by
     sigmoid(gate) as it is written; ``sink``: the score of one more key that
     has no value and that every query sees (0.0: one more in the softmax's
-    denominator)."""
+    denominator); ``bias`` (float32 ``[heads, far + 1]``): what joins a capped
+    score by head and distance, its last entry for all keys further back."""
     dtype = q.dtype
     _check(q, "q", tuple(_CODES), 3)
     _check(out, "out", (dtype,), 3)
@@ -1165,7 +1300,7 @@ def paged_attention_tile(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor
           tile_start.data_ptr(), tile_length.data_ptr(), positions.data_ptr(), tiles, heads,
           kv_heads, head_dim, page_tokens, num_pages, int(window or 0), int(chunk or 0), float(scale), _CODES[dtype],
           _ptr(gate), gate_stride, planes, value_dim, float(softcap), 1 if gate_per_head else 0,
-          *_sink(sink, heads), status_word(q.device).data_ptr(), _stream())
+          *_sink(sink, heads), *_score_bias(bias, heads), status_word(q.device).data_ptr(), _stream())
     return out
 
 
@@ -1214,7 +1349,7 @@ def flash_prefill(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block
                   tile_request: torch.Tensor, tile_start: torch.Tensor, tile_length: torch.Tensor,
                   positions: torch.Tensor, scale: float, window: int = 0, kernel: str = "auto",
                   longest_context: int = 0, chunk: int = 0, gate: Optional[torch.Tensor] = None,
-                  softcap: float = 0.0, sink=None) -> torch.Tensor:
+                  softcap: float = 0.0, sink=None, bias=None) -> torch.Tensor:
     """Causal attention of prompt portions on the tensor cores (bfloat16,
     float32 softmax and accumulation); tiles hold up to 128 consecutive tokens
     of one request. ``kernel``: "tcgen05" (TMA, tensor memory), "mma" (the
@@ -1223,7 +1358,8 @@ def flash_prefill(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block
     lets the tcgen05 kernel share a tile's keys out among several blocks when
     the tiles alone would leave most of the GPU idle. ``softcap`` c: scores
     pass c tanh(s / c) ahead of the softmax. ``sink``: the score of one more
-    key that has no value and that every query sees."""
+    key that has no value and that every query sees. ``bias`` (float32
+    ``[heads, far + 1]``): joins the scores by head and distance."""
     _need(softcap >= 0.0, "the cap on the scores cannot be negative")
     _check(q, "q", (torch.bfloat16,), 3)
     _check(out, "out", (torch.bfloat16,), 3)
@@ -1260,7 +1396,7 @@ def flash_prefill(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block
               block_tables.data_ptr(), block_tables.shape[1], tile_request.data_ptr(), tile_start.data_ptr(),
               tile_length.data_ptr(), positions.data_ptr(), tokens, tiles, heads, kv_heads, head_dim,
               page_tokens, num_pages, int(window or 0), int(chunk or 0), float(scale), _CODES[q.dtype], shares, _ptr(partial),
-              _ptr(gate), gate_stride, float(softcap), *_sink(sink, heads),
+              _ptr(gate), gate_stride, float(softcap), *_sink(sink, heads), *_score_bias(bias, heads),
               status_word(q.device).data_ptr(), _stream())
         if shares > 1:
             global _launches
@@ -1270,7 +1406,7 @@ def flash_prefill(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block
           block_tables.shape[1], tile_request.data_ptr(), tile_start.data_ptr(), tile_length.data_ptr(),
           positions.data_ptr(), tiles, heads, kv_heads, head_dim, page_tokens, num_pages,
           int(window or 0), int(chunk or 0), float(scale), _CODES[q.dtype], _ptr(gate), gate_stride, float(softcap),
-          *_sink(sink, heads), status_word(q.device).data_ptr(), _stream())
+          *_sink(sink, heads), *_score_bias(bias, heads), status_word(q.device).data_ptr(), _stream())
     return out
 
 
@@ -1302,7 +1438,7 @@ def paged_attention_decode(q: torch.Tensor, cache: torch.Tensor, out: torch.Tens
                            longest_context: int, window: int = 0,
                            partial: Optional[torch.Tensor] = None, chunk: int = 0,
                            gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                           sink=None) -> torch.Tensor:
+                           sink=None, bias=None) -> torch.Tensor:
     """Attention of single tokens over their requests' cached keys, split
     along the keys. ``row_token[i]`` is the token (row of q and out) of the
     i-th decoded request, negative for a padding row; ``row_request[i]`` its
@@ -1313,7 +1449,8 @@ def paged_attention_decode(q: torch.Tensor, cache: torch.Tensor, out: torch.Tens
     the output is multiplied by sigmoid(gate) as it is written. ``softcap`` c:
     scores pass c tanh(s / c) ahead of the softmax. ``sink``: the score of one
     more key that has no value and that every query sees (it joins the
-    denominator where the splits are put together)."""
+    denominator where the splits are put together). ``bias`` (float32
+    ``[heads, far + 1]``): joins the scores by head and distance."""
     dtype = q.dtype
     _need(softcap >= 0.0, "the cap on the scores cannot be negative")
     _check(q, "q", tuple(_CODES), 3)
@@ -1341,7 +1478,7 @@ def paged_attention_decode(q: torch.Tensor, cache: torch.Tensor, out: torch.Tens
           block_tables.data_ptr(), block_tables.shape[1], row_token.data_ptr(), row_request.data_ptr(),
           positions.data_ptr(), rows, heads, kv_heads, head_dim, page_tokens, num_pages, splits,
           int(window or 0), int(chunk or 0), float(scale), _CODES[dtype], _ptr(gate), gate_stride, float(softcap),
-          *_sink(sink, heads), status_word(q.device).data_ptr(), _stream())
+          *_sink(sink, heads), *_score_bias(bias, heads), status_word(q.device).data_ptr(), _stream())
     return out
 
 
@@ -1370,7 +1507,7 @@ def paged_attention_decode_project(q: torch.Tensor, cache: torch.Tensor, block_t
                                    scale: float, longest_context: int, weight: torch.Tensor,
                                    window: int = 0, chunk: int = 0,
                                    gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                                   sink=None) -> torch.Tensor:
+                                   sink=None, bias=None) -> torch.Tensor:
     """``paged_attention_decode`` followed at once by the output projection
     ``weight`` ``[hidden, heads * head_dim]``, for steps of up to 64 tokens in
     bfloat16. Returns float32 ``[heads, tokens, hidden]``: the projection's sum
@@ -1398,7 +1535,7 @@ def paged_attention_decode_project(q: torch.Tensor, cache: torch.Tensor, block_t
           block_tables.data_ptr(), block_tables.shape[1], row_token.data_ptr(), row_request.data_ptr(),
           positions.data_ptr(), rows, tokens, heads, kv_heads, head_dim, page_tokens, num_pages, splits,
           int(window or 0), int(chunk or 0), float(scale), weight.data_ptr(), weight.stride(0), hidden, summands.data_ptr(),
-          _ptr(gate), gate_stride, float(softcap), *_sink(sink, heads),
+          _ptr(gate), gate_stride, float(softcap), *_sink(sink, heads), *_score_bias(bias, heads),
           status_word(q.device).data_ptr(), _stream())
     return summands
 
@@ -1472,15 +1609,18 @@ def gemm_skinny_takes(a: torch.Tensor, w: torch.Tensor, swiglu: bool = False) ->
     return gemm_stream_supported(a, w, swiglu) or gemm_skinny_supported(a, w)
 
 
-GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1}   # act of a gated feed-forward, act(gate) * up
+# act of a gated feed-forward, act(gate) * up; "clamped": min(gate, limit) sigmoid(1.702 min(gate, limit)) *
+# (clamp(up, -limit, limit) + 1)
+GATE_ACTIVATIONS = {"silu": 0, "gelu_tanh": 1, "clamped": 2}
 
 
 def gemm_skinny(a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype = torch.bfloat16,
                 swiglu: bool = False, out: Optional[torch.Tensor] = None, kernel: str = "auto",
-                activation: str = "silu") -> torch.Tensor:
+                activation: str = "silu", limit: float = 0.0) -> torch.Tensor:
     """a [m <= 64, k] times w [n, k] transposed, reading w once. With
     ``swiglu`` w holds gate rows then up rows and the result is
-    act(gate) * up, [m, n / 2], act being ``activation`` ("silu", "gelu_tanh"). ``kernel``: "stream" (rows of w by bulk copy
+    act(gate) * up, [m, n / 2], act being ``activation`` ("silu", "gelu_tanh";
+    "clamped" with ``limit``, see GATE_ACTIVATIONS). ``kernel``: "stream" (rows of w by bulk copy
     into shared memory, m <= 16), "load" (16-byte loads into registers) or
     "auto": stream where it takes the shape, the output is not wider than
     STREAM_COLUMNS and k is at most STREAM_K (the layers of a small model,
@@ -1505,10 +1645,11 @@ def gemm_skinny(a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype = torch
     if streams and (kernel == "stream" or not loads or (columns <= STREAM_COLUMNS and k <= STREAM_K)):
         _call("mxb_gemm_stream", out.data_ptr(), _CODES[out_dtype], a.data_ptr(), w.data_ptr(), m, n, k,
               a.stride(0), w.stride(0), out.stride(0), columns if swiglu else 0, GATE_ACTIVATIONS[activation],
-              status_word(a.device).data_ptr(), _stream())
+              float(limit), status_word(a.device).data_ptr(), _stream())
         return out
     _call("mxb_gemm_skinny", out.data_ptr(), _CODES[out_dtype], a.data_ptr(), w.data_ptr(), m, n, k,
-          a.stride(0), w.stride(0), out.stride(0), columns if swiglu else 0, GATE_ACTIVATIONS[activation], _stream())
+          a.stride(0), w.stride(0), out.stride(0), columns if swiglu else 0, GATE_ACTIVATIONS[activation],
+          float(limit), _stream())
     return out
 
 
@@ -1558,9 +1699,11 @@ def gemm_bf16(a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype = torch.b
     return result
 
 
-def silu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, activation: str = "silu") -> torch.Tensor:
+def silu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, activation: str = "silu",
+             limit: float = 0.0) -> torch.Tensor:
     """out[t, i] = act(gate_up[t, i]) * gate_up[t, I + i], float32 inside; act is
-    silu, or with ``activation="gelu_tanh"`` the tanh form of gelu."""
+    silu, or with ``activation="gelu_tanh"`` the tanh form of gelu, or "clamped"
+    with ``limit`` (see GATE_ACTIVATIONS)."""
     _check(gate_up, "gate_up", tuple(_CODES), 2)
     tokens, width = gate_up.shape
     _need(width % 2 == 0, "gate_up must hold gate and up side by side")
@@ -1570,7 +1713,7 @@ def silu_mul(gate_up: torch.Tensor, out: Optional[torch.Tensor] = None, activati
     _check(out, "out", (gate_up.dtype,), 2)
     _need(out.shape == (tokens, inter), "out has the wrong shape")
     _call("mxb_silu_mul", out.data_ptr(), gate_up.data_ptr(), _CODES[gate_up.dtype], tokens, inter,
-          GATE_ACTIVATIONS[activation], _stream())
+          GATE_ACTIVATIONS[activation], float(limit), _stream())
     return out
 
 

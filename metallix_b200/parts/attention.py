@@ -26,6 +26,13 @@ query head a learned score of its own. ``q_bias`` / ``k_bias`` / ``v_bias``
 compute type. ``shared_kv`` marks a layer without key and value projections:
 it reads the rows another layer of the same head layout and rotation wrote
 into the cache entry it is given, with its own queries, mask, cap and sink.
+``out_bias`` (a tensor name)
+is added to the output projection. ``query_factors`` (a position part with a
+table ``factors``) multiplies a query by a number of its position.
+``distance_bias`` = {weight, far} adds a learned number per head and distance
+to the scores: the tensor ``[rows, heads]`` gives its first half of rows to the
+distances 0, 1, ... and the others, logarithmically wider, to those up to ``far``
+(``distance_rows``).
 ``value_position`` (a rotary position part over
 the values' width) turns the value of position j by j before it is cached and
 turns each head's output at position i back by i, so that what a query takes
@@ -38,7 +45,9 @@ called through its own interface and only the cache write stays here.
 """
 from __future__ import annotations
 
-from typing import Dict, Optional
+import math
+from fractions import Fraction
+from typing import Dict, List, Optional
 
 import numpy as np
 import torch
@@ -54,6 +63,30 @@ TILE_TOKENS = 16     # query tokens per tile of the general kernel (csrc/kernels
 WIDE_TOKENS = 128    # ... of the tensor-core prompt kernels (csrc/kernels/attention_prefill*.cu)
 PROJECT_TOKENS = 32  # decode steps of up to this many tokens merge their splits and project in one kernel
 LONG_CONTEXT = 2048  # a portion of a prompt that sees this many keys or more counts as behind a long context
+
+
+def distance_rows(rows: int, far) -> List[int]:
+    """For each distance n = 0, 1, ... the row of a bias table that it reads, up
+    to and including the first distance from which on every one reads the last
+    row. With h = rows // 2: n itself below h, else min(rows - 1, h + floor(ln(n / h)
+    / ln(far / h) * (rows - h))). The floor is taken exactly, in integers: the
+    expression reaches k where n^w >= h^w (far / h)^k, w = rows - h."""
+    half, wide = rows // 2, rows - rows // 2
+    far = Fraction(far)
+    if half < 1 or far <= half:
+        raise ValueError(f"a bias table of {rows} rows and distances up to {far}: the far half would be empty")
+    out = list(range(half))
+    begin = half
+    for step in range(1, wide):       # row half + step starts at the first n that reaches step
+        bound = Fraction(half) ** wide * (far / half) ** step
+        n = max(begin, int(half * math.exp(math.log(far / half) * step / wide)) - 1)
+        while n > begin and (n - 1) ** wide >= bound:
+            n -= 1
+        while n ** wide < bound:
+            n += 1
+        out.extend([half + step - 1] * (n - begin))
+        begin = n
+    return out + [rows - 1]
 
 
 def attention_tiles(plan: StepPlan) -> Prepared:
@@ -141,7 +174,8 @@ def tiles_of(ctx: StepContext) -> Dict[str, object]:
 
 def attend_cached(q_heads: torch.Tensor, cache: CacheView, ctx: StepContext, *, scale: float, window: int = 0,
                   chunk: int = 0, softcap: float = 0.0, gate: Optional[torch.Tensor] = None, gate_per_head: bool = False,
-                  split_decode: bool = False, flash: bool = False, project=None, sink: Optional[float] = None):
+                  split_decode: bool = False, flash: bool = False, project=None, sink: Optional[float] = None,
+                  bias: Optional[torch.Tensor] = None):
     """Attention of a step's queries ``[tokens, heads, head_dim]`` over what the
     cache entry holds (this step's rows included), each kind of request on the
     kernel made for it: single tokens split along the keys, portions of prompts
@@ -164,20 +198,20 @@ def attend_cached(q_heads: torch.Tensor, cache: CacheView, ctx: StepContext, *, 
         return ops.paged_attention_decode_project(
             q_heads, cache.pool, cache.block_tables, tiles["decode_token"], tiles["decode_request"],
             ctx.positions, scale, tiles["longest_context"], project.weight, window, chunk, gate=gate,
-            softcap=softcap, sink=sink), True
+            softcap=softcap, sink=sink, bias=bias), True
     out = torch.empty_like(q_heads)
     if split:
         # Requests that bring one token: split along the keys.
         ops.paged_attention_decode(q_heads, cache.pool, out, cache.block_tables, tiles["decode_token"],
                                    tiles["decode_request"], ctx.positions, scale, tiles["longest_context"], window,
-                                   chunk=chunk, gate=gate, softcap=softcap, sink=sink)
+                                   chunk=chunk, gate=gate, softcap=softcap, sink=sink, bias=bias)
     if flash:
         # Requests that bring several tokens: tensor cores, tiles of 128.
         if tiles["wide_request"].numel():
             ops.flash_prefill(q_heads, cache.pool, out, cache.block_tables, tiles["wide_request"],
                               tiles["wide_start"], tiles["wide_length"], ctx.positions, scale, window,
                               longest_context=tiles["longest_keys"], chunk=chunk, gate=gate, softcap=softcap,
-                              sink=sink)
+                              sink=sink, bias=bias)
         rest = None if split else slice(multi_tiles, None)   # single tokens not yet served
     else:
         rest = slice(0, multi_tiles) if split else slice(0, None)
@@ -185,7 +219,7 @@ def attend_cached(q_heads: torch.Tensor, cache: CacheView, ctx: StepContext, *, 
         ops.paged_attention_tile(q_heads, cache.pool, out, cache.block_tables, tiles["tile_request"][rest],
                                  tiles["tile_start"][rest], tiles["tile_length"][rest], ctx.positions,
                                  scale, window, chunk, gate=gate, softcap=softcap, gate_per_head=gate_per_head,
-                                 sink=sink)
+                                 sink=sink, bias=bias)
     return out, False
 
 
@@ -260,6 +294,23 @@ class GQAttention:
         self.o = Linear(weights.take(spec["o_proj"]), runtime)
         if (self.o.out_features, self.o.in_features) != (self.hidden_size, self.out_size):
             raise ValueError(f"{spec['o_proj']} is {tuple(self.o.weight.shape)}")
+        # added to the output projection; kept apart for a caller that adds it in a pass it makes anyway
+        self.out_bias = None
+        if spec.get("out_bias"):
+            values = weights.take(spec["out_bias"])
+            if values.numel() != self.hidden_size:
+                raise ValueError(f"{spec['out_bias']} has {values.numel()} values, expected {self.hidden_size}")
+            self.out_bias = values.to(device=runtime.device, dtype=torch.float32).reshape(-1).contiguous()
+        factors = build_part("position", spec.get("query_factors"), weights, runtime)
+        self.query_factors = None if factors is None else factors.factors
+        self.distance_bias = None      # float32 [heads, distances]: the table spread over the distances
+        if spec.get("distance_bias") is not None:
+            name, far = spec["distance_bias"]["weight"], spec["distance_bias"]["far"]
+            table = weights.take(name)
+            if table.dim() != 2 or table.shape[1] != self.num_heads:
+                raise ValueError(f"{name} is {tuple(table.shape)}, expected [rows, {self.num_heads}]")
+            rows = torch.tensor(distance_rows(table.shape[0], far), dtype=torch.long, device=table.device)
+            self.distance_bias = table.to(torch.float32)[rows].t().contiguous().to(runtime.device)
         self.q_norm = build_part("norm", spec.get("q_norm"), weights, runtime)
         self.k_norm = build_part("norm", spec.get("k_norm"), weights, runtime)
         self.position = build_part("position", spec.get("position"), weights, runtime)
@@ -311,16 +362,25 @@ class GQAttention:
         return tiles_of(ctx)
 
     def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
-        return self._attend(x, ctx, cache, summands=False)
+        if self.out_bias is None:
+            return self._attend(x, ctx, cache, summands=False)
+        return ops.add_bias(self._attend(x, ctx, cache, summands=False, out_dtype=torch.float32), self.out_bias, self.dtype)
 
     def forward_summands(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
         """``forward`` for a caller that adds up summands: where one kernel can
         put the splits of a decode step together and project them head by head,
         the result is float32 ``[heads, tokens, hidden]`` whose sum over the
         heads is ``forward``'s output; otherwise ``forward``'s output itself."""
+        if self.out_bias is not None:
+            return self.forward(x, ctx, cache)
         return self._attend(x, ctx, cache, summands=True)
 
-    def _attend(self, x: torch.Tensor, ctx: StepContext, cache: CacheView, summands: bool) -> torch.Tensor:
+    def forward_unbiased(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
+        """``forward_summands`` without ``out_bias``, for a caller that adds it itself."""
+        return self._attend(x, ctx, cache, summands=True)
+
+    def _attend(self, x: torch.Tensor, ctx: StepContext, cache: CacheView, summands: bool,
+                out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
         tokens = x.shape[0]
         if self.bias is not None:
             # the product leaves in float32 and meets the bias there: one rounding to the compute type
@@ -335,7 +395,7 @@ class GQAttention:
         if self.value_position is not None and self.own_keys:     # cached turned by their own position
             v = self._turn_values(v, ctx).view(tokens, self.v_size)
         if self.value_dim != self.head_dim:
-            return self._attend_unequal(x, q, k, v, gate, ctx, cache)
+            return self._attend_unequal(x, q, k, v, gate, ctx, cache, out_dtype)
         q_heads = torch.empty((tokens, self.num_heads, self.head_dim), dtype=self.dtype, device=x.device)
         write = cache.write and cache.slots is not None and self.own_keys
         if not self.own_keys and self.fused:
@@ -345,7 +405,8 @@ class GQAttention:
                 cos=self.position.cos if self.position is not None else None,
                 sin=self.position.sin if self.position is not None else None,
                 eps=self.q_norm.eps if self.q_norm is not None else 0.0,
-                interleaved=bool(getattr(self.position, "interleaved", False)), norm_scope=self.norm_scope)
+                interleaved=bool(getattr(self.position, "interleaved", False)), norm_scope=self.norm_scope,
+                factors=self.query_factors)
         elif self.fused:
             eps = self.q_norm.eps if self.q_norm is not None else (self.k_norm.eps if self.k_norm else 0.0)
             ops.qk_norm_rope_cache(
@@ -355,7 +416,8 @@ class GQAttention:
                 self.k_norm.weight if self.k_norm is not None else None,
                 self.position.cos if self.position is not None else None,
                 self.position.sin if self.position is not None else None, eps,
-                interleaved=bool(getattr(self.position, "interleaved", False)), norm_scope=self.norm_scope)
+                interleaved=bool(getattr(self.position, "interleaved", False)), norm_scope=self.norm_scope,
+                q_factors=self.query_factors)
         else:
             if not self.own_keys:
                 raise ValueError("a layer that reads another layer's keys needs head norms and a position part "
@@ -374,6 +436,9 @@ class GQAttention:
                 k = k_rot.contiguous().view(tokens, self.kv_size)
             else:
                 q_heads = q.contiguous().view(tokens, self.num_heads, self.head_dim)
+            if self.query_factors is not None:
+                q_heads = ops.norm_rotate_heads(q_heads.view(tokens, self.q_size), self.head_dim, ctx.positions,
+                                                factors=self.query_factors)
             if write:
                 ops.write_cache(k, v, cache.pool, cache.slots, ctx.positions)
         if self.gate_scope == "head" and gate is not None and (self.split_decode or self.flash):
@@ -385,14 +450,16 @@ class GQAttention:
         out, projected = attend_cached(
             q_heads, cache, ctx, scale=self.scale, window=self.window, chunk=self.chunk, softcap=self.softcap, gate=gate,
             gate_per_head=per_head_gate, split_decode=self.split_decode, flash=self.flash,
-            project=self.o if summands and self.value_position is None else None, sink=self.sink)
+            project=self.o if summands and self.value_position is None else None, sink=self.sink,
+            bias=self.distance_bias)
         if projected:
             return out
         if self.value_position is not None:
             out = self._turn_values(out.view(tokens, self.q_size), ctx, back=True)
-        return self.o.forward(out.view(tokens, self.q_size))
+        return self.o.forward(out.view(tokens, self.q_size), out_dtype=out_dtype)
 
-    def _attend_unequal(self, x, q, k, v, gate, ctx: StepContext, cache: CacheView) -> torch.Tensor:
+    def _attend_unequal(self, x, q, k, v, gate, ctx: StepContext, cache: CacheView,
+                        out_dtype: Optional[torch.dtype] = None) -> torch.Tensor:
         """Values wider or narrower than the keys: a cached row is as wide as
         the wider of the two; queries, keys or values are padded with zeros up
         to it, and the output keeps the first ``value_dim`` values."""
@@ -414,7 +481,8 @@ class GQAttention:
             parts.append(ops.norm_rotate_heads(
                 rows, self.head_dim, ctx.positions, weight=weight, cos=self.position.cos if tables else None,
                 sin=self.position.sin if tables else None, eps=norm.eps if weight is not None else 0.0,
-                interleaved=bool(getattr(self.position, "interleaved", False)), norm_scope=self.norm_scope))
+                interleaved=bool(getattr(self.position, "interleaved", False)), norm_scope=self.norm_scope,
+                factors=self.query_factors if not parts else None))     # the queries come first
         q_heads, k_heads = parts
         pad = lambda t, have: torch.nn.functional.pad(t, (0, width - have)) if have < width else t
         q_rows = pad(q_heads, self.head_dim).contiguous()
@@ -428,10 +496,10 @@ class GQAttention:
         ops.paged_attention_tile(q_rows, cache.pool, out, cache.block_tables, tiles["tile_request"],
                                  tiles["tile_start"], tiles["tile_length"], ctx.positions, self.scale, self.window,
                                  self.chunk, gate=gate, softcap=self.softcap,
-                                 gate_per_head=self.gate_scope == "head", sink=self.sink)
+                                 gate_per_head=self.gate_scope == "head", sink=self.sink, bias=self.distance_bias)
         if self.value_position is not None:
             out = self._turn_values(out.view(tokens, self.out_size), ctx, back=True)
-        return self.o.forward(out.view(tokens, self.out_size))
+        return self.o.forward(out.view(tokens, self.out_size), out_dtype=out_dtype)
 
     def weight_bytes(self) -> int:
         return self.qkv.weight_bytes() + self.o.weight_bytes()

@@ -7,6 +7,10 @@ is float32; a block receives the previous block's output not yet added
 (``pending``) so that every residual sum runs inside the norm kernel that
 follows it.
 
+The feed-forward half is optional. A mixer made of two may hand on a pair whose
+parts pass norms of their own on their way into the stream; the second norm's
+kernel then does that too.
+
 ``sandwich_residual`` puts a second norm behind each sublayer:
 r = x + post1(mixer(norm1(x))); x' = r + post2(feed_forward(norm2(r))), the
 feed-forward half being optional. What a sublayer leaves is handed on with
@@ -53,26 +57,33 @@ class PreNormResidualBlock:
         self.name = layer.name
         self.mixer_norm = build_part("norm", layer.mixer_norm, weights, runtime)
         self.mixer = build_part("mixer", layer.mixer, weights, runtime)
-        self.feed_forward_norm = build_part("norm", layer.feed_forward_norm, weights, runtime)
         self.feed_forward = build_part("feed_forward", layer.feed_forward, weights, runtime)
+        self.feed_forward_norm = None
+        if self.feed_forward is not None:
+            if layer.feed_forward_norm is None:
+                raise ValueError(f"{layer.name}: a feed-forward needs its norm")
+            self.feed_forward_norm = build_part("norm", layer.feed_forward_norm, weights, runtime)
         self.dtype = runtime.dtype
         # A mixer may leave its output as summands [parts, tokens, hidden] when
         # the norm that takes it next adds them up in its own pass over the row.
         summands = getattr(self.mixer, "forward_summands", None)
         self.mix = summands if summands is not None and getattr(self.feed_forward_norm, "adds_summands", False) \
             else self.mixer.forward
+        # ... or as something that joins the stream in a way of its own.
+        if getattr(self.mixer, "leaves_pending", False):
+            self.mix = self.mixer.forward_pending
 
     def parts(self):
         return [self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward]
 
-    def forward(self, residual: torch.Tensor, pending, ctx: StepContext,
-                cache: CacheView) -> torch.Tensor:
+    def forward(self, residual: torch.Tensor, pending, ctx: StepContext, cache: CacheView):
         """``residual`` (float32, updated in place) plus ``pending`` (a tensor,
-        or a ``Pending`` that carries the norm it passes first) is the layer's
-        input; returns the feed-forward output, to be added by whoever runs
-        next."""
+        or what carries the way it joins) is the layer's input; returns the last
+        sublayer's output, to be added by whoever runs next."""
         mixer_in = self.mixer_norm.add_forward(residual, pending, self.dtype)
         mixed = self.mix(mixer_in, ctx, cache)
+        if self.feed_forward is None:
+            return mixed
         feed_in = self.feed_forward_norm.add_forward(residual, mixed, self.dtype)
         return self.feed_forward.forward(feed_in, ctx)
 

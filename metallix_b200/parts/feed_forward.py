@@ -2,7 +2,9 @@
 u = m Wu^T (crates/models/qwen/src/forward.rs:1904-1920). Gate and up weights
 are stacked so that one product yields both; SiLU and the product with u are
 float32 inside the kernel. ``activation="gelu_tanh"`` puts the tanh form of
-gelu in SiLU's place, in every kernel that holds the activation.
+gelu in SiLU's place, in every kernel that holds the activation;
+``activation="clamped"`` bounds both halves by ``limit``: with g = min(gate, limit)
+and u = clamp(up, -limit, limit), g sigmoid(1.702 g) (u + 1).
 
 ``dense_ff`` is the feed-forward without a gate: d = act(m Wu^T) Wd^T, the
 activation a parameter (``relu_squared``: max(z, 0)^2).
@@ -16,7 +18,9 @@ its own; ``groups`` = (count, keep) lets the choice fall only on the best
 groups of neighbouring experts; ``scale`` multiplies the weights;
 ``activation="swiglu"`` makes an expert a gated feed-forward
 down(silu(gate(h)) * up(h)); ``shared`` names a gated feed-forward that every
-token uses, added behind a sigmoid gate of one number per token."""
+token uses, added behind a sigmoid gate of one number per token, or as it is
+without ``shared_gate``; ``scores="chosen"`` chooses by the logits plus
+``logit_bias`` and weighs by the softmax over the chosen ones alone."""
 from __future__ import annotations
 
 import torch
@@ -46,13 +50,17 @@ class SwiGLU:
         self.activation = spec.get("activation") or "silu"
         if self.activation not in ops.GATE_ACTIVATIONS:
             raise ValueError(f"activation {self.activation!r}; one of {sorted(ops.GATE_ACTIVATIONS)}")
+        self.limit = float(spec.get("limit") or 0.0)
+        if self.activation == "clamped" and not self.limit > 0.0:
+            raise ValueError("the clamped activation needs a positive limit")
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
         few = ops.SKINNY_ROWS if x.shape[1] <= ops.STREAM_K else ops.SKINNY_ROWS // 2   # as ops.gemm_bf16
         if (x.shape[0] <= few and self.gate_up.backend in ("auto", "skinny")
                 and ops.gemm_skinny_takes(x, self.gate_up.weight, swiglu=True)):
             # A decode step: gate, up and the activation in one pass over the weights.
-            return self.down.forward(ops.gemm_skinny(x, self.gate_up.weight, swiglu=True, activation=self.activation))
+            return self.down.forward(ops.gemm_skinny(x, self.gate_up.weight, swiglu=True, activation=self.activation,
+                                                     limit=self.limit))
         # From about 1,500 rows on the tcgen05 product with the activation in its
         # epilogue beats the library's product followed by an activation pass
         # (28 against 31 us at 2,048 rows of this model; 21 against 19 at 1,024,
@@ -64,8 +72,9 @@ class SwiGLU:
             from .. import tensor_core
             if tensor_core.supports(x, self.gate_up.weight, torch.bfloat16):
                 # gate, up and the activation in the product's epilogue
-                return self.down.forward(tensor_core.gemm_swiglu(x, self.gate_up.weight, activation=self.activation))
-        return self.down.forward(ops.silu_mul(self.gate_up.forward(x), activation=self.activation))
+                return self.down.forward(tensor_core.gemm_swiglu(x, self.gate_up.weight, activation=self.activation,
+                                                                 limit=self.limit))
+        return self.down.forward(ops.silu_mul(self.gate_up.forward(x), activation=self.activation, limit=self.limit))
 
     def weight_bytes(self) -> int:
         return self.gate_up.weight_bytes() + self.down.weight_bytes()
@@ -126,8 +135,8 @@ class RoutedExperts:
         self.scores = spec.get("scores") or "softmax"
         self.groups = tuple(int(v) for v in spec["groups"]) if spec.get("groups") else None
         self.weight_scale = float(spec.get("scale") or 1.0)
-        if self.scores not in ("softmax", "sigmoid"):
-            raise ValueError(f"scores {self.scores!r}; 'softmax' or 'sigmoid'")
+        if self.scores not in ops.ROUTE_SCORES:
+            raise ValueError(f"scores {self.scores!r}; one of {sorted(ops.ROUTE_SCORES)}")
         if self.groups is not None:
             count, keep = self.groups
             if count < 1 or outputs % count or not 1 <= keep <= count or keep * (outputs // count) < self.top:
@@ -155,16 +164,21 @@ class RoutedExperts:
         self.outputs = outputs
         self.shared = None
         if spec.get("shared") is not None:
-            # an expert for every token, out += sigmoid(h . w) shared(h): its gate's row rides under the router's
+            # an expert for every token, out += sigmoid(h . w) shared(h): its gate's row rides under the router's;
+            # without a gate, out += shared(h)
             self.shared = build_part("feed_forward", spec["shared"], weights, runtime)
+        self.shared_gated = self.shared is not None and spec.get("shared_gate") is not None
+        if self.shared_gated:
             gate = weights.take(spec["shared_gate"])
             if gate.numel() != hidden:
                 raise ValueError(f"{spec['shared_gate']} has {gate.numel()} values, expected {hidden}")
             router = torch.cat([router.to(runtime.device), gate.reshape(1, hidden).to(runtime.device)], dim=0)
         self.router = Linear(router, runtime)
-        correction = weights.take(spec["correction"]) if spec.get("correction") else torch.zeros(outputs)
+        # what joins the scores for the choice alone, or (logit_bias) the logits themselves
+        extra = spec.get("logit_bias") if self.scores == "chosen" else spec.get("correction")
+        correction = weights.take(extra) if extra else torch.zeros(outputs)
         if correction.numel() != outputs:
-            raise ValueError(f"{spec['correction']} has {correction.numel()} values, expected {outputs}")
+            raise ValueError(f"{extra} has {correction.numel()} values, expected {outputs}")
         self.correction = correction.to(device=runtime.device, dtype=torch.float32).reshape(-1).contiguous()
         self.hidden_size, self.intermediate_size = hidden, ff
 
@@ -172,7 +186,9 @@ class RoutedExperts:
         """float32 ``[tokens, hidden]``."""
         logits = self.router.forward(x, out_dtype=torch.float32)
         out = self._routed(x, logits[:, :self.outputs])
-        if self.shared is not None:
+        if self.shared is not None and not self.shared_gated:
+            ops.add_(out, self.shared.forward(x, ctx))
+        elif self.shared is not None:
             ops.add_gated_rows(out, self.shared.forward(x, ctx), logits[:, self.outputs:])
         return out
 

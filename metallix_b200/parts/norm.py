@@ -36,8 +36,10 @@ class RMSNorm:
     def add_forward(self, residual: torch.Tensor, delta, out_dtype: torch.dtype) -> torch.Tensor:
         """residual += delta (float32, in place), then the norm of the sum.
         ``delta`` may be float32 ``[parts, rows, size]``: its parts are added up
-        first. A ``Pending`` delta passes its own norm before the sum, in the
+        first; or ``[size]``: it joins every row. A ``Pending`` delta passes its own norm before the sum, in the
         same pass over the row when that norm is an RMSNorm too."""
+        if delta is not None and hasattr(delta, "settle_and_norm"):   # ... that makes this norm in the same pass
+            return delta.settle_and_norm(residual, self.weight, self.eps, out_dtype)
         if delta is not None and hasattr(delta, "settle"):   # a block arrangement's own way of joining the stream
             delta.settle(residual)
             delta = None
@@ -107,6 +109,9 @@ class DynamicTanh:
             delta = None
         if delta is not None and delta.dim() == 3:
             delta = delta.sum(0)
+        elif delta is not None and delta.dim() == 1:      # one row for all
+            ops.add_(residual, delta)
+            delta = None
         return ops.stream_mix(residual.view(residual.shape[0], 1, self.size), result=delta, mix=self._one,
                               out_weights=self._one, alpha=self.alpha, norm_weight=self.weight, norm_bias=self.bias,
                               out_dtype=out_dtype)

@@ -22,6 +22,11 @@ pair that makes t turns over ``original`` positions, lo = max(floor(where(fast))
 max(hi - lo, 0.001), 0, 1), pair i gets f_i / factor * ramp_i + f_i (1 - ramp_i),
 and cos and sin are both multiplied by 0.1 ln(factor) + 1 (``rotary_magnitude``).
 
+A query's temperature is the third kind: ``log_temperature`` multiplies the
+query at position p by 1 + coef * ln(floor((p + 1) / every) + 1), a table of float32
+numbers (``factors``) formed in float64 that the attention hands to the kernel
+that writes the queries.
+
 Angles are formed in float64 (position times frequency), cos and sin are
 rounded once to float32 tables that the kernels index by position.
 """
@@ -135,3 +140,22 @@ def _builder(cls):
 
 register_part("position", "rope_half", _builder(RotaryHalf))
 register_part("position", "rope_interleaved", _builder(RotaryInterleaved))
+
+
+class LogTemperature:
+    kind = "log_temperature"
+
+    def __init__(self, coef: float, every: float, runtime: Runtime):
+        if not every > 0:
+            raise ValueError(f"a temperature that rises every {every} positions")
+        # Layers with the same parameters share one table.
+        key = ("log_temperature", float(coef), float(every), runtime.max_positions, str(runtime.device))
+        if key not in runtime.shared:
+            position = torch.arange(runtime.max_positions, dtype=torch.float64)
+            factors = 1.0 + float(coef) * torch.log(torch.floor((position + 1.0) / float(every)) + 1.0)
+            runtime.shared[key] = factors.to(torch.float32).contiguous().to(runtime.device)
+        self.factors = runtime.shared[key]
+
+
+register_part("position", "log_temperature",
+              lambda spec, weights, runtime: LogTemperature(spec["coef"], spec["every"], runtime))

@@ -314,3 +314,180 @@ class ChannelDelta:
 
 
 register_part("mixer", "channel_delta", lambda spec, weights, runtime: ChannelDelta(spec, weights, runtime))
+
+
+def _named(spec: PartSpec, weights: WeightStore, runtime: Runtime):
+    """(matrix, vector): readers of the tensors that a part's parameters name, with their shapes checked."""
+    def matrix(name, shape):
+        weight = weights.take(spec[name])
+        if tuple(weight.shape) != shape:
+            raise ValueError(f"{spec[name]} is {tuple(weight.shape)}, expected {shape}")
+        return weight
+
+    def vector(name, size):
+        tensor = weights.take(spec[name])
+        if tensor.numel() != size:
+            raise ValueError(f"{spec[name]} has {tensor.numel()} values, expected {size}")
+        return tensor.to(device=runtime.device, dtype=torch.float32).reshape(-1).contiguous()
+
+    return matrix, vector
+
+
+def _stacked_rows(matrices, runtime: Runtime, multiple: int = 8) -> Linear:
+    """One product over the same input, with rows of zeros at the end so that a
+    row of the result starts on the boundary that vector accesses need."""
+    rows = sum(m.shape[0] for m in matrices)
+    extra = -rows % multiple
+    if extra:
+        matrices = list(matrices) + [torch.zeros((extra, matrices[0].shape[1]), dtype=matrices[0].dtype,
+                                                 device=matrices[0].device)]
+    return Linear.stacked(matrices, runtime)
+
+
+class HeadDelta:
+    """The gated delta rule with one decay per head. As ``ChannelDelta``, but
+
+        g = exp(-exp(A_log_h) * softplus((a Wa^T)_h + dt_bias_h))      one number per head
+        S <- g S;  u = beta (v - S^T kn);  S <- S + kn u^T;  o = S^T qn
+
+    and each head's o over its root mean square, times a weight over V (shared by
+    the heads), is multiplied by silu(a Wg^T) ahead of Wo. One product gives q, k,
+    v, the gate and the pre-activations of the write strength and of the step
+    size; what enters the recurrence is float32 from there on."""
+
+    kind = "head_delta"
+    graph_safe = True
+    step_key = "request_rows"
+    prepare_step = staticmethod(request_rows)
+
+    def __init__(self, spec: PartSpec, weights: WeightStore, runtime: Runtime):
+        from .short_conv import ShortConv
+        hidden = spec["hidden_size"]
+        self.heads, self.groups = int(spec["num_heads"]), int(spec.get("num_kv_heads") or spec["num_heads"])
+        self.dim, self.vdim, self.eps = int(spec["head_dim"]), int(spec["value_dim"]), float(spec["eps"])
+        if self.heads % self.groups:
+            raise ValueError(f"{self.heads} heads cannot share {self.groups} groups of queries and keys")
+        if not 0 < self.dim <= ops.delta_rule_max_dim():
+            raise ValueError(f"keys of {self.dim} channels; the recurrence takes up to {ops.delta_rule_max_dim()}")
+        H, G, D, V = self.heads, self.groups, self.dim, self.vdim
+        matrix, vector = _named(spec, weights, runtime)
+        self.conv_channels = 2 * G * D + H * V
+        stacked, self.offsets, cursor = [], {}, 0
+        for name, rows in (("q_proj", G * D), ("k_proj", G * D), ("v_proj", H * V), ("gate_proj", H * V),
+                           ("beta_proj", H), ("step_proj", H)):
+            stacked.append(matrix(name, (rows, hidden)))
+            self.offsets[name] = cursor
+            cursor += rows
+        self.inputs = _stacked_rows(stacked, runtime)
+        self.step_bias = vector("step_bias", H)
+        self.rate = torch.exp(vector("a_log", H)).contiguous()
+        self.norm_weight = vector("norm", V).repeat(H).contiguous()       # one weight over V, the same for every head
+        taps = int(spec["conv_taps"])
+        conv_weight = torch.cat([matrix(name, (rows, taps)) for name, rows in
+                                 (("q_conv", G * D), ("k_conv", G * D), ("v_conv", H * V))], dim=0)
+        self.conv = ShortConv(PartSpec("short_conv", {"channels": self.conv_channels, "taps": taps, "weight": "conv",
+                                                      "bias": None, "activation": "silu"}),
+                              WeightStore({"conv": conv_weight}), runtime)
+        self.o = Linear(matrix("o_proj", (hidden, H * V)), runtime)
+        self.dtype = runtime.dtype
+
+    def cache_need(self) -> CacheNeed:
+        return CacheNeed(kind="several", members=(
+            CacheNeed(kind="state", state_shape=(self.heads, self.vdim, self.dim), state_dtype="float32"),
+            self.conv.cache_need()))
+
+    def parts(self):
+        return [self.conv]
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
+        if len(cache.members) != 2 or cache.members[0].state is None:
+            raise ValueError("the delta-rule mixer needs its two state entries of the cache")
+        rows = request_rows_of(ctx)
+        H, G, D, V, at = self.heads, self.groups, self.dim, self.vdim, self.offsets
+        proj = self.inputs.forward(x)       # every later step reads column ranges of it in place
+        qkv = self.conv.forward(proj[:, :self.conv_channels], ctx, cache.members[1])
+        mixed = ops.delta_rule(qkv, (0, G * D, 2 * G * D), proj[:, at["beta_proj"]:at["beta_proj"] + H],
+                               proj[:, at["step_proj"]:at["step_proj"] + H], self.step_bias, self.rate,
+                               cache.members[0].state, rows["row_start"], rows["row_length"], ctx.request_slots, H, G, D, V,
+                               longest=rows.get("longest", 0), decay="head")
+        gate = proj[:, at["gate_proj"]:at["gate_proj"] + H * V]
+        return self.o.forward(ops.head_norm_gate(mixed, self.norm_weight, gate, H, self.eps, self.dtype, activation="silu"))
+
+    def weight_bytes(self) -> int:
+        return self.inputs.weight_bytes() + self.o.weight_bytes()
+
+
+register_part("mixer", "head_delta", lambda spec, weights, runtime: HeadDelta(spec, weights, runtime))
+
+
+class StateSpaceDual:
+    """The state-space dual (Mamba-2): a Win^T = [z | x | B | C | dt] with H heads
+    of V values in z and x, G groups of N in B and C (head h reads group
+    h // (H / G)) and one dt per head; x, B and C together pass a short causal
+    convolution with bias and silu;
+
+        dt <- softplus(dt + dt_bias),  g = exp(-exp(A_log_h) dt)
+        S <- g S + dt B x^T,   y = S^T C + D_h x                          per head, S [N, V]
+
+    then y silu(z) (the gate comes first), each of ``norm_groups`` equal parts over
+    its own root mean square, times a weight, and Wo. S (float32, kept transposed
+    as ``[H, V, N]``) and the convolution's last inputs are kept per request in the
+    cache's state slots; the recurrence and the norm are float32 in both
+    precisions."""
+
+    kind = "state_space_dual"
+    graph_safe = True
+    step_key = "request_rows"
+    prepare_step = staticmethod(request_rows)
+
+    def __init__(self, spec: PartSpec, weights: WeightStore, runtime: Runtime):
+        from .short_conv import ShortConv
+        hidden = spec["hidden_size"]
+        self.heads, self.vdim = int(spec["num_heads"]), int(spec["value_dim"])
+        self.states, self.groups = int(spec["state_size"]), int(spec.get("groups") or 1)
+        self.norm_groups, self.eps = int(spec.get("norm_groups") or 1), float(spec["eps"])
+        H, V, N, G = self.heads, self.vdim, self.states, self.groups
+        self.inner = H * V
+        if H % G or self.inner % self.norm_groups:
+            raise ValueError(f"{H} heads in {G} groups, {self.inner} values normed in {self.norm_groups} parts")
+        if not 0 < N <= ops.delta_rule_max_dim():
+            raise ValueError(f"{N} states per value column; the recurrence takes up to {ops.delta_rule_max_dim()}")
+        matrix, vector = _named(spec, weights, runtime)
+        self.conv_channels = self.inner + 2 * G * N
+        self.inputs = _stacked_rows([matrix("in_proj", (2 * self.inner + 2 * G * N + H, hidden))], runtime)
+        self.conv = ShortConv(PartSpec("short_conv", {
+            "channels": self.conv_channels, "taps": int(spec["conv_taps"]), "weight": spec["conv_weight"],
+            "bias": spec["conv_bias"], "activation": "silu"}), weights, runtime)
+        self.step_bias = vector("step_bias", H)
+        self.rate = torch.exp(vector("a_log", H)).contiguous()
+        self.skip = vector("skip", H)
+        self.norm_weight = vector("norm", self.inner)
+        self.o = Linear(matrix("o_proj", (hidden, self.inner)), runtime)
+        self.dtype = runtime.dtype
+
+    def cache_need(self) -> CacheNeed:
+        return CacheNeed(kind="several", members=(
+            CacheNeed(kind="state", state_shape=(self.heads, self.vdim, self.states), state_dtype="float32"),
+            self.conv.cache_need()))
+
+    def parts(self):
+        return [self.conv]
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
+        if len(cache.members) != 2 or cache.members[0].state is None:
+            raise ValueError("the state-space mixer needs its two state entries of the cache")
+        rows = request_rows_of(ctx)
+        H, V, N, G, inner = self.heads, self.vdim, self.states, self.groups, self.inner
+        proj = self.inputs.forward(x)       # every later step reads column ranges of it in place
+        xbc = self.conv.forward(proj[:, inner:inner + self.conv_channels], ctx, cache.members[1])
+        at = inner + self.conv_channels
+        y = ops.state_space_dual(xbc, (inner + G * N, inner, 0), proj[:, at:at + H], self.step_bias, self.rate, self.skip,
+                                 cache.members[0].state, rows["row_start"], rows["row_length"], ctx.request_slots, H, G, N, V,
+                                 longest=rows.get("longest", 0))
+        return self.o.forward(ops.gated_norm(y, self.norm_weight, proj[:, :inner], self.norm_groups, self.eps, self.dtype))
+
+    def weight_bytes(self) -> int:
+        return self.inputs.weight_bytes() + self.o.weight_bytes()
+
+
+register_part("mixer", "state_space_dual", lambda spec, weights, runtime: StateSpaceDual(spec, weights, runtime))

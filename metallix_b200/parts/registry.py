@@ -4,7 +4,8 @@ A part is built from a ``PartSpec`` (kind + parameters), a ``WeightStore``
 (tensors by name) and a ``Runtime`` (device, compute dtype, capacity). It
 never learns which model it is in. Five categories exist: ``mixer``,
 ``feed_forward``, ``norm``, ``position`` and ``block``; plus ``embedding`` and
-``head`` at the model's two ends. Registering a new kind is one call::
+``head`` at the model's two ends, and ``join`` for what happens to the residual
+stream ahead of a layer run. Registering a new kind is one call::
 
     register_part("mixer", "my_mixer", lambda spec, weights, runtime: MyMixer(...))
 
@@ -19,7 +20,7 @@ import torch
 
 from ..config.spec import CacheNeed, PartSpec
 
-CATEGORIES = ("mixer", "feed_forward", "norm", "position", "block", "embedding", "head")
+CATEGORIES = ("mixer", "feed_forward", "norm", "position", "block", "embedding", "head", "join")
 _BUILDERS: Dict[Tuple[str, str], Callable] = {}
 
 

@@ -8,7 +8,7 @@ import torch
 
 from . import ops
 
-STORE_BF16, STORE_F32, SWIGLU, RELU_SQUARED, GEGLU = 0, 1, 2, 3, 4
+STORE_BF16, STORE_F32, SWIGLU, RELU_SQUARED, GEGLU, CLAMPED_GLU = 0, 1, 2, 3, 4, 5
 
 
 def why_not(a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype) -> str:
@@ -31,9 +31,10 @@ def supports(a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype) -> bool:
     return why_not(a, w, out_dtype) == ""
 
 
-def _launch(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, n: int, epilogue: int) -> torch.Tensor:
+def _launch(out: torch.Tensor, a: torch.Tensor, w: torch.Tensor, n: int, epilogue: int,
+            limit: float = 0.0) -> torch.Tensor:
     ops._call("mxb_gemm_tcgen05", out.data_ptr(), a.data_ptr(), w.data_ptr(), a.shape[0], n, a.shape[1],
-              a.stride(0), w.stride(0), out.stride(0), epilogue, ops.status_word(a.device).data_ptr(),
+              a.stride(0), w.stride(0), out.stride(0), epilogue, float(limit), ops.status_word(a.device).data_ptr(),
               ops._stream())
     return out
 
@@ -52,10 +53,10 @@ def gemm(a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype = torch.bfloat
 
 
 def gemm_swiglu(a: torch.Tensor, gate_up: torch.Tensor, out: Optional[torch.Tensor] = None,
-                activation: str = "silu") -> torch.Tensor:
+                activation: str = "silu", limit: float = 0.0) -> torch.Tensor:
     """act(a gate^T) * (a up^T) for gate_up = [gate rows; up rows], without
     gate and up ever reaching memory; act is silu or ("gelu_tanh") the tanh
-    form of gelu. Returns bfloat16 [m, inter]."""
+    form of gelu, or "clamped" with ``limit`` (ops.GATE_ACTIVATIONS). Returns bfloat16 [m, inter]."""
     reason = why_not(a, gate_up, torch.bfloat16)
     if reason:
         raise ops.KernelError("the tcgen05 kernel does not take this call: " + reason)
@@ -64,7 +65,7 @@ def gemm_swiglu(a: torch.Tensor, gate_up: torch.Tensor, out: Optional[torch.Tens
     if out is None:
         out = torch.empty((m, inter), dtype=torch.bfloat16, device=a.device)
     ops._need(out.shape == (m, inter) and out.dtype == torch.bfloat16 and out.stride(1) == 1, "out does not fit")
-    return _launch(out, a, gate_up, inter, {"silu": SWIGLU, "gelu_tanh": GEGLU}[activation])
+    return _launch(out, a, gate_up, inter, {"silu": SWIGLU, "gelu_tanh": GEGLU, "clamped": CLAMPED_GLU}[activation], limit)
 
 
 def gemm_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, groups: int, epilogue: int) -> torch.Tensor:
