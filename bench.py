@@ -9,6 +9,7 @@
     python bench.py --design zitezen                              the Zitezen decoder beside Qwen3 at equal width, heads and feed-forward
     python bench.py --design sadosun                              the Sadosun decoder beside Qwen3 and Zitezen at equal width and active weights
     python bench.py --design dimorax                              the Dimorax decoder beside Qwen3 and Sadosun at equal width and active weights
+    python bench.py --design kokolorn                             the Kokolorn decoder beside Qwen3 and Dimorax at equal width and active weights
 
 Default workload: a Qwen3-0.6B-shaped model (28 layers,
 hidden 1024, 16 query and 8 key/value heads of 128, SwiGLU 3072, vocabulary
@@ -669,6 +670,9 @@ def workload(args):
         elif args.design == "dimorax":   # its layers come in fours; a layer that reads another's keys has its source among them
             other = _dimorax(hidden, heads, kv_heads, dim, inter, {"0.6b": "0.6b-layers", "8b": "8b-layers"}[args.shape])
             config = parse_config(dict(other, layers=other["layers"][:4] if layers <= 4 else other["layers"][:layers]))
+        elif args.design == "kokolorn":   # all eight layer runs (two layers of them looped), or its first layers without the loop
+            other = _kokolorn(hidden, heads, kv_heads, dim, inter, {"0.6b": "0.6b-layers", "8b": "8b-layers"}[args.shape])
+            config = parse_config(other if layers >= DESIGN_LAYERS else dict(other, loop=None, layers=other["layers"][:layers]))
         elif args.design == "sadosun":   # its layers come in twos
             other = _sadosun(hidden, heads, kv_heads, dim, inter, {"0.6b": "0.6b-layers", "8b": "8b-layers"}[args.shape],
                              args.chunk or 4096)
@@ -1557,6 +1561,251 @@ def design_dimorax(args):
     return 0
 
 
+# Kokolorn layers at the two sizes: the delta rule's (heads, query/key groups, key channels, value columns, taps),
+# the state-space dual's (heads, value columns, states, groups, norm parts, taps), the experts' (count, top, ff) with a
+# shared expert of the same ff, so that (top + 1) * 2 matrices of ff = the dense model's 3 * inter; the distances'
+# biases (rows, far end). Six layers, of which the first two run twice: eight layer runs.
+KOKOLORN_SIZES = {"0.6b-layers": ((16, 8, 128, 128, 4), (32, 64, 128, 1, 1, 4), (12, 2, 1536), (32, 1024)),
+                  "8b-layers": ((32, 8, 128, 128, 4), (128, 64, 128, 1, 1, 4), (12, 2, 6144), (32, 1024))}
+
+
+def _kokolorn(hidden, heads, kv_heads, dim, inter, size):
+    (dh, dg, dd, dv, taps), (sh, sv, states, groups, parts, s_taps), (count, top, ff), (rows, far) = KOKOLORN_SIZES[size]
+    experts = {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": ff}, "router": {"experts": count, "top": top}}
+    dense = {"kind": "dense", "ff": inter, "limit": 7.0}
+    attention = {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                 "q_temp": {"coef": 0.1, "every": 4096}}
+    delta = {"heads": dh, "kv_heads": dg, "dim": dd, "vdim": dv, "conv": taps}
+    pair = {"left": dict(attention, bias_max=far, bias_rows=rows),
+            "right": {"heads": sh, "vdim": sv, "state": states, "groups": groups, "norm_groups": parts, "conv": s_taps}}
+    return {"architecture": "Kokolorn", "vocab": DESIGN_VOCAB, "width": hidden, "norm": {"eps": 1e-6},
+            "embedding": {"scale": hidden ** 0.5}, "loop": {"start": 0, "stop": 2, "times": 2},
+            "layers": [{"type": "attention", "mixer": attention, "mlp": dense}, {"type": "delta", "mixer": delta, "mlp": experts},
+                       {"type": "parallel", "mixer": pair, "mlp": experts}, {"type": "attention", "mixer": attention, "mlp": dense},
+                       {"type": "delta", "mixer": delta, "mlp": dense}, {"type": "parallel", "mixer": pair, "mlp": experts}]}
+
+
+def design_kokolorn(args):
+    """Prompt and decode throughput of the Kokolorn decoder beside the Qwen3
+    decoder (equal width, heads and active feed-forward weights) and the
+    Dimorax decoder (the other model with a delta rule, biased attention and
+    experts beside a shared one), random weights, bfloat16, 8 layer runs; then
+    each kernel the design adds beside the like kernel of those models: bytes
+    that must move over time against the measured copy bandwidth, or arithmetic
+    over time against the measured bf16 matrix peak. One JSON line."""
+    import numpy as np
+    import torch
+    from metallix_b200 import ops, parse_config
+    from metallix_b200.config.kokolorn import ChosenExperts
+    from metallix_b200.config.spec import PartSpec
+    from metallix_b200.parts.registry import Runtime, WeightStore, build_part
+
+    peak, peak_source = peaks()
+    warmup, steps = max(args.warmup, 3), min(max(args.steps, 1), 64)
+    rng = np.random.default_rng(0)
+    out = {"design": "kokolorn", "beside": ["qwen3", "dimorax"], "dtype": "bf16", "layers": DESIGN_LAYERS,
+           "vocab": DESIGN_VOCAB, "prompt_len": args.prompt_len, "peaks": peak_source, "sizes": {}}
+    for size, (hidden, heads, kv_heads, dim, inter) in ({} if args.kernels_only else DESIGN_SIZES).items():
+        configs = {"kokolorn": parse_config(_kokolorn(hidden, heads, kv_heads, dim, inter, size)),
+                   "qwen3": parse_config(dict(_qwen3(DESIGN_LAYERS, hidden, heads, kv_heads, inter, False),
+                                              vocab_size=DESIGN_VOCAB, head_dim=dim)),
+                   "dimorax": parse_config(_dimorax(hidden, heads, kv_heads, dim, inter, size))}
+        out["sizes"][size] = {family: _engine_numbers(config, args, peak, rng, warmup, steps)
+                              for family, config in configs.items()}
+
+    def measure(function):
+        for _ in range(3):
+            function()
+        flush = torch.empty(192 << 20, dtype=torch.uint8, device="cuda")
+        times = []
+        for _ in range(7):
+            flush.zero_()    # a buffer larger than L2 between the timed launches
+            times.append(timed(torch, "cuda", lambda _: function(), 1))
+        return statistics.median(times)
+
+    def gbs(bytes_moved, function):
+        ms = measure(function)
+        return {"us": ms * 1e3, "gb_s": bytes_moved / (ms * 1e-3) / 1e9,
+                "frac_of_copy_bandwidth": bytes_moved / (ms * 1e-3) / 1e9 / peak["hbm_gbs"]}
+
+    def tflops(flops, function):
+        ms = measure(function)
+        return {"us": ms * 1e3, "tflop_s": flops / (ms * 1e-3) / 1e12,
+                "frac_of_bf16_matrix_peak": flops / (ms * 1e-3) / 1e12 / peak["bf16_tflops"]}
+
+    ops.require_cuda()
+    kernels = {}
+    size = "8b-layers"
+    hidden, heads, kv_heads, dim, inter = DESIGN_SIZES[size]
+    (dh, dg, dd, dv, taps), (sh, sv, states, groups, parts, s_taps), (count, top, ff), (rows_of_table, far) = KOKOLORN_SIZES[size]
+    bf16, f32 = torch.bfloat16, torch.float32
+    ints = lambda values: torch.tensor(values, dtype=torch.int32, device="cuda")
+    normal = lambda *shape: torch.randn(*shape, device="cuda")
+    prompt = args.prompt_len
+    runtime = Runtime(device=torch.device("cuda"), dtype=bf16, max_positions=args.context, gemm_backend=args.gemm)
+
+    def weights_of(shapes):
+        return WeightStore({name: (normal(*shape) * 0.02).to(bf16) for name, shape in shapes.items()})
+
+    # ---- the residual stream: two outputs behind norms of their own, what a pass's product reads, a vector for all rows
+    inner, ones = sh * sv, torch.ones(hidden, device="cuda")
+    for tokens in (8, prompt * 4):
+        x, a, b, row = normal(tokens, hidden), normal(tokens, hidden).to(bf16), normal(tokens, hidden).to(bf16), normal(hidden)
+        kernels[f"sublayer_input_{tokens}"] = {
+            "kokolorn: x += norm(a + bias) / 2 + norm(b) / 2; y = norm(x)": gbs(
+                tokens * hidden * (4 + 4 + 2 + 2 + 2),
+                lambda: ops.pair_norm(x, a, b, ones, ones, 1e-6, 1e-6, 0.5, 0.5, left_bias=row, weight=ones, eps=1e-6,
+                                      out_dtype=bf16)),
+            "dimorax: x += m (a + b); two norms of x": gbs(
+                tokens * hidden * (4 + 4 + 2 + 2 + 2 + 2), lambda: ops.pair_add_rmsnorm(x, a, b, 0.5, ones, ones, 1e-6, bf16)),
+            "qwen3: x += d; y = norm(x)": gbs(tokens * hidden * (4 + 4 + 2 + 2), lambda: ops.add_rmsnorm(x, a, ones, 1e-6, bf16)),
+            "kokolorn: [x + d | x0] rounded": gbs(tokens * hidden * (4 + 2 + 4 + 4), lambda: ops.join_rows(x, a, x, bf16)),
+            "kokolorn: x += row; y = norm(x)": gbs(tokens * hidden * (4 + 4 + 2), lambda: ops.add_rmsnorm(x, row, ones, 1e-6, bf16))}
+        wide, product = normal(tokens, inner), normal(tokens, 2 * inner).to(bf16)
+        weight = torch.ones(inner, device="cuda")
+        kernels[f"recurrent_output_{tokens}"] = {
+            "kokolorn: x silu(gate), then its norm (%d values)" % inner: gbs(
+                tokens * inner * (4 + 2 + 2), lambda: ops.gated_norm(wide, weight, product[:, :inner], parts, 1e-6, bf16)),
+            "kokolorn: each head's norm, times silu(gate)": gbs(
+                tokens * inner * (4 + 2 + 2), lambda: ops.head_norm_gate(wide, weight, product[:, :inner], inner // dv, 1e-6,
+                                                                       bf16, activation="silu")),
+            "dimorax: each head's norm, times sigmoid(gate)": gbs(
+                tokens * inner * (4 + 2 + 2), lambda: ops.head_norm_gate(wide, weight, product[:, :inner], inner // dv, 1e-6, bf16))}
+        q_width, k_width = heads * dim, kv_heads * dim
+        pages = -(-tokens // 16)
+        qk, pool = normal(tokens, q_width + k_width).to(bf16), torch.zeros(pages, 2, kv_heads, 16, dim, dtype=bf16, device="cuda")
+        q_out, at = torch.empty(tokens, heads, dim, dtype=bf16, device="cuda"), torch.arange(tokens, dtype=torch.int32, device="cuda")
+        gain, factors = torch.ones(dim, device="cuda"), torch.ones(max(tokens, 8), device="cuda")
+        table = torch.ones(max(tokens, 8), dim // 2, device="cuda")
+        moved = tokens * (2 * q_width + 4 * k_width) * 2
+        keys = qk[:, q_width:]
+        kernels[f"queries_and_cache_{tokens}"] = {
+            "kokolorn: norms, query factors, keys and raw keys into the cache": gbs(
+                moved, lambda: ops.qk_norm_rope_cache(qk[:, :q_width], keys, keys, q_out, pool, at, at, gain, gain, None, None,
+                                                      1e-6, q_factors=factors)),
+            "qwen3: norms, rotation, keys and values into the cache": gbs(
+                moved + tokens * dim * 4, lambda: ops.qk_norm_rope_cache(qk[:, :q_width], keys, keys, q_out, pool, at, at, gain,
+                                                                         gain, table, table, 1e-6))}
+        del pool, qk, q_out
+
+    # ---- the feed-forward: experts weighed by the softmax over the chosen, with a shared one, beside Dimorax's gated
+    # ones and the dense one
+    typed = ChosenExperts(ff=ff, experts=count, top=top, shared_ff=ff)
+    chosen_experts = build_part("feed_forward", typed.part("m", hidden), weights_of(typed.shapes("m", hidden)), runtime)
+    (_, _, (d_count, d_groups, d_keep, d_top, d_ff)) = DIMORAX_SIZES[size]
+    names = {f"m.e{e}.{which}": (hidden, d_ff) if which == "down" else (d_ff, hidden) for e in range(d_count)
+             for which in ("gate", "up", "down")}
+    names.update({"m.router": (d_count, hidden), "m.shared.gate": (d_ff, hidden), "m.shared.up": (d_ff, hidden),
+                  "m.shared.down": (hidden, d_ff), "m.shared.sg": (1, hidden)})
+    store = weights_of(names)
+    store._tensors["m.correction"] = torch.zeros(d_count, device="cuda")
+    gated = build_part("feed_forward", PartSpec("routed_experts", {
+        "hidden_size": hidden, "intermediate_size": d_ff, "experts": d_count, "identity": 0, "top": d_top, "activation": "swiglu",
+        "scores": "sigmoid", "scale": 2.0, "groups": (d_groups, d_keep), "gate_proj": "m.e{}.gate", "up_proj": "m.e{}.up",
+        "down_proj": "m.e{}.down", "router": "m.router", "correction": "m.correction", "shared_gate": "m.shared.sg",
+        "shared": PartSpec("swiglu", {"hidden_size": hidden, "intermediate_size": d_ff, "gate_proj": "m.shared.gate",
+                                      "up_proj": "m.shared.up", "down_proj": "m.shared.down", "activation": "silu"})}),
+        store, runtime)
+    dense = {act: build_part("feed_forward", PartSpec("swiglu", {
+        "hidden_size": hidden, "intermediate_size": inter, "gate_proj": "g", "up_proj": "u", "down_proj": "d",
+        "activation": act, "limit": 7.0}), weights_of({"g": (inter, hidden), "u": (inter, hidden), "d": (hidden, inter)}), runtime)
+        for act in ("silu", "clamped")}
+    del store
+    for tokens in (8, prompt * 4):
+        h = normal(tokens, hidden).to(bf16)
+        logits = chosen_experts.router.forward(h, out_dtype=f32)
+        picked = ops.route_experts(logits[:, :count], chosen_experts.correction, count, top, scores="chosen")[0]
+        distinct = int(torch.unique(picked).numel())
+        logits = gated.router.forward(h, out_dtype=f32)
+        picked = ops.route_experts(logits[:, :d_count], gated.correction, d_count, d_top, scores="sigmoid",
+                                   groups=(d_groups, d_keep))[0]
+        d_distinct = int(torch.unique(picked).numel())
+        label = f"feed_forward_{tokens}"
+        if tokens == 8:     # a decode step: the weights that must be read
+            kernels[label] = {
+                "kokolorn: router, choice, %d distinct experts of %d, the shared one" % (distinct, count): gbs(
+                    (distinct + 1) * 2 * ff * hidden * 2 + count * hidden * 2, lambda: chosen_experts.forward(h, None)),
+                "dimorax: router, choice, %d distinct gated experts of %d, the shared one" % (d_distinct, d_count): gbs(
+                    (d_distinct + 1) * 3 * d_ff * hidden * 2 + (d_count + 1) * hidden * 2, lambda: gated.forward(h, None)),
+                "qwen3: gate, up, silu, down": gbs(3 * inter * hidden * 2, lambda: dense["silu"].forward(h, None)),
+                "kokolorn: gate, up, clamped, down": gbs(3 * inter * hidden * 2, lambda: dense["clamped"].forward(h, None))}
+        else:               # a prompt: the products that must be made
+            kernels[label] = {
+                "kokolorn: router, choice, the chosen experts, the shared one": tflops(
+                    (top + 1) * tokens * 4.0 * ff * hidden + tokens * 2.0 * count * hidden, lambda: chosen_experts.forward(h, None)),
+                "dimorax: router, choice, the chosen gated experts, the shared one": tflops(
+                    (d_top + 1) * tokens * 6.0 * d_ff * hidden + tokens * 2.0 * (d_count + 1) * hidden, lambda: gated.forward(h, None)),
+                "qwen3: gate, up, silu, down": tflops(tokens * 6.0 * inter * hidden, lambda: dense["silu"].forward(h, None)),
+                "kokolorn: gate, up, clamped, down": tflops(tokens * 6.0 * inter * hidden, lambda: dense["clamped"].forward(h, None))}
+    del chosen_experts, gated, dense
+
+    # ---- the mixers: a decode step of 8 requests, then a prompt in one step
+    (ch, cg, cd, cv, _, _), _, _ = DIMORAX_SIZES[size]
+    per_channel, c_bias, c_rate = ch * cd, normal(ch * cd) - 3.0, torch.exp(normal(ch) * 0.3)
+    h_bias, h_rate = normal(dh) - 3.0, torch.exp(normal(dh) * 0.3)
+    s_bias, s_rate, skip = normal(sh) - 3.0, torch.exp(normal(sh) * 0.3), normal(sh)
+    biases = normal(heads, far + 1)
+    states_of = lambda slots: (torch.zeros(slots, dh, dv, dd, device="cuda"), torch.zeros(slots, ch, cv, cd, device="cuda"),
+                               torch.zeros(slots, sh, sv, states, device="cuda"))
+
+    def recurrences(tokens, rows, lengths, slots, longest):
+        """(name, bytes of rows, bytes of state, call) of the three recurrences."""
+        h_state, c_state, s_state = states_of(rows.numel())
+        h_in, h_side = normal(tokens, 2 * dg * dd + dh * dv).to(bf16), normal(tokens, 2 * dh).to(bf16)
+        c_in, c_side, c_step = normal(tokens, 2 * cg * cd + ch * cv).to(bf16), normal(tokens, ch).to(bf16), normal(tokens, per_channel)
+        s_in, s_side = normal(tokens, 2 * groups * states + sh * sv).to(bf16), normal(tokens, sh).to(bf16)
+        return [
+            ("kokolorn: delta rule, a decay per head", tokens * (h_in.shape[1] * 2 + 2 * dh * 2 + dh * dv * 4), 2 * h_state.numel() * 4,
+             lambda: ops.delta_rule(h_in, (0, dg * dd, 2 * dg * dd), h_side[:, :dh], h_side[:, dh:], h_bias, h_rate, h_state, rows,
+                                    lengths, slots, dh, dg, dd, dv, longest=longest, decay="head")),
+            ("dimorax: delta rule, a decay per head and channel",
+             tokens * (c_in.shape[1] * 2 + ch * 2 + per_channel * 4 + ch * cv * 4), 2 * c_state.numel() * 4,
+             lambda: ops.delta_rule(c_in, (0, cg * cd, 2 * cg * cd), c_side, c_step, c_bias, c_rate, c_state, rows, lengths, slots,
+                                    ch, cg, cd, cv, longest=longest)),
+            ("kokolorn: state-space dual, %d heads of %d, %d states" % (sh, sv, states),
+             tokens * (s_in.shape[1] * 2 + sh * 2 + sh * sv * 4), 2 * s_state.numel() * 4,
+             lambda: ops.state_space_dual(s_in, (sh * sv + groups * states, sh * sv, 0), s_side, s_bias, s_rate, skip, s_state, rows,
+                                          lengths, slots, sh, groups, states, sv, longest=longest))]
+
+    batch, context = 8, prompt
+    rows, one_each = ints(range(batch)), ints([1] * batch)
+    label = "decode_step_mixer_8_requests"
+    kernels[label] = {name + ", state read and written": gbs(state, call)
+                      for name, _, state, call in recurrences(batch, rows, one_each, rows, 1)}
+    pages = batch * (-(-context // 16))
+    table = torch.arange(pages, dtype=torch.int32, device="cuda").view(batch, -1)
+    positions = ints([context - 1] * batch)
+    cache = normal(pages, 2, kv_heads, 16, dim).to(bf16)
+    q = normal(batch, heads, dim).to(bf16)
+    attended = torch.empty_like(q)
+    for name, bias in (("qwen3: split-key attention over %d cached positions" % context, None),
+                       ("kokolorn: the same with a bias per head and distance", biases)):
+        kernels[label][name] = gbs(cache.numel() * 2, lambda: ops.paged_attention_decode(
+            q, cache, attended, table, rows, rows, positions, dim ** -0.5, context, bias=bias))
+
+    tokens, label = prompt, f"prompt_mixer_{prompt}"
+    one_row, length = ints([0]), ints([tokens])
+    kernels[label] = {name + ", one request (rows read and written)": gbs(moved, call)
+                      for name, moved, _, call in recurrences(tokens, one_row, length, one_row, tokens)}
+    pages = -(-tokens // 16)
+    table = torch.arange(pages, dtype=torch.int32, device="cuda").view(1, -1)
+    positions = torch.arange(tokens, dtype=torch.int32, device="cuda")
+    cache = normal(pages, 2, kv_heads, 16, dim).to(bf16)
+    q = normal(tokens, heads, dim).to(bf16)
+    attended = torch.empty_like(q)
+    flops = 4.0 * dim * heads * tokens * (tokens + 1) / 2
+    tile = ops.flash_prefill_tile()
+    starts = list(range(0, tokens, tile))[::-1]
+    tiles = (ints([0] * len(starts)), ints(starts), ints([min(tile, tokens - s) for s in starts]))
+    for name, bias in (("qwen3: tensor-core attention", None), ("kokolorn: the same with a bias per head and distance", biases)):
+        kernels[label][name] = tflops(flops, lambda: ops.flash_prefill(
+            q, cache, attended, table, *tiles, positions, dim ** -0.5, longest_context=tokens, bias=bias))
+    ops.check_status("cuda")
+    out["kernels"] = kernels
+    print(json.dumps(out))
+    return 0
+
+
 def main():
     parser = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
     parser.add_argument("--gpus", type=int, default=1)
@@ -1595,7 +1844,7 @@ def main():
     parser.add_argument("--kernel", default="both", choices=("both", "tcgen05", "mma"))
     parser.add_argument("--page-tokens", type=int, default=16, help="workloads: tokens per cache page")
     parser.add_argument("--max-context", type=int, default=0, help="workloads: the engine's context limit")
-    parser.add_argument("--design", choices=("mekazen", "zitezen", "sadosun", "dimorax"),
+    parser.add_argument("--design", choices=("mekazen", "zitezen", "sadosun", "dimorax", "kokolorn"),
                         help="another decoder design beside Qwen3 at equal layer sizes, and its kernels beside their like")
     parser.add_argument("--chunk", type=int, default=0, help="--design: positions per chunk of the mask (0: the context)")
     parser.add_argument("--kernels-only", action="store_true",
@@ -1617,6 +1866,8 @@ def main():
         return design_sadosun(args)
     if args.design == "dimorax" and not args.workload:
         return design_dimorax(args)
+    if args.design == "kokolorn" and not args.workload:
+        return design_kokolorn(args)
     if args.design and not args.workload:
         return design(args)
     if args.workload:

@@ -12,6 +12,9 @@
 // their scores are tiny beside it, the float32 sum would round the scores
 // away and leave the choice to the tie rule instead of to the scores. The
 // last `identity` outputs stand for experts that return their input.
+// Behind its `top` choices a token may have `always` more that no router decides: the
+// experts with the indices experts, experts + 1, ... with weight 1 (only where
+// there are no identity outputs).
 // route_kernel leaves, per token, the chosen indices and weights, a dense row
 // of weights over the real experts (zeros for those not chosen) and the sum of
 // the weights that fell on identity experts.
@@ -43,7 +46,7 @@ __global__ void __launch_bounds__(kRouteThreads)
 route_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int* __restrict__ chosen,
              float* __restrict__ weights, float* __restrict__ dense, float* __restrict__ identity_weight,
              int tokens, int outputs, int experts, int top, int scores, int group_count, int group_keep,
-             float weight_scale, long long ld) {
+             float weight_scale, long long ld, int always) {
   extern __shared__ double shared[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * (kRouteThreads / 32) + warp;
@@ -124,6 +127,7 @@ route_kernel(const float* __restrict__ logits, const float* __restrict__ correct
       if (!isnan(group_score[r / size])) choice[r] = -INFINITY;
     __syncwarp();
   }
+  const int choices = top + always;     // of a token, in chosen and weights
   float picked_sum = 0.0f;
   for (int k = 0; k < top; ++k) {
     double best = -INFINITY;
@@ -140,7 +144,7 @@ route_kernel(const float* __restrict__ logits, const float* __restrict__ correct
     }
     if (where >= outputs) where = k < outputs ? k : 0;   // nothing comparable left (non-finite logits)
     if (lane == 0) {
-      chosen[static_cast<size_t>(t) * top + k] = where;
+      chosen[static_cast<size_t>(t) * choices + k] = where;
       choice[where] = -INFINITY;
     }
     picked_sum += score[where];
@@ -150,11 +154,15 @@ route_kernel(const float* __restrict__ logits, const float* __restrict__ correct
   if (lane == 0) {
     float on_identity = 0.0f;
     for (int k = 0; k < top; ++k) {
-      const int where = chosen[static_cast<size_t>(t) * top + k];
+      const int where = chosen[static_cast<size_t>(t) * choices + k];
       const float w = score[where] * scale;
-      weights[static_cast<size_t>(t) * top + k] = w;
+      weights[static_cast<size_t>(t) * choices + k] = w;
       if (where < experts) dense[static_cast<size_t>(t) * experts + where] = w;
       else on_identity += w;
+    }
+    for (int k = top; k < choices; ++k) {
+      chosen[static_cast<size_t>(t) * choices + k] = experts + k - top;
+      weights[static_cast<size_t>(t) * choices + k] = 1.0f;
     }
     identity_weight[t] = on_identity;
   }
@@ -351,15 +359,16 @@ routed_down_kernel(const float* __restrict__ act, const T* __restrict__ w_down, 
 
 using namespace mxb;
 
-// logits: float32 [tokens, outputs]; correction: float32 [outputs]; chosen: int32 [tokens, top];
-// weights: float32 [tokens, top]; dense: float32 [tokens, experts]; identity_weight: float32 [tokens].
+// logits: float32 [tokens, outputs]; correction: float32 [outputs]; chosen: int32 [tokens, top + always];
+// weights: float32 [tokens, top + always]; dense: float32 [tokens, experts]; identity_weight: float32 [tokens].
 // scores: 0 s = softmax(z), 1 s = sigmoid(z), 2 z + correction chooses and the softmax over the chosen weighs. group_count > 1: the outputs form that many equal groups of
 // neighbours, and only outputs of the group_keep best groups can be chosen. weight_scale multiplies the weights.
 MXB_API int mxb_route_experts(const float* logits, const float* correction, int* chosen, float* weights, float* dense,
                               float* identity_weight, int tokens, int outputs, int experts, int top,
                               int scores, int group_count, int group_keep, float weight_scale,
-                              long long ld, cudaStream_t stream) {
+                              long long ld, int always, cudaStream_t stream) {
   if (tokens <= 0) return 0;
+  if (always < 0 || (always > 0 && experts != outputs)) return static_cast<int>(cudaErrorInvalidValue);
   if (scores < kScoreSoftmax || scores > kScoreChosen) return static_cast<int>(cudaErrorInvalidValue);
   if (outputs <= 0 || experts < 0 || experts > outputs || top <= 0 || top > outputs)
     return static_cast<int>(cudaErrorInvalidValue);
@@ -371,7 +380,7 @@ MXB_API int mxb_route_experts(const float* logits, const float* correction, int*
   if (shared > 48 * 1024) return static_cast<int>(cudaErrorInvalidValue);
   route_kernel<<<ceil_div(tokens, kRouteThreads / 32), kRouteThreads, shared, stream>>>(
       logits, correction, chosen, weights, dense, identity_weight, tokens, outputs, experts, top, scores,
-      group_count, group_keep, weight_scale, ld < outputs ? outputs : ld);
+      group_count, group_keep, weight_scale, ld < outputs ? outputs : ld, always);
   return static_cast<int>(cudaGetLastError());
 }
 

@@ -40,7 +40,7 @@ _SIGNATURES = {
     "mxb_short_conv": [_P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "mxb_selective_scan": [_P, _L, _P, _L, _P, _P, _P, _P, _L, _P, _P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I,
                            _I, _P, _P],
-    "mxb_route_experts": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _L, _P],
+    "mxb_route_experts": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _L, _I, _P],
     "mxb_expert_rows": [_P, _P, _P, _I, _I, _I, _P],
     "mxb_expert_rows_tile": [],
     "mxb_expert_rows_experts": [],
@@ -680,12 +680,14 @@ ROUTER_OUTPUTS = 1024   # the most router outputs the routing kernel keeps in sh
 
 
 def route_experts(logits: torch.Tensor, correction: torch.Tensor, experts: int, top: int, scores: str = "softmax",
-                  groups: Optional[tuple] = None, scale: float = 1.0):
+                  groups: Optional[tuple] = None, scale: float = 1.0, always: int = 0):
     """Scores over all router outputs (``scores``: "softmax" over the row, or
     "sigmoid" of each logit on its own), the ``top`` largest score + correction
     chosen, weights = the chosen scores over their sum, times ``scale``. With
     "chosen" the ``top`` largest logit + correction (a bias of the router's) are
-    chosen and their weights are the softmax over these sums alone.
+    chosen and their weights are the softmax over these sums alone. ``always``: that
+    many choices more per token, the experts from index ``experts`` on with weight
+    1 (not beside identity outputs).
     ``groups`` = (count, keep): the outputs form ``count`` equal groups of
     neighbours and only outputs of the ``keep`` groups with the largest sum of
     their two largest score + correction can be chosen. ``logits`` is float32
@@ -706,13 +708,14 @@ def route_experts(logits: torch.Tensor, correction: torch.Tensor, experts: int, 
         _need(outputs % count == 0 and 1 <= keep <= count and keep * (outputs // count) >= top
               and outputs <= ROUTER_OUTPUTS // 2, "the router's groups do not fit")
     device = logits.device
-    chosen = torch.empty((tokens, top), dtype=torch.int32, device=device)
-    weights = torch.empty((tokens, top), dtype=torch.float32, device=device)
+    _need(always >= 0 and (always == 0 or experts == outputs), "experts for every token beside identity outputs")
+    chosen = torch.empty((tokens, top + always), dtype=torch.int32, device=device)
+    weights = torch.empty((tokens, top + always), dtype=torch.float32, device=device)
     dense = torch.empty((tokens, experts), dtype=torch.float32, device=device)
     on_identity = torch.empty((tokens,), dtype=torch.float32, device=device)
     _call("mxb_route_experts", logits.data_ptr(), correction.data_ptr(), chosen.data_ptr(), weights.data_ptr(),
           dense.data_ptr(), on_identity.data_ptr(), tokens, outputs, experts, top, ROUTE_SCORES[scores],
-          count, keep, float(scale), logits.stride(0), _stream())
+          count, keep, float(scale), logits.stride(0), int(always), _stream())
     return chosen, weights, dense, on_identity
 
 

@@ -141,9 +141,19 @@ class RoutedExperts:
             count, keep = self.groups
             if count < 1 or outputs % count or not 1 <= keep <= count or keep * (outputs // count) < self.top:
                 raise ValueError(f"{count} groups of which {keep} are kept do not fit {outputs} outputs and top {self.top}")
+        # A shared expert without a gate that looks like the others is one more of them, chosen by every token with
+        # weight 1: its work then rides in the same launches.
+        shared = spec.get("shared")
+        self.always = int(shared is not None and spec.get("shared_gate") is None and self.identity == 0 and not self.gated
+                          and shared.kind == "dense_ff" and shared["activation"] == spec["activation"]
+                          and shared["intermediate_size"] == ff)
+        names = [(spec["up_proj"].format(index), spec["down_proj"].format(index)) for index in range(self.experts)]
+        if self.always:
+            names.append((shared["up_proj"], shared["down_proj"]))
+        self.stacked = len(names)
         ups, downs = [], []
-        for index in range(self.experts):
-            up, down = weights.take(spec["up_proj"].format(index)), weights.take(spec["down_proj"].format(index))
+        for index, (up_name, down_name) in enumerate(names):
+            up, down = weights.take(up_name), weights.take(down_name)
             if tuple(up.shape) != (ff, hidden) or tuple(down.shape) != (hidden, ff):
                 raise ValueError(f"expert {index}: up is {tuple(up.shape)}, down is {tuple(down.shape)}; "
                                  f"expected {(ff, hidden)} and {(hidden, ff)}")
@@ -163,10 +173,10 @@ class RoutedExperts:
             raise ValueError(f"{spec['router']} is {tuple(router.shape)}, expected {(outputs, hidden)}")
         self.outputs = outputs
         self.shared = None
-        if spec.get("shared") is not None:
+        if shared is not None and not self.always:
             # an expert for every token, out += sigmoid(h . w) shared(h): its gate's row rides under the router's;
             # without a gate, out += shared(h)
-            self.shared = build_part("feed_forward", spec["shared"], weights, runtime)
+            self.shared = build_part("feed_forward", shared, weights, runtime)
         self.shared_gated = self.shared is not None and spec.get("shared_gate") is not None
         if self.shared_gated:
             gate = weights.take(spec["shared_gate"])
@@ -195,17 +205,17 @@ class RoutedExperts:
     def _routed(self, x: torch.Tensor, logits: torch.Tensor) -> torch.Tensor:
         chosen, weights, dense, on_identity = ops.route_experts(logits, self.correction, self.experts, self.top,
                                                                 scores=self.scores, groups=self.groups,
-                                                                scale=self.weight_scale)
+                                                                scale=self.weight_scale, always=self.always)
         if self.up is None:     # identity experts only
             return ops.experts_add_identity(torch.zeros(x.shape, dtype=torch.float32, device=x.device), x, on_identity)
         if x.shape[0] > self.ROUTED_TOKENS and self.grouped(x):
             from .. import tensor_core
-            position, tile_group, rows = ops.expert_rows(chosen, self.experts)
+            position, tile_group, rows = ops.expert_rows(chosen, self.stacked)
             act = tensor_core.gemm_grouped(ops.expert_gather_rows(x, position, rows), self.up.weight, tile_group,
-                                           self.experts, tensor_core.SWIGLU if self.gated else tensor_core.RELU_SQUARED)
-            out = tensor_core.gemm_grouped(act, self.down.weight, tile_group, self.experts, tensor_core.STORE_F32)
+                                           self.stacked, tensor_core.SWIGLU if self.gated else tensor_core.RELU_SQUARED)
+            out = tensor_core.gemm_grouped(act, self.down.weight, tile_group, self.stacked, tensor_core.STORE_F32)
             return ops.expert_combine_rows(out, position, weights, on_identity, x)
-        return ops.experts_routed(x, self.up.weight, self.down.weight, chosen, weights, self.experts,
+        return ops.experts_routed(x, self.up.weight, self.down.weight, chosen, weights, self.stacked,
                                   self.intermediate_size, gated=self.gated)
 
     def grouped(self, x: torch.Tensor) -> bool:
@@ -216,9 +226,9 @@ class RoutedExperts:
 
     def weight_bytes(self) -> int:
         """What a decode step of one token reads: the router and ``top`` experts."""
-        per_expert = (self.up.weight_bytes() + self.down.weight_bytes()) // self.experts if self.up is not None else 0
+        per_expert = (self.up.weight_bytes() + self.down.weight_bytes()) // self.stacked if self.up is not None else 0
         shared = self.shared.weight_bytes() if self.shared is not None else 0
-        return self.router.weight_bytes() + min(self.top, self.experts) * per_expert + shared
+        return self.router.weight_bytes() + (min(self.top, self.experts) + self.always) * per_expert + shared
 
 
 register_part("feed_forward", "routed_experts", lambda spec, weights, runtime: RoutedExperts(spec, weights, runtime))
