@@ -43,12 +43,13 @@ constexpr int kDeltaMaxWarps = 8;     // tokens of a batch: one warp prepares ea
 template <int DPT>
 __device__ __forceinline__ int delta_slot(int d) { return d + (d / DPT) * 4; }
 
+template <typename T> struct alignas(4 * sizeof(T)) DeltaFour { T v[4]; };   // four neighbouring values, one access
 __device__ __forceinline__ float delta_softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 
 // LANES lanes share a value column, each with DPT of its key channels; COLS neighbouring columns a thread.
 // MODE: see DeltaMode; `step_pre` is float32 [.., heads * dim] with a decay per channel, else of T with one value per head.
 template <typename T, int DPT, int LANES, int COLS, int MODE>
-__global__ void __launch_bounds__(512)
+__global__ void __launch_bounds__(MODE == kDeltaDual ? 256 : 512)   // four columns a thread want more registers each
 delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off, int v_off,
                   const T* __restrict__ beta_pre, long long ldb, int b_off,
                   const void* __restrict__ step_pre, long long lds, const float* __restrict__ step_bias,
@@ -98,15 +99,35 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
   // In memory a column's channels lie side by side ([heads, vdim, dim]): a lane's share is one run of DPT values.
   float* column_state = state + static_cast<long long>(slot) * slot_stride +
                         (static_cast<long long>(head) * vdim + column) * dim + part * DPT;
+  // shares that are whole and start on 16-byte boundaries move as vectors
+  const bool whole = dim % DPT == 0 && slot_stride % 4 == 0 && (reinterpret_cast<uintptr_t>(state) & 15) == 0;
+  if (whole) {
 #pragma unroll
-  for (int i = 0; i < DPT; ++i) {
-    const int d = part * DPT + i;
+    for (int c = 0; c < COLS; ++c)
 #pragma unroll
-    for (int c = 0; c < COLS; ++c) s[c][i] = live[c] && d < dim ? column_state[static_cast<long long>(c) * dim + i] : 0.0f;
+      for (int i = 0; i < DPT; i += 4) {
+        const float4 q = live[c] && part * DPT < dim
+                             ? *reinterpret_cast<const float4*>(column_state + static_cast<long long>(c) * dim + i)
+                             : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+        s[c][i] = q.x; s[c][i + 1] = q.y; s[c][i + 2] = q.z; s[c][i + 3] = q.w;
+      }
+  } else {
+#pragma unroll
+    for (int i = 0; i < DPT; ++i) {
+      const int d = part * DPT + i;
+#pragma unroll
+      for (int c = 0; c < COLS; ++c) s[c][i] = live[c] && d < dim ? column_state[static_cast<long long>(c) * dim + i] : 0.0f;
+    }
   }
   // What the next batch needs from memory, asked for a batch ahead: the raw q, k and step size of the token
   // this warp prepares, its write strength, and this thread's value of every token of the batch.
-  float raw_q[NL], raw_k[NL], raw_step[NL], raw_beta = 0.0f, next_v[kDeltaMaxWarps][COLS];
+  // Everything stays as it was loaded until it is used: a conversion here would wait for the load.
+  const T none = from_float<T>(0.0f);
+  T raw_q[NL], raw_k[NL], raw_head_step = none, raw_beta = none, next_v[kDeltaMaxWarps][COLS];
+  float raw_step[PER_CHANNEL ? NL : 1];
+  // whether four neighbouring columns of a token's values are one access (a block's first column is a multiple of four)
+  const bool v_vectors = COLS == 4 && vdim % 4 == 0 && v_off % 4 == 0 && ld % 4 == 0 &&
+                         (reinterpret_cast<uintptr_t>(qkv) & (4 * sizeof(T) - 1)) == 0;
   auto fetch = [&](int base) {
     const int batch = min(warps, length - base);
     if (warp < batch) {
@@ -117,30 +138,38 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
 #pragma unroll
       for (int i = 0; i < NL; ++i) {
         const int d = lane + 32 * i;
-        raw_q[i] = d < dim ? to_float(q_row[d]) : 0.0f;
-        raw_k[i] = d < dim ? to_float(k_row[d]) : 0.0f;
-        if (PER_CHANNEL) raw_step[i] = d < dim ? step_row[d] : 0.0f;
+        raw_q[i] = d < dim ? q_row[d] : none;
+        raw_k[i] = d < dim ? k_row[d] : none;
+        if (PER_CHANNEL) raw_step[PER_CHANNEL ? i : 0] = d < dim ? step_row[d] : 0.0f;
       }
-      if (!PER_CHANNEL) raw_step[0] = to_float(static_cast<const T*>(step_pre)[t * lds + head]);
-      if (MODE != kDeltaDual) raw_beta = to_float(beta_pre[t * ldb + b_off + head]);
+      if (!PER_CHANNEL) raw_head_step = static_cast<const T*>(step_pre)[t * lds + head];
+      if (MODE != kDeltaDual) raw_beta = beta_pre[t * ldb + b_off + head];
     }
+    const T* v_rows = qkv + (static_cast<long long>(first + base)) * ld + v_off + head * vdim + column;
 #pragma unroll
-    for (int j = 0; j < kDeltaMaxWarps; ++j)
+    for (int j = 0; j < kDeltaMaxWarps; ++j) {
+      if (COLS == 4 && v_vectors) {
+        DeltaFour<T> four = {{none, none, none, none}};
+        if (live[0] && j < batch) four = *reinterpret_cast<const DeltaFour<T>*>(v_rows + j * ld);
 #pragma unroll
-      for (int c = 0; c < COLS; ++c)
-        next_v[j][c] = live[c] && j < batch
-                           ? to_float(qkv[(static_cast<long long>(first + base + j)) * ld + v_off + head * vdim + column + c])
-                           : 0.0f;
+        for (int c = 0; c < COLS; ++c) next_v[j][c] = four.v[c];
+      } else {
+#pragma unroll
+        for (int c = 0; c < COLS; ++c) next_v[j][c] = live[c] && j < batch ? v_rows[j * ld + c] : none;
+      }
+    }
   };
   fetch(0);
   for (int base = 0; base < length; base += warps) {
     const int batch = min(warps, length - base);
     __syncthreads();   // the batch before this one has been read
     if (warp < batch) {   // unit norms, decay, write strength and qn . kn of this warp's token, from what was fetched
-      float qq = 0.0f, kk = 0.0f, qk = 0.0f;
+      float qq = 0.0f, kk = 0.0f, qk = 0.0f, q_in[NL], k_in[NL];
 #pragma unroll
       for (int i = 0; i < NL; ++i) {
-        qq = fmaf(raw_q[i], raw_q[i], qq); kk = fmaf(raw_k[i], raw_k[i], kk); qk = fmaf(raw_q[i], raw_k[i], qk);
+        q_in[i] = to_float(raw_q[i]);
+        k_in[i] = to_float(raw_k[i]);
+        qq = fmaf(q_in[i], q_in[i], qq); kk = fmaf(k_in[i], k_in[i], kk); qk = fmaf(q_in[i], k_in[i], qk);
       }
       qk = warp_sum(qk);
       float q_unit = 1.0f, k_unit = 1.0f;
@@ -154,15 +183,15 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
         const int d = lane + 32 * i;
         if (d < dim) {
           const int at = delta_slot<DPT>(d);
-          s_q[warp][at] = raw_q[i] * q_unit;
-          s_k[warp][at] = raw_k[i] * k_unit;
-          if (PER_CHANNEL) s_g[warp][at] = expf(-head_rate * delta_softplus(raw_step[i] + bias[i]));
+          s_q[warp][at] = q_in[i] * q_unit;
+          s_k[warp][at] = k_in[i] * k_unit;
+          if (PER_CHANNEL) s_g[warp][at] = expf(-head_rate * delta_softplus(raw_step[PER_CHANNEL ? i : 0] + bias[i]));
         }
       }
       if (lane == 0) {
-        const float step = PER_CHANNEL ? 0.0f : delta_softplus(raw_step[0] + bias[0]);
+        const float step = PER_CHANNEL ? 0.0f : delta_softplus(to_float(raw_head_step) + bias[0]);
         if (!PER_CHANNEL) s_decay[warp] = expf(-head_rate * step);
-        s_beta[warp] = MODE == kDeltaDual ? step : sigmoid_of(raw_beta);
+        s_beta[warp] = MODE == kDeltaDual ? step : sigmoid_of(to_float(raw_beta));
         s_qk[warp] = qk * q_unit * k_unit;
       }
     }
@@ -170,7 +199,7 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
 #pragma unroll
     for (int j = 0; j < kDeltaMaxWarps; ++j)
 #pragma unroll
-      for (int c = 0; c < COLS; ++c) v[j][c] = next_v[j][c];
+      for (int c = 0; c < COLS; ++c) v[j][c] = to_float(next_v[j][c]);
     __syncthreads();
     if (base + warps < length) fetch(base + warps);   // on its way while this batch is walked through
 #pragma unroll
@@ -204,12 +233,14 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
       float u[COLS];
 #pragma unroll
       for (int c = 0; c < COLS; ++c) {
+        if (MODE != kDeltaDual) {
 #pragma unroll
-        for (int offset = 1; offset < LANES; offset <<= 1) {   // over the lanes that share the column
-          if (MODE != kDeltaDual) k_dot[c] += __shfl_xor_sync(0xffffffffu, k_dot[c], offset);
-          q_dot[c] += __shfl_xor_sync(0xffffffffu, q_dot[c], offset);
+          for (int offset = 1; offset < LANES; offset <<= 1) {   // over the lanes that share the column
+            k_dot[c] += __shfl_xor_sync(0xffffffffu, k_dot[c], offset);
+            q_dot[c] += __shfl_xor_sync(0xffffffffu, q_dot[c], offset);
+          }
         }
-        u[c] = s_beta[j] * (v[j][c] - k_dot[c]);
+        u[c] = s_beta[j] * (v[j][c] - k_dot[c]);   // the dual looks at nothing: k_dot is 0
       }
 #pragma unroll
       for (int i = 0; i < DPT; i += 4) {   // the write
@@ -222,14 +253,37 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
           s[c][i + 2] = fmaf(k.z, u[c], s[c][i + 2]); s[c][i + 3] = fmaf(k.w, u[c], s[c][i + 3]);
         }
       }
-      if (part == 0) {
+      float* out_row = out + (static_cast<long long>(first + base + j)) * (static_cast<long long>(heads) * vdim) + head * vdim + column;
+      if (MODE == kDeltaDual && COLS == 4) {
+        // Four columns over LANES lanes: each exchange halves the columns a lane still adds up, so that a quarter of
+        // the lanes ends with each column's sum instead of every lane with all four.
+        const bool upper = (part & (LANES / 2)) != 0, odd = (part & (LANES / 4)) != 0;
+        float keep0 = upper ? q_dot[2 % COLS] : q_dot[0], keep1 = upper ? q_dot[3 % COLS] : q_dot[1 % COLS];
+        keep0 += __shfl_xor_sync(0xffffffffu, upper ? q_dot[0] : q_dot[2 % COLS], LANES / 2);
+        keep1 += __shfl_xor_sync(0xffffffffu, upper ? q_dot[1 % COLS] : q_dot[3 % COLS], LANES / 2);
+        float sum = odd ? keep1 : keep0;
+        sum += __shfl_xor_sync(0xffffffffu, odd ? keep0 : keep1, LANES / 4);
+#pragma unroll
+        for (int offset = LANES / 8; offset > 0; offset >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
+        const float mine = upper ? (odd ? v[j][3 % COLS] : v[j][2 % COLS]) : (odd ? v[j][1 % COLS] : v[j][0]);
+        const int c = (upper ? 2 : 0) + (odd ? 1 : 0);
+        if (part % (LANES / 4) == 0 && column + c < vdim) out_row[c] = fmaf(s_qk[j], s_beta[j] * mine, sum) + head_skip * mine;
+      } else if (part == 0) {
 #pragma unroll
         for (int c = 0; c < COLS; ++c)
-          if (live[c])
-            out[(static_cast<long long>(first + base + j)) * (static_cast<long long>(heads) * vdim) + head * vdim + column + c] =
-                fmaf(s_qk[j], u[c], q_dot[c]) + (MODE == kDeltaDual ? head_skip * v[j][c] : 0.0f);
+          if (live[c]) out_row[c] = fmaf(s_qk[j], u[c], q_dot[c]);
       }
     }
+  }
+  if (whole) {
+#pragma unroll
+    for (int c = 0; c < COLS; ++c)
+#pragma unroll
+      for (int i = 0; i < DPT; i += 4)
+        if (live[c] && part * DPT < dim)
+          *reinterpret_cast<float4*>(column_state + static_cast<long long>(c) * dim + i) =
+              make_float4(s[c][i], s[c][i + 1], s[c][i + 2], s[c][i + 3]);
+    return;
   }
 #pragma unroll
   for (int i = 0; i < DPT; ++i) {
@@ -275,18 +329,22 @@ MXB_API int mxb_delta_rule(const void* qkv, long long ld, int q_off, int k_off, 
   const int lanes = dim <= 32 ? 4 : (dim <= 64 ? 8 : 16);
   const int per_lane = dim <= 16 ? 4 : (dim <= 128 ? 8 : 16);
   const int step = 32 / lanes;                                   // columns of a warp
-  int columns = ((vdim + step - 1) / step) * step;
+  // The dual has no chain from token to token but the decay, so a thread takes four columns: what is read from shared
+  // memory serves four, and the sums over the lanes cost a third of the exchanges.
+  const int cols = mode == kDeltaDual ? 4 : 1;                   // columns of a thread
+  int columns = ((vdim + cols * step - 1) / (cols * step)) * step;     // ... of a block, in units of `cols`
   // A step of single tokens (`longest`, the most tokens of any row, if the caller knows it; 0: unknown) is one
   // chain of trips to memory per block: small blocks, several of them resident on an SM, overlap their chains.
-  const int most = (longest > 0 && longest < 8 ? 128 : 512) / lanes;
+  const int most = (longest > 0 && longest < 8 ? 128 : (mode == kDeltaDual ? 256 : 512)) / lanes;
   if (columns > most) columns = most;
+  const int units = (vdim + cols - 1) / cols;
   while (columns > 2 * step && columns >= 32 &&
-         static_cast<long long>(rows) * heads * ((vdim + columns - 1) / columns) < 128)
+         static_cast<long long>(rows) * heads * ((units + columns - 1) / columns) < 128)
     columns /= 2;
   columns = ((columns + step - 1) / step) * step;
-  const dim3 grid(rows, heads, (vdim + columns - 1) / columns), block(columns * lanes);
+  const dim3 grid(rows, heads, (units + columns - 1) / columns), block(columns * lanes);
 #define LAUNCH_MODE(T, DPT, LANES, MODE)                                                                            \
-  delta_rule_kernel<T, DPT, LANES, 1, MODE><<<grid, block, 0, stream>>>(static_cast<const T*>(qkv), ld, q_off, k_off,      \
+  delta_rule_kernel<T, DPT, LANES, MODE == kDeltaDual ? 4 : 1, MODE><<<grid, block, 0, stream>>>(static_cast<const T*>(qkv), ld, q_off, k_off,      \
       v_off, static_cast<const T*>(beta_pre), ldb, b_off, step_pre, lds, step_bias, rate, skip, state, slot_stride, \
       num_slots, row_start, row_length, request_slots, out, heads, groups, dim, vdim, status)
 #define LAUNCH(T, DPT, LANES)                                        \
