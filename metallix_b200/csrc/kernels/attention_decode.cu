@@ -243,14 +243,15 @@ __device__ __forceinline__ float decode_exp2(float x) {
   asm("ex2.approx.ftz.f32 %0, %1;\n" : "=f"(y) : "f"(x));
   return y;
 }
-// The biases of a thread's eight keys (zeros without a table): key nb * 8 + j of its own lies `back` - nb * 8 - j
-// positions back. Asked for ahead of the wait for the keys: a table is no kernel's output.
+// The biases of a thread's eight keys: key nb * 8 + j of its own lies `back` - nb * 8 - j positions back. Asked for
+// ahead of the wait for the keys: a table is no kernel's output. The kernels below are built with and without them
+// (BIASED): the registers they take would cost an unbiased step its third block on an SM.
 __device__ __forceinline__ void decode_biases(float (&near)[4][2], ScoreBias bias, int head, bool live, int back) {
 #pragma unroll
   for (int nb = 0; nb < 4; ++nb)
 #pragma unroll
     for (int j = 0; j < 2; ++j)
-      near[nb][j] = bias.table != nullptr && live ? bias_at(bias.row(head), back - nb * 8 - j, bias.far) : 0.0f;
+      near[nb][j] = live ? bias_at(bias.row(head), back - nb * 8 - j, bias.far) : 0.0f;
 }
 // Key rows lie in shared memory as they lie in the cache, each followed by 16
 // bytes of padding: eight consecutive rows then start in eight different bank
@@ -259,7 +260,7 @@ template <int HD> __device__ __forceinline__ uint32_t decode_tile_offset(int row
   return static_cast<uint32_t>(row * (HD * 2 + 16) + (chunk << 4));
 }
 
-template <int HD>
+template <int HD, bool BIASED>
 __global__ void __launch_bounds__(kDecodeThreads)
 paged_attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ cache,
                                   float* __restrict__ partial, const int* __restrict__ block_tables,
@@ -357,7 +358,7 @@ paged_attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __n
     }
   }
   float near[4][2];
-  decode_biases(near, bias, kv * group + g, g < group, pos - begin - warp * 32 - 2 * t);
+  if (BIASED) decode_biases(near, bias, kv * group + g, g < group, pos - begin - warp * 32 - 2 * t);
   const bool keys_landed = barrier_wait(&barriers[0], 0, status);
   __syncthreads();  // also orders the zero rows written by other threads
 
@@ -387,7 +388,7 @@ paged_attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __n
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int kk = key_base + nb * 8 + 2 * t + j;
-      sc[nb][j] = kk < count ? (capped_score(sc[nb][j] * scale, softcap) + near[nb][j]) * kLog2E : -INFINITY;
+      sc[nb][j] = kk < count ? (capped_score(sc[nb][j] * scale, softcap) + (BIASED ? near[nb][j] : 0.0f)) * kLog2E : -INFINITY;
       m_w = fmaxf(m_w, sc[nb][j]);
     }
   }
@@ -475,7 +476,7 @@ template <int HD> __device__ __forceinline__ uint32_t decode_swizzled_offset(int
   return static_cast<uint32_t>((chunk >> 3) * (kSplitKeys * 128) + row * 128 + (((chunk & 7) ^ (row & 7)) << 4));
 }
 
-template <int HD>
+template <int HD, bool BIASED>
 __global__ void __launch_bounds__(kDecodeThreads)
 paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache, const __nv_bfloat16* __restrict__ q,
                                   float* __restrict__ partial, const int* __restrict__ block_tables,
@@ -563,7 +564,7 @@ paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache,
     }
   }
   float near[4][2];
-  decode_biases(near, bias, kv * group + g, g < group, pos - key0 - warp * 32 - 2 * t);
+  if (BIASED) decode_biases(near, bias, kv * group + g, g < group, pos - key0 - warp * 32 - 2 * t);
   const bool keys_landed = barrier_wait(&barriers[0], 0, status);
 
   // ---- scores of this warp's 32 keys
@@ -593,7 +594,7 @@ paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache,
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int kk = key_base + nb * 8 + 2 * t + j;
-      sc[nb][j] = kk >= lo && kk <= hi ? (capped_score(sc[nb][j] * scale, softcap) + near[nb][j]) * kLog2E : -INFINITY;
+      sc[nb][j] = kk >= lo && kk <= hi ? (capped_score(sc[nb][j] * scale, softcap) + (BIASED ? near[nb][j] : 0.0f)) * kLog2E : -INFINITY;
       m_w = fmaxf(m_w, sc[nb][j]);
     }
   }
@@ -697,8 +698,8 @@ paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache,
 // leaves one partial result (slot s of the pair); the merge kernel puts the
 // slots together in slot order. Which block takes which tile depends on the
 // token's position and on `slots` alone.
-template <int HD>
-__global__ void __launch_bounds__(kDecodeThreads)
+template <int HD, bool BIASED>
+__global__ void __launch_bounds__(kDecodeThreads, 3)
 paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_cache, const __nv_bfloat16* __restrict__ q,
                                        float* __restrict__ partial, const int* __restrict__ block_tables,
                                        int max_pages, const int* __restrict__ row_token,
@@ -805,7 +806,7 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
     const int lo = max(first_key - key0, 0), hi = min(pos - key0, kSplitKeys - 1);   // the tile's rows that count
     const bool has_keys = key_base <= hi && key_base + 31 >= lo;
     float near[4][2];
-    decode_biases(near, bias, kv * group + g, g < group, pos - key0 - warp * 32 - 2 * t);
+    if (BIASED) decode_biases(near, bias, kv * group + g, g < group, pos - key0 - warp * 32 - 2 * t);
     const bool keys_landed = barrier_wait(&barriers[0], parity, status);
 
     // ---- scores of this warp's 32 keys
@@ -832,7 +833,7 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int kk = key_base + nb * 8 + 2 * t + j;
-        sc[nb][j] = kk >= lo && kk <= hi ? (capped_score(sc[nb][j] * scale, softcap) + near[nb][j]) * kLog2E : -INFINITY;
+        sc[nb][j] = kk >= lo && kk <= hi ? (capped_score(sc[nb][j] * scale, softcap) + (BIASED ? near[nb][j] : 0.0f)) * kLog2E : -INFINITY;
         m_t = fmaxf(m_t, sc[nb][j]);
       }
     }
@@ -1117,7 +1118,8 @@ static int launch_decode_mma(const void* q, const void* cache, void* out, float*
       slots = target / pairs > 0 ? target / pairs : 1;
     }
     if (slots > 0 && 2 * slots <= max_splits) {
-      auto kernel = paged_attention_decode_resident_kernel<HD>;
+      auto kernel = project.bias.table != nullptr ? paged_attention_decode_resident_kernel<HD, true>
+                                                  : paged_attention_decode_resident_kernel<HD, false>;
       cudaError_t attribute = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, shared);
       if (attribute != cudaSuccess) return static_cast<int>(attribute);
       e = launch_chained(kernel, dim3(slots, kv_heads, rows), dim3(kDecodeThreads), shared, stream, map_cache,
@@ -1126,7 +1128,8 @@ static int launch_decode_mma(const void* q, const void* cache, void* out, float*
       if (e != cudaSuccess) return static_cast<int>(e);
       return finish(slots);
     }
-    auto kernel = paged_attention_decode_tma_kernel<HD>;
+    auto kernel = project.bias.table != nullptr ? paged_attention_decode_tma_kernel<HD, true>
+                                                : paged_attention_decode_tma_kernel<HD, false>;
     cudaError_t attribute = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, shared);
     if (attribute != cudaSuccess) return static_cast<int>(attribute);
     e = launch_chained(kernel, grid, dim3(kDecodeThreads), shared, stream, map_cache,
@@ -1134,7 +1137,8 @@ static int launch_decode_mma(const void* q, const void* cache, void* out, float*
                        positions, heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, project.softcap, project.bias, status);
   } else {
     const int shared = 2 * kSplitKeys * (HD * 2 + 16);
-    auto kernel = paged_attention_decode_mma_kernel<HD>;
+    auto kernel = project.bias.table != nullptr ? paged_attention_decode_mma_kernel<HD, true>
+                                                : paged_attention_decode_mma_kernel<HD, false>;
     cudaError_t attribute = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, shared);
     if (attribute != cudaSuccess) return static_cast<int>(attribute);
     e = launch_chained(kernel, grid, dim3(kDecodeThreads), shared, stream,

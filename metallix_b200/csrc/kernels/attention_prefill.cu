@@ -67,7 +67,7 @@ template <int HD> __device__ __forceinline__ uint32_t tile_offset(int row, int c
   return static_cast<uint32_t>(row * (HD * 2) + ((chunk ^ (row & 7)) << 4));
 }
 
-template <int HD>
+template <int HD, bool BIASED>
 __global__ void __launch_bounds__(kFlashThreads, 3)
 flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* __restrict__ cache,
                      __nv_bfloat16* __restrict__ out, const int* __restrict__ block_tables, int max_pages,
@@ -201,7 +201,7 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
       }
     }
     // ---- a bias per head and distance, if any, kept over scale as well
-    if (bias.table != nullptr) {
+    if (BIASED) {
       const float* table = bias.row(head);
       const float over = 1.0f / scale;
 #pragma unroll
@@ -323,7 +323,7 @@ static int launch_flash(const void* q, const void* cache, void* out, const int* 
                         float softcap, int has_sink, float sink_score, const float* sink_heads, ScoreBias bias, int* status,
                         cudaStream_t stream) {
   const int shared = 4 * kFlashKeys * HD * 2;
-  auto kernel = flash_prefill_kernel<HD>;
+  auto kernel = bias.table != nullptr ? flash_prefill_kernel<HD, true> : flash_prefill_kernel<HD, false>;
   cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, shared);
   if (e != cudaSuccess) return static_cast<int>(e);
   dim3 grid(heads, 2 * tiles);

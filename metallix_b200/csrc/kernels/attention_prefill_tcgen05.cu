@@ -69,7 +69,7 @@ __device__ __forceinline__ uint32_t fa_pack(float lo, float hi) {
   return *reinterpret_cast<uint32_t*>(&pair);
 }
 
-template <int HD>
+template <int HD, bool BIASED>   // BIASED: built apart, its registers and instructions are no unbiased call's
 __global__ void __launch_bounds__(kFaThreads, 1)
 flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_cache,
                              __nv_bfloat16* __restrict__ out, const int* __restrict__ block_tables, int max_pages,
@@ -152,7 +152,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
     barrier_init_fence();
     failed = 0;
   }
-  if (bias_bytes > 0)
+  if (BIASED && bias_bytes > 0)
     for (int i = threadIdx.x; i <= bias.far; i += kFaThreads) near_bias[i] = bias.row(head)[i];
   if (warp == 1) {
     asm volatile("tcgen05.alloc.cta_group::1.sync.aligned.shared::cta.b32 [%0], %1;\n"
@@ -307,7 +307,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
     const float scale_log2 = scale * 1.4426950408889634f;
     const uint32_t tmem_lane = tmem_base + (static_cast<uint32_t>(lane_base) << 16);
     uint64_t* meet = &row_ready[warp & 3];
-    const float* bias_row = bias.table == nullptr ? nullptr : (bias_bytes > 0 ? near_bias : bias.row(head));
+    const float* bias_row = !BIASED ? nullptr : (bias_bytes > 0 ? near_bias : bias.row(head));
     const float over_scale = 1.0f / scale;
     float acc[PART_HD];
 #pragma unroll
@@ -342,7 +342,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
 #pragma unroll
         for (int j = 0; j < PART_KEYS; ++j) raw[j] = __float_as_uint(outer * tanhf(__uint_as_float(raw[j]) * inner));
       }
-      if (bias.table != nullptr) {   // over scale as well; keys from bias.far positions back on share one number
+      if (BIASED) {   // over scale as well; keys from bias.far positions back on share one number
         const int back = pos - key0;
         if (back - (PART_KEYS - 1) >= bias.far) {
           const float far = bias_row[bias.far] * over_scale;
@@ -512,7 +512,7 @@ static int launch_flash_tc(const void* q, const void* cache, void* out, const in
   if (!make_map(&map_q, q, tokens, heads * HD, static_cast<long long>(heads) * HD, kFaRows) ||
       !make_map(&map_cache, cache, static_cast<int>(cache_rows), HD, HD, page_tokens))
     return static_cast<int>(cudaErrorInvalidValue);
-  auto kernel = flash_prefill_tcgen05_kernel<HD>;
+  auto kernel = bias.table != nullptr ? flash_prefill_tcgen05_kernel<HD, true> : flash_prefill_tcgen05_kernel<HD, false>;
   static int shared_limit = 0;
   if (shared_limit == 0) {
     int device = 0;
