@@ -1651,6 +1651,7 @@ def design_kokolorn(args):
     inner, ones = sh * sv, torch.ones(hidden, device="cuda")
     for tokens in (8, prompt * 4):
         x, a, b, row = normal(tokens, hidden), normal(tokens, hidden).to(bf16), normal(tokens, hidden).to(bf16), normal(hidden)
+        first = normal(tokens, hidden)
         kernels[f"sublayer_input_{tokens}"] = {
             "kokolorn: x += norm(a + bias) / 2 + norm(b) / 2; y = norm(x)": gbs(
                 tokens * hidden * (4 + 4 + 2 + 2 + 2),
@@ -1659,7 +1660,7 @@ def design_kokolorn(args):
             "dimorax: x += m (a + b); two norms of x": gbs(
                 tokens * hidden * (4 + 4 + 2 + 2 + 2 + 2), lambda: ops.pair_add_rmsnorm(x, a, b, 0.5, ones, ones, 1e-6, bf16)),
             "qwen3: x += d; y = norm(x)": gbs(tokens * hidden * (4 + 4 + 2 + 2), lambda: ops.add_rmsnorm(x, a, ones, 1e-6, bf16)),
-            "kokolorn: [x + d | x0] rounded": gbs(tokens * hidden * (4 + 2 + 4 + 4), lambda: ops.join_rows(x, a, x, bf16)),
+            "kokolorn: [x + d | x0] rounded": gbs(tokens * hidden * (4 + 2 + 4 + 4), lambda: ops.join_rows(x, a, first, bf16)),
             "kokolorn: x += row; y = norm(x)": gbs(tokens * hidden * (4 + 4 + 2), lambda: ops.add_rmsnorm(x, row, ones, 1e-6, bf16))}
         wide, product = normal(tokens, inner), normal(tokens, 2 * inner).to(bf16)
         weight = torch.ones(inner, device="cuda")
