@@ -3,6 +3,7 @@ the architecture registry."""
 from .dimorax import DimoraxConfig
 from .kokolorn import KokolornConfig
 from .mekazen import MekazenConfig
+from .mekuvik import MekuvikConfig
 from .qwen3 import ConfigError, Qwen3Config
 from .registry import (ModelFamily, family_by_kind, parse_config, read_config, register,
                        resolve, unregister)
@@ -11,6 +12,7 @@ from .zitezen import ZitezenConfig
 from .spec import CacheNeed, LayerRun, LayerSpec, ModelSpec, PartSpec
 
 __all__ = ["ConfigError", "MekazenConfig", "Qwen3Config", "ZitezenConfig", "SadosunConfig", "DimoraxConfig", "KokolornConfig",
+           "MekuvikConfig",
            "ModelFamily", "family_by_kind", "parse_config",
            "read_config", "register", "resolve", "unregister", "CacheNeed", "LayerRun",
            "LayerSpec", "ModelSpec", "PartSpec"]

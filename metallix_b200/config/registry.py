@@ -18,6 +18,7 @@ from typing import Any, Dict, Mapping, Optional, Type
 from .dimorax import DimoraxConfig
 from .kokolorn import KokolornConfig
 from .mekazen import MekazenConfig
+from .mekuvik import MekuvikConfig
 from .qwen3 import ConfigError, Qwen3Config
 from .sadosun import SadosunConfig
 from .zitezen import ZitezenConfig
@@ -144,3 +145,6 @@ register(DIMORAX)
 KOKOLORN = ModelFamily(architecture=KokolornConfig.ARCHITECTURE, model_type=KokolornConfig.MODEL_TYPE,
                        kind="kokolorn", config_class=KokolornConfig)
 register(KOKOLORN)
+MEKUVIK = ModelFamily(architecture=MekuvikConfig.ARCHITECTURE, model_type=MekuvikConfig.MODEL_TYPE,
+                      kind="mekuvik", config_class=MekuvikConfig)
+register(MEKUVIK)

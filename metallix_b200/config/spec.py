@@ -82,7 +82,8 @@ class CacheNeed:
     ``head_dim`` for every position (``window is None``) or for the last
     ``window`` positions; with ``chunk`` only the positions of the chunk of
     that many positions (counted from position 0) the next query lies in are
-    ever read again. ``planes`` is 2 for keys and values, 1 for a pool with
+    ever read again; the first ``keep`` positions of a sequence are kept beside
+    either. ``planes`` is 2 for keys and values, 1 for a pool with
     one row per position that serves as both (a latent that all heads share).
     ``kind == "state"``: ``state_shape`` values of fixed
     size per request, zeroed when the request is admitted. ``kind == "none"``:
@@ -99,9 +100,10 @@ class CacheNeed:
     state_dtype: str = "float32"
     planes: int = 2
     members: Tuple["CacheNeed", ...] = ()
+    keep: int = 0
 
     def group_key(self) -> tuple:
-        return (self.kind, self.kv_heads, self.head_dim, self.window, self.chunk,
+        return (self.kind, self.kv_heads, self.head_dim, self.window, self.chunk, self.keep,
                 tuple(self.state_shape), self.state_dtype, self.planes,
                 tuple(member.group_key() for member in self.members))
 

@@ -5,8 +5,9 @@
 // group, and every group has pages and block tables of its own: a group either
 // keeps every position (window == 0, chunk == 0), only the last `window`
 // positions, or only the positions of the chunk of `chunk` positions that the
-// next query lies in (chunks counted from position 0); pages that no later
-// query can see go back to the free list as soon as they have been passed.
+// next query lies in (chunks counted from position 0), either rule widened by
+// the first `keep` positions of a sequence; pages that no later query can see
+// go back to the free list as soon as they have been passed.
 // The protocol per step is the reference's (crates/core/engine/src/blocks.rs:17-45):
 // reserve (all or nothing) -> the forward pass writes -> commit.
 // Beside the pages every request holds one slot of fixed-size state.
@@ -35,6 +36,7 @@ struct GroupConfig {
   int window = 0;        // 0: every position is kept; else the last `window`
   int chunk = 0;         // 0: no chunks; else queries see keys of their own chunk of this many positions only
   int num_pages = 0;     // pages of this group's pool
+  int keep = 0;          // the first positions of a sequence that stay whatever the window or chunk
 };
 
 // Raised when a reservation does not fit; the manager is unchanged
@@ -56,6 +58,7 @@ class CacheManager {
       if (g.page_tokens <= 0) throw std::invalid_argument("page_tokens must be positive");
       if (g.window < 0) throw std::invalid_argument("window must not be negative");
       if (g.chunk < 0) throw std::invalid_argument("chunk must not be negative");
+      if (g.keep < 0) throw std::invalid_argument("keep must not be negative");
       if (g.num_pages < 0) throw std::invalid_argument("num_pages must not be negative");
     }
     free_pages_.resize(groups_.size());
@@ -163,7 +166,8 @@ class CacheManager {
       if (cfg.chunk > 0) first_needed = std::max<int64_t>(first_needed, r.computed - r.computed % cfg.chunk);
       if (first_needed <= 0) continue;
       int64_t dead_pages = first_needed / cfg.page_tokens;  // pages wholly below
-      for (int64_t p = r.first_live[g]; p < dead_pages && p < static_cast<int64_t>(r.tables[g].size()); ++p) {
+      // Pages that hold kept positions stay: the table has a hole behind them.
+      for (int64_t p = std::max(r.first_live[g], ceil_div(cfg.keep, cfg.page_tokens)); p < dead_pages && p < static_cast<int64_t>(r.tables[g].size()); ++p) {
         give_back(static_cast<int>(g), r.tables[g][p]);
         r.tables[g][p] = -1;
       }
@@ -255,7 +259,7 @@ class CacheManager {
   int references(int g, int page) const { return refs_.at(g).at(page); }
 
   // Logical page -> physical page of one group, -1 where the window has
-  // passed the page.
+  // passed the page (and it holds no position that is kept).
   const std::vector<int>& table(int64_t id, int g) const { return get(id).tables.at(g); }
   int64_t first_live_page(int64_t id, int g) const { return get(id).first_live.at(g); }
 
@@ -282,6 +286,8 @@ class CacheManager {
         for (size_t p = 0; p < r.tables[g].size(); ++p) {
           int page = r.tables[g][p];
           if (page < 0) {
+            if (static_cast<int64_t>(p) < ceil_div(groups_[g].keep, groups_[g].page_tokens))
+              throw std::logic_error("a page of kept positions is gone");
             if (static_cast<int64_t>(p) >= r.first_live[g]) throw std::logic_error("a hole inside the live pages");
             continue;
           }

@@ -60,7 +60,7 @@ paged_attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ cac
                               int max_pages, const int* __restrict__ row_token,
                               const int* __restrict__ row_request, const int* __restrict__ positions,
                               int heads, int kv_heads, int page_tokens, int num_pages, int max_splits,
-                              int window, int chunk, float scale, float softcap, ScoreBias bias, int* status) {
+                              int window, int chunk, int keep, float scale, float softcap, ScoreBias bias, int* status) {
   constexpr int E = Vec16<T>::kElems;  // elements per 16-byte piece
   constexpr int LPK = HD / E;          // 16-byte pieces (and lanes) per key row
   constexpr int KPW = 32 / LPK;        // key rows a warp reads at once
@@ -82,9 +82,10 @@ paged_attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ cac
   const int pos = positions[token];
   const int group = heads / kv_heads;  // query heads per key/value head, <= G
   const int first_key = first_visible_key(pos, window, chunk);
-  const int begin = max(split * kSplitKeys, first_key);
-  const int end = min((split + 1) * kSplitKeys, pos + 1);
-  if (begin >= end) return;  // the merge skips splits outside [first_key, pos]
+  const int key0 = split * kSplitKeys;
+  const int begin = key0 < keep ? key0 : max(key0, first_key);
+  const int end = min(key0 + kSplitKeys, pos + 1);
+  if (begin >= end) return;  // the merge skips splits without keys of the token
   const int count = end - begin;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
   const int* table = block_tables + static_cast<size_t>(row_request[row]) * max_pages;
@@ -99,12 +100,14 @@ paged_attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ cac
     T* dst_base = pass == 0 ? sK : sV;
     for (int kk = tid / LPK; kk < count; kk += ROWS) {
       const int key = begin + kk;
-      int page = table[key / page_tokens];
+      const bool seen = key_seen(key, pos, first_key, keep);   // else: between the kept keys and the window
+      int page = seen ? table[key / page_tokens] : 0;
       bool ok = page >= 0 && page < num_pages;
       if (!ok) {
         if (piece == 0 && pass == 0) atomicOr(status, kStatusBadPage);
         page = 0;
       }
+      ok = ok && seen;
       const T* src = head_base + page * page_stride + (pass == 0 ? 0 : v_offset) +
                      static_cast<size_t>(key % page_tokens) * HD + piece * E;
       decode_copy_async_16(dst_base + kk * HD + piece * E, src, ok ? 16 : 0);
@@ -152,7 +155,7 @@ paged_attention_decode_kernel(const T* __restrict__ q, const T* __restrict__ cac
       if (sub == 0 && kk < count) {
         float s = capped_score(dots[h] * scale, softcap);
         if (bias.table != nullptr && h < group) s += bias_at(bias.row(kv * group + h), pos - begin - kk, bias.far);
-        s_score[h * kSplitKeys + kk] = s;
+        s_score[h * kSplitKeys + kk] = key_seen(begin + kk, pos, first_key, keep) ? s : -INFINITY;
       }
     }
   }
@@ -267,7 +270,7 @@ paged_attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __n
                                   int max_pages, const int* __restrict__ row_token,
                                   const int* __restrict__ row_request, const int* __restrict__ positions,
                                   int heads, int kv_heads, int page_tokens, int num_pages, int max_splits,
-                                  int window, int chunk, float scale, float softcap, ScoreBias bias, int* status) {
+                                  int window, int chunk, int keep, float scale, float softcap, ScoreBias bias, int* status) {
   constexpr int ROW_BYTES = HD * 2;
   constexpr int TILE_BYTES = kSplitKeys * (ROW_BYTES + 16);
   extern __shared__ __align__(128) unsigned char mma_shared[];
@@ -286,8 +289,9 @@ paged_attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __n
   const int pos = positions[token];
   const int group = heads / kv_heads;  // <= 8
   const int first_key = first_visible_key(pos, window, chunk);
-  const int begin = max(split * kSplitKeys, first_key);
-  const int end = min((split + 1) * kSplitKeys, pos + 1);
+  const int key0 = split * kSplitKeys;
+  const int begin = key0 < keep ? key0 : max(key0, first_key);
+  const int end = min(key0 + kSplitKeys, pos + 1);
   if (begin >= end) return;
   const int count = end - begin;
   const int tid = threadIdx.x, lane = tid & 31, warp = tid >> 5;
@@ -308,7 +312,7 @@ paged_attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __n
     const size_t v_offset = static_cast<size_t>(kv_heads) * page_tokens * HD;
     const int kk = tid;  // kSplitKeys == kDecodeThreads
     const int key = begin + kk;
-    bool ok = kk < count;
+    bool ok = kk < count && key_seen(key, pos, first_key, keep);
     int page = 0;
     if (ok) {
       page = table[key / page_tokens];
@@ -336,7 +340,7 @@ paged_attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __n
       bulk_copy(sV + decode_tile_offset<HD>(kk, 0), src + v_offset, ROW_BYTES, &barriers[1]);
     }
     if (!ok) {
-      // A row beyond the split's keys: zeros, written by the thread itself.
+      // A row that is none of the token's keys: zeros, written by the thread itself.
       uint4* zk = reinterpret_cast<uint4*>(sK + decode_tile_offset<HD>(kk, 0));
       uint4* zv = reinterpret_cast<uint4*>(sV + decode_tile_offset<HD>(kk, 0));
 #pragma unroll
@@ -388,7 +392,7 @@ paged_attention_decode_mma_kernel(const __nv_bfloat16* __restrict__ q, const __n
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int kk = key_base + nb * 8 + 2 * t + j;
-      sc[nb][j] = kk < count ? (capped_score(sc[nb][j] * scale, softcap) + (BIASED ? near[nb][j] : 0.0f)) * kLog2E : -INFINITY;
+      sc[nb][j] = kk < count && key_seen(begin + kk, pos, first_key, keep) ? (capped_score(sc[nb][j] * scale, softcap) + (BIASED ? near[nb][j] : 0.0f)) * kLog2E : -INFINITY;
       m_w = fmaxf(m_w, sc[nb][j]);
     }
   }
@@ -483,7 +487,7 @@ paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache,
                                   int max_pages, const int* __restrict__ row_token,
                                   const int* __restrict__ row_request, const int* __restrict__ positions,
                                   int heads, int kv_heads, int page_tokens, int num_pages, int max_splits,
-                                  int window, int chunk, float scale, float softcap, ScoreBias bias, int* status) {
+                                  int window, int chunk, int keep, float scale, float softcap, ScoreBias bias, int* status) {
   constexpr int HALVES = HD / kTmaColumns;                 // 64-value halves of a row
   constexpr int TILE_BYTES = kSplitKeys * HD * 2;
   extern __shared__ unsigned char tma_decode_raw[];
@@ -524,8 +528,9 @@ paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache,
   const int pos = positions[token];
   const int group = heads / kv_heads;  // <= 8
   const int first_key = first_visible_key(pos, window, chunk);
-  if (key0 > pos || key0 + kSplitKeys <= first_key) return;   // the merge skips splits outside [first_key, pos]
-  const int lo = max(first_key - key0, 0), hi = min(pos - key0, kSplitKeys - 1);   // the split's rows that count
+  if (key0 > pos || (key0 + kSplitKeys <= first_key && key0 >= keep)) return;   // the merge skips splits without keys of the token
+  // The split's rows that count: lo .. hi, and up to hi those ahead of row `kept`.
+  const int lo = max(first_key - key0, 0), hi = min(pos - key0, kSplitKeys - 1), kept = keep - key0;
 
   if (tid == 0) {
     barrier_init(&barriers[0], 1);
@@ -540,7 +545,7 @@ paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache,
   // page that holds none of the token's keys is not wanted: its box starts
   // beyond the cache's last row, where the copy engine writes zeros.
   const bool fresh = fetcher && pos >= page_key && pos < page_key + page_tokens;
-  bool wanted = fetcher && page_key <= pos && page_key + page_tokens > first_key;
+  bool wanted = fetcher && page_key <= pos && (page_key + page_tokens > first_key || page_key < keep);
   if (wanted && (page < 0 || page >= num_pages)) {
     atomicOr(status, kStatusBadPage);
     wanted = false;
@@ -569,7 +574,7 @@ paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache,
 
   // ---- scores of this warp's 32 keys
   const int key_base = warp * 32;
-  const bool has_keys = key_base <= hi && key_base + 31 >= lo;
+  const bool has_keys = key_base <= hi && (key_base + 31 >= lo || key_base < kept);
   float sc[4][4];
 #pragma unroll
   for (int i = 0; i < 4; ++i) sc[i][0] = sc[i][1] = sc[i][2] = sc[i][3] = 0.0f;
@@ -594,7 +599,7 @@ paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache,
 #pragma unroll
     for (int j = 0; j < 2; ++j) {
       const int kk = key_base + nb * 8 + 2 * t + j;
-      sc[nb][j] = kk >= lo && kk <= hi ? (capped_score(sc[nb][j] * scale, softcap) + (BIASED ? near[nb][j] : 0.0f)) * kLog2E : -INFINITY;
+      sc[nb][j] = (kk >= lo || kk < kept) && kk <= hi ? (capped_score(sc[nb][j] * scale, softcap) + (BIASED ? near[nb][j] : 0.0f)) * kLog2E : -INFINITY;
       m_w = fmaxf(m_w, sc[nb][j]);
     }
   }
@@ -627,7 +632,7 @@ paged_attention_decode_tma_kernel(const __grid_constant__ CUtensorMap map_cache,
   if (has_keys && (key_base < lo || key_base + 31 > hi)) {
     for (int i = lane; i < 32 * (HD / 8); i += 32) {
       const int vrow = key_base + i / (HD / 8);
-      if (vrow < lo || vrow > hi)
+      if ((vrow < lo && vrow >= kept) || vrow > hi)
         *reinterpret_cast<uint4*>(sV + decode_swizzled_offset<HD>(vrow, i % (HD / 8))) = make_uint4(0u, 0u, 0u, 0u);
     }
     __syncwarp();
@@ -705,7 +710,7 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
                                        int max_pages, const int* __restrict__ row_token,
                                        const int* __restrict__ row_request, const int* __restrict__ positions,
                                        int heads, int kv_heads, int page_tokens, int num_pages, int max_splits,
-                                       int window, int chunk, float scale, float softcap, ScoreBias bias, int* status) {
+                                       int window, int chunk, int keep, float scale, float softcap, ScoreBias bias, int* status) {
   constexpr int HALVES = HD / kTmaColumns;                 // 64-value halves of a row
   constexpr int TILE_BYTES = kSplitKeys * HD * 2;
   extern __shared__ unsigned char tma_decode_raw[];
@@ -737,9 +742,9 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
   const int pos = positions[token];
   const int group = heads / kv_heads;  // <= 8
   const int first_key = first_visible_key(pos, window, chunk);
-  const int first_tile = first_key / kSplitKeys, last_tile = pos / kSplitKeys;
-  int tile = first_tile + rank;
-  if (first_tile > 0) {
+  const KeyWalk walk = key_walk(first_key, pos, keep, kSplitKeys);
+  int step = rank, tile = walk.tile(step);   // the block's tiles: steps rank, rank + slots, ... of the walk
+  if (tile != rank) {
     page = 0;
     if (fetcher && tile * pages + slot < max_pages) page = table[tile * pages + slot];
   }
@@ -748,7 +753,7 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
     barrier_init(&barriers[0], 1);
     barrier_init(&barriers[1], 1);
     barrier_init_fence();
-    if (tile <= last_tile) {
+    if (step < walk.count) {
       barrier_arrive_expect(&barriers[0], TILE_BYTES);   // every box is fetched, whatever it holds
       barrier_arrive_expect(&barriers[1], TILE_BYTES);
     }
@@ -759,7 +764,7 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
   // cache's last row (zeros) when the page holds none of the token's keys.
   auto box_row_of = [&](int of_tile, int page_id) {
     const int page_key = of_tile * kSplitKeys + slot * page_tokens;
-    bool wanted = page_key <= pos && page_key + page_tokens > first_key;
+    bool wanted = page_key <= pos && (page_key + page_tokens > first_key || page_key < keep);
     if (wanted && (page_id < 0 || page_id >= num_pages)) {
       atomicOr(status, kStatusBadPage);
       wanted = false;
@@ -770,7 +775,7 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
   // ahead of this one: it waits; every other page of the first tile is
   // fetched right away.
   bool fresh = false;
-  if (fetcher && tile <= last_tile) {
+  if (fetcher && step < walk.count) {
     const int page_key = tile * kSplitKeys + slot * page_tokens;
     fresh = pos >= page_key && pos < page_key + page_tokens;
     if (!fresh) tma_load_2d(dst, &map_cache, half * kTmaColumns, box_row_of(tile, page), &barriers[which]);
@@ -796,15 +801,18 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
 #pragma unroll
   for (int i = 0; i < HD / 8; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.0f;
 
-  if (tile > last_tile) return;   // more slots than tiles: the merge skips this one
-  for (uint32_t turn = 0; tile <= last_tile; tile += slots, ++turn) {
+  if (step >= walk.count) return;   // more slots than tiles: the merge skips this one
+  for (uint32_t turn = 0; step < walk.count; step += slots, ++turn) {
     const uint32_t parity = turn & 1;
-    const int next = tile + slots;
+    tile = walk.tile(step);
+    const bool more = step + slots < walk.count;
+    const int next = walk.tile(step + slots);
     int next_page = 0;   // asked for now, needed when this tile's keys are used up
-    if (fetcher && next <= last_tile && next * pages + slot < max_pages) next_page = table[next * pages + slot];
+    if (fetcher && more && next * pages + slot < max_pages) next_page = table[next * pages + slot];
     const int key0 = tile * kSplitKeys;
-    const int lo = max(first_key - key0, 0), hi = min(pos - key0, kSplitKeys - 1);   // the tile's rows that count
-    const bool has_keys = key_base <= hi && key_base + 31 >= lo;
+    // The tile's rows that count: lo .. hi, and up to hi those ahead of row `kept`.
+    const int lo = max(first_key - key0, 0), hi = min(pos - key0, kSplitKeys - 1), kept = keep - key0;
+    const bool has_keys = key_base <= hi && (key_base + 31 >= lo || key_base < kept);
     float near[4][2];
     if (BIASED) decode_biases(near, bias, kv * group + g, g < group, pos - key0 - warp * 32 - 2 * t);
     const bool keys_landed = barrier_wait(&barriers[0], parity, status);
@@ -833,7 +841,7 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
 #pragma unroll
       for (int j = 0; j < 2; ++j) {
         const int kk = key_base + nb * 8 + 2 * t + j;
-        sc[nb][j] = kk >= lo && kk <= hi ? (capped_score(sc[nb][j] * scale, softcap) + (BIASED ? near[nb][j] : 0.0f)) * kLog2E : -INFINITY;
+        sc[nb][j] = (kk >= lo || kk < kept) && kk <= hi ? (capped_score(sc[nb][j] * scale, softcap) + (BIASED ? near[nb][j] : 0.0f)) * kLog2E : -INFINITY;
         m_t = fmaxf(m_t, sc[nb][j]);
       }
     }
@@ -860,7 +868,7 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
     // Every warp is done with the keys: the next tile's may come. One
     // decision for the whole block if a wait ran out (the status word says so).
     if (__syncthreads_or(!keys_landed)) break;
-    if (next <= last_tile) {
+    if (more) {
       if (tid == 0) barrier_arrive_expect(&barriers[0], TILE_BYTES);
       if (fetcher && which == 0) tma_load_2d(dst, &map_cache, half * kTmaColumns, box_row_of(next, next_page), &barriers[0]);
     }
@@ -872,7 +880,7 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
     if (has_keys && (key_base < lo || key_base + 31 > hi)) {
       for (int i = lane; i < 32 * (HD / 8); i += 32) {
         const int vrow = key_base + i / (HD / 8);
-        if (vrow < lo || vrow > hi)
+        if ((vrow < lo && vrow >= kept) || vrow > hi)
           *reinterpret_cast<uint4*>(sV + decode_swizzled_offset<HD>(vrow, i % (HD / 8))) = make_uint4(0u, 0u, 0u, 0u);
       }
       __syncwarp();
@@ -897,7 +905,7 @@ paged_attention_decode_resident_kernel(const __grid_constant__ CUtensorMap map_c
       }
     }
     if (__syncthreads_or(!values_landed)) break;   // every warp is done with the values
-    if (next <= last_tile) {
+    if (more) {
       if (tid == 0) barrier_arrive_expect(&barriers[1], TILE_BYTES);
       if (fetcher && which == 1) tma_load_2d(dst, &map_cache, half * kTmaColumns, box_row_of(next, next_page), &barriers[1]);
     }
@@ -950,7 +958,7 @@ template <typename T>
 __global__ void __launch_bounds__(256)
 paged_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__ out,
                              const int* __restrict__ row_token, const int* __restrict__ positions,
-                             int rows, int heads, int head_dim, int max_splits, int window, int chunk, int slots,
+                             int rows, int heads, int head_dim, int max_splits, int window, int chunk, int keep, int slots,
                              const T* __restrict__ gate, long long gate_stride, int has_sink, float sink_score, const float* sink_heads,
                              int* status) {
   chain_release();
@@ -959,19 +967,19 @@ paged_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__ 
   if (token < 0 || d >= head_dim) return;
   const int pos = positions[token];
   const int first_key = first_visible_key(pos, window, chunk);
-  const int first_split = first_key / kSplitKeys, last_split = pos / kSplitKeys;
-  if (last_split >= max_splits) {
+  const KeyWalk walk = key_walk(first_key, pos, keep, kSplitKeys);
+  if (pos / kSplitKeys >= max_splits) {
     // The caller's bound on the contexts does not cover this row: its partial
     // results lie outside what the scratch was sized for. The row is left as it is.
     if (d == 0) atomicOr(status, kStatusBadSlot);
     return;
   }
   // One partial result per split of 128 keys, or (slots > 0) per block of the
-  // resident kernel: slot s gathered the tiles first + s, first + s + slots, ...
-  const int splits = slots > 0 ? min(slots, last_split - first_split + 1) : last_split - first_split + 1;
+  // resident kernel: slot s gathered the steps s, s + slots, ... of the walk.
+  const int splits = slots > 0 ? min(slots, walk.count) : walk.count;
+  const int kept = slots > 0 ? splits : walk.kept;   // from the kept-th on, results lie `skip` places further
   const int stride = head_dim + 2;
-  const float* base = partial + (slots > 0 ? (static_cast<size_t>(row) * heads + head) * slots
-                                            : (static_cast<size_t>(row) * heads + head) * max_splits + first_split) * stride;
+  const float* base = partial + (static_cast<size_t>(row) * heads + head) * (slots > 0 ? slots : max_splits) * stride;
   chain_wait();
   base = behind_wait(base);  // the partial results are written by the kernel ahead of this one
   float m = kDecodeMinusHuge, acc = 0.0f, l = 0.0f;
@@ -980,7 +988,8 @@ paged_attention_merge_kernel(const float* __restrict__ partial, T* __restrict__ 
 #pragma unroll
     for (int j = 0; j < kMergeSplits; ++j) {
       const bool live = round + j < splits;
-      const float* p = base + static_cast<size_t>(live ? round + j : 0) * stride;
+      const int at = live ? round + j : 0;
+      const float* p = base + static_cast<size_t>(at < kept ? at : at + walk.skip) * stride;
       ms[j] = live ? p[head_dim] : kDecodeMinusHuge;
       ls[j] = live ? p[head_dim + 1] : 0.0f;
       values[j] = live ? p[d] : 0.0f;
@@ -1042,7 +1051,7 @@ template <typename T, int HD, int G>
 static int launch_decode(const void* q, const void* cache, void* out, float* partial,
                          const int* block_tables, int max_pages, const int* row_token,
                          const int* row_request, const int* positions, int rows, int heads,
-                         int kv_heads, int page_tokens, int num_pages, int max_splits, int window, int chunk,
+                         int kv_heads, int page_tokens, int num_pages, int max_splits, int window, int chunk, int keep,
                          float scale, int* status, cudaStream_t stream, DecodeProject project = DecodeProject()) {
   dim3 grid(max_splits, kv_heads, rows);
   constexpr int kElems = Vec16<T>::kElems;
@@ -1057,13 +1066,13 @@ static int launch_decode(const void* q, const void* cache, void* out, float* par
   }
   kernel<<<grid, kDecodeThreads, shared, stream>>>(
       static_cast<const T*>(q), static_cast<const T*>(cache), partial, block_tables, max_pages,
-      row_token, row_request, positions, heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk,
+      row_token, row_request, positions, heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, keep,
       scale, project.softcap, project.bias, status);
   cudaError_t e = cudaGetLastError();
   if (e != cudaSuccess) return static_cast<int>(e);
   return static_cast<int>(launch_chained(paged_attention_merge_kernel<T>, dim3(rows, heads), dim3(HD <= 64 ? 64 : (HD <= 128 ? 128 : 256)), 0,
                                          stream, static_cast<const float*>(partial), static_cast<T*>(out),
-                                         row_token, positions, rows, heads, HD, max_splits, window, chunk, 0,
+                                         row_token, positions, rows, heads, HD, max_splits, window, chunk, keep, 0,
                                          static_cast<const T*>(project.gate), project.gate_stride, project.has_sink,
                                          project.sink_score, project.sink_heads, status));
 }
@@ -1075,21 +1084,21 @@ template <int HD>
 static int launch_decode_mma(const void* q, const void* cache, void* out, float* partial,
                              const int* block_tables, int max_pages, const int* row_token,
                              const int* row_request, const int* positions, int rows, int heads,
-                             int kv_heads, int page_tokens, int num_pages, int max_splits, int window, int chunk,
+                             int kv_heads, int page_tokens, int num_pages, int max_splits, int window, int chunk, int keep,
                              float scale, int* status, cudaStream_t stream, DecodeProject project = DecodeProject()) {
   static_assert(kSplitKeys == kDecodeThreads, "one thread per key row of a split");
   auto finish = [&](int slots) -> int {
     if (project.w != nullptr)
       return static_cast<int>(launch_merge_project<HD>(partial, project.w, project.ldw, project.summands, row_token,
                                                        positions, rows, project.tokens, heads, project.hidden,
-                                                       max_splits, window, chunk, slots, kSplitKeys, kDecodeMinusHuge,
+                                                       max_splits, window, chunk, keep, slots, kSplitKeys, kDecodeMinusHuge,
                                                        static_cast<const __nv_bfloat16*>(project.gate),
                                                        project.gate_stride, project.has_sink, project.sink_score, project.sink_heads,
                                                        status, stream));
     return static_cast<int>(launch_chained(paged_attention_merge_kernel<__nv_bfloat16>, dim3(rows, heads),
                                            dim3(HD <= 64 ? 64 : (HD <= 128 ? 128 : 256)), 0, stream,
                                            static_cast<const float*>(partial), static_cast<__nv_bfloat16*>(out),
-                                           row_token, positions, rows, heads, HD, max_splits, window, chunk, slots,
+                                           row_token, positions, rows, heads, HD, max_splits, window, chunk, keep, slots,
                                            static_cast<const __nv_bfloat16*>(project.gate), project.gate_stride,
                                            project.has_sink, project.sink_score, project.sink_heads, status));
   };
@@ -1124,7 +1133,7 @@ static int launch_decode_mma(const void* q, const void* cache, void* out, float*
       if (attribute != cudaSuccess) return static_cast<int>(attribute);
       e = launch_chained(kernel, dim3(slots, kv_heads, rows), dim3(kDecodeThreads), shared, stream, map_cache,
                          static_cast<const __nv_bfloat16*>(q), partial, block_tables, max_pages, row_token, row_request,
-                         positions, heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, project.softcap, project.bias, status);
+                         positions, heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, keep, scale, project.softcap, project.bias, status);
       if (e != cudaSuccess) return static_cast<int>(e);
       return finish(slots);
     }
@@ -1134,7 +1143,7 @@ static int launch_decode_mma(const void* q, const void* cache, void* out, float*
     if (attribute != cudaSuccess) return static_cast<int>(attribute);
     e = launch_chained(kernel, grid, dim3(kDecodeThreads), shared, stream, map_cache,
                        static_cast<const __nv_bfloat16*>(q), partial, block_tables, max_pages, row_token, row_request,
-                       positions, heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, project.softcap, project.bias, status);
+                       positions, heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, keep, scale, project.softcap, project.bias, status);
   } else {
     const int shared = 2 * kSplitKeys * (HD * 2 + 16);
     auto kernel = project.bias.table != nullptr ? paged_attention_decode_mma_kernel<HD, true>
@@ -1144,7 +1153,7 @@ static int launch_decode_mma(const void* q, const void* cache, void* out, float*
     e = launch_chained(kernel, grid, dim3(kDecodeThreads), shared, stream,
                        static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(cache),
                        partial, block_tables, max_pages, row_token, row_request, positions, heads,
-                       kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, project.softcap, project.bias, status);
+                       kv_heads, page_tokens, num_pages, max_splits, window, chunk, keep, scale, project.softcap, project.bias, status);
   }
   if (e != cudaSuccess) return static_cast<int>(e);
   return finish(0);
@@ -1183,7 +1192,7 @@ MXB_API int mxb_paged_attention_decode(const void* q, const void* cache, void* o
                                        const int* block_tables, int max_pages, const int* row_token,
                                        const int* row_request, const int* positions, int rows,
                                        int heads, int kv_heads, int head_dim, int page_tokens,
-                                       int num_pages, int max_splits, int window, int chunk, float scale,
+                                       int num_pages, int max_splits, int window, int chunk, int keep, float scale,
                                        int dtype, const void* gate, long long gate_stride, float softcap, int has_sink,
                                        float sink_score, const float* sink_heads, const float* bias_table, int bias_far,
                                        int* status, cudaStream_t stream) {
@@ -1201,7 +1210,7 @@ MXB_API int mxb_paged_attention_decode(const void* q, const void* cache, void* o
   project.sink_heads = sink_heads;
   project.bias = ScoreBias{bias_table, bias_far};
 #define ARGS q, cache, out, partial, block_tables, max_pages, row_token, row_request, positions, rows, \
-             heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, status, stream, project
+             heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, keep, scale, status, stream, project
 #define BY_GROUP(T, HD)                                        \
   if (group == 1) return launch_decode<T, HD, 1>(ARGS);        \
   if (group == 2) return launch_decode<T, HD, 2>(ARGS);        \
@@ -1236,7 +1245,7 @@ MXB_API int mxb_paged_attention_decode_project(const void* q, const void* cache,
                                                const int* block_tables, int max_pages, const int* row_token,
                                                const int* row_request, const int* positions, int rows, int tokens,
                                                int heads, int kv_heads, int head_dim, int page_tokens, int num_pages,
-                                               int max_splits, int window, int chunk, float scale, const void* w, long long ldw,
+                                               int max_splits, int window, int chunk, int keep, float scale, const void* w, long long ldw,
                                                int hidden, float* summands, const void* gate, long long gate_stride,
                                                float softcap, int has_sink, float sink_score, const float* sink_heads,
                                                const float* bias_table, int bias_far, int* status, cudaStream_t stream) {
@@ -1259,7 +1268,7 @@ MXB_API int mxb_paged_attention_decode_project(const void* q, const void* cache,
   project.bias = ScoreBias{bias_table, bias_far};
   void* out = nullptr;
 #define ARGS q, cache, out, partial, block_tables, max_pages, row_token, row_request, positions, rows, \
-             heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, scale, status, stream, project
+             heads, kv_heads, page_tokens, num_pages, max_splits, window, chunk, keep, scale, status, stream, project
   return head_dim == 64 ? launch_decode_mma<64>(ARGS) : launch_decode_mma<128>(ARGS);
 #undef ARGS
 }
@@ -1328,7 +1337,7 @@ MXB_API int mxb_paged_attention_decode_noalloc(const void* q, const void* cache,
   if (e != cudaSuccess) return static_cast<int>(e);
   return mxb_paged_attention_decode(q, cache, out, scratch, block_tables, max_pages, row_token,
                                     row_request, positions, rows, heads, kv_heads, head_dim, page_tokens,
-                                    num_pages, splits, window, 0, scale, dtype, nullptr, 0, 0.0f, 0, 0.0f, nullptr, nullptr, 0, status, stream);
+                                    num_pages, splits, window, 0, 0, scale, dtype, nullptr, 0, 0.0f, 0, 0.0f, nullptr, nullptr, 0, status, stream);
 }
 
 MXB_TIMELINE_EXPORT(mxb_timeline_attention)

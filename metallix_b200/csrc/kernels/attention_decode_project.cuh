@@ -30,7 +30,7 @@ __global__ void __launch_bounds__(kProjectThreads)
 decode_merge_project_kernel(const float* __restrict__ partial, const __nv_bfloat16* __restrict__ w, long long ldw,
                             float* __restrict__ summands, const int* __restrict__ row_token,
                             const int* __restrict__ positions, int rows, int tokens, int heads, int hidden,
-                            int max_splits, int window, int chunk, int slots, int split_keys, float minus_huge,
+                            int max_splits, int window, int chunk, int keep, int slots, int split_keys, float minus_huge,
                             const __nv_bfloat16* __restrict__ gate, long long gate_stride, int has_sink,
                             float sink_score, const float* sink_heads, int* status) {
   constexpr int PITCH = HD * 2 + 16;  // bytes per row of a tile: rows a warp reads together fall on all banks
@@ -66,26 +66,29 @@ decode_merge_project_kernel(const float* __restrict__ partial, const __nv_bfloat
   const int stride = HD + 2;
   int turn_token[TURNS], turn_splits[TURNS];
   size_t turn_base[TURNS];
+  const int kept = slots > 0 ? 0x7fffffff : (keep + split_keys - 1) / split_keys;
+  int turn_skip[TURNS];                 // from the kept-th on, results lie `skip` places further
 #pragma unroll
   for (int turn = 0; turn < TURNS; ++turn) {
     const int row = warp + turn * (kProjectThreads / 32);
     turn_token[turn] = -1;
     turn_splits[turn] = 0;
     turn_base[turn] = 0;
+    turn_skip[turn] = 0;
     if (row >= rows) continue;
     const int token = row_token[row];
     if (token < 0 || token >= X_ROWS) continue;
     const int pos = positions[token];
     const int first_key = first_visible_key(pos, window, chunk);
-    const int first_split = first_key / split_keys, last_split = pos / split_keys;
-    if (last_split >= max_splits) {
+    const KeyWalk walk = key_walk(first_key, pos, keep, split_keys);
+    if (pos / split_keys >= max_splits) {
       if (lane == 0) atomicOr(status, kStatusBadSlot);
       continue;
     }
     turn_token[turn] = token;
-    turn_splits[turn] = slots > 0 ? min(slots, last_split - first_split + 1) : last_split - first_split + 1;
-    turn_base[turn] = (slots > 0 ? (static_cast<size_t>(row) * heads + head) * slots
-                                 : (static_cast<size_t>(row) * heads + head) * max_splits + first_split) * stride;
+    turn_splits[turn] = slots > 0 ? min(slots, walk.count) : walk.count;
+    turn_base[turn] = (static_cast<size_t>(row) * heads + head) * (slots > 0 ? slots : max_splits) * stride;
+    turn_skip[turn] = walk.skip;
   }
   chain_wait();
   partial = behind_wait(partial);  // written by the attention kernel ahead of this one
@@ -96,6 +99,8 @@ decode_merge_project_kernel(const float* __restrict__ partial, const __nv_bfloat
     const int token = turn_token[turn], splits = turn_splits[turn];
     if (token < 0) continue;
     const float* base = partial + turn_base[turn];
+    const int skip = turn_skip[turn];
+    auto place = [&](int i) { return static_cast<size_t>(i < kept ? i : i + skip) * stride; };
     float m = minus_huge, l = 0.0f;
     float2 acc[HD / 64];
 #pragma unroll
@@ -112,7 +117,7 @@ decode_merge_project_kernel(const float* __restrict__ partial, const __nv_bfloat
       const int live = min(kChunk, splits - round);
       float mine = minus_huge, mine_sum = 0.0f;
       if (lane < live) {
-        const float2 stats = *reinterpret_cast<const float2*>(base + static_cast<size_t>(round + lane) * stride + HD);
+        const float2 stats = *reinterpret_cast<const float2*>(base + place(round + lane) + HD);
         mine = stats.x;
         mine_sum = stats.y;
       }
@@ -121,7 +126,7 @@ decode_merge_project_kernel(const float* __restrict__ partial, const __nv_bfloat
       auto fetch = [&](float2 (&into)[kBatch][HD / 64], int from) {
 #pragma unroll
         for (int j = 0; j < kBatch; ++j) {
-          const float* p = base + static_cast<size_t>(round + (from + j < live ? from + j : 0)) * stride + lane * 2;
+          const float* p = base + place(round + (from + j < live ? from + j : 0)) + lane * 2;
 #pragma unroll
           for (int h = 0; h < HD / 64; ++h)
             into[j][h] = from + j < live ? *reinterpret_cast<const float2*>(p + h * 64) : make_float2(0.0f, 0.0f);
@@ -234,7 +239,7 @@ static bool decode_project_takes(int head_dim, int tokens, const void* w, long l
 template <int HD>
 static cudaError_t launch_merge_project(const float* partial, const __nv_bfloat16* w, long long ldw, float* summands,
                                         const int* row_token, const int* positions, int rows, int tokens, int heads,
-                                        int hidden, int max_splits, int window, int chunk, int slots, int split_keys,
+                                        int hidden, int max_splits, int window, int chunk, int keep, int slots, int split_keys,
                                         float minus_huge, const __nv_bfloat16* gate, long long gate_stride, int has_sink,
                                         float sink_score, const float* sink_heads, int* status, cudaStream_t stream) {
   const dim3 grid((hidden + kProjectColumns - 1) / kProjectColumns, heads);
@@ -247,7 +252,7 @@ static cudaError_t launch_merge_project(const float* partial, const __nv_bfloat1
       if (e != cudaSuccess) return e;                                                                                \
     }                                                                                                                \
     return launch_chained(kernel, grid, dim3(kProjectThreads), shared, stream, partial, w, ldw, summands, row_token,  \
-                          positions, rows, tokens, heads, hidden, max_splits, window, chunk, slots, split_keys, minus_huge,  \
+                          positions, rows, tokens, heads, hidden, max_splits, window, chunk, keep, slots, split_keys, minus_huge,  \
                           gate, gate_stride, has_sink, sink_score, sink_heads, status);                                                             \
   }
   if (tokens <= 8) GO(1)

@@ -73,7 +73,7 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
                      __nv_bfloat16* __restrict__ out, const int* __restrict__ block_tables, int max_pages,
                      const int* __restrict__ tile_request, const int* __restrict__ tile_start,
                      const int* __restrict__ tile_length, const int* __restrict__ positions, int heads,
-                     int kv_heads, int page_tokens, int num_pages, int window, int chunk, float scale, float softcap,
+                     int kv_heads, int page_tokens, int num_pages, int window, int chunk, int keep, float scale, float softcap,
                      const __nv_bfloat16* __restrict__ gate, long long gate_stride, int has_sink, float sink_log2, const float* __restrict__ sink_heads,
                      ScoreBias bias, int* status) {
   constexpr int CHUNKS = HD / 8;                      // 16-byte chunks per row
@@ -113,7 +113,7 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
   auto load_keys = [&](int key_tile, int stage) {
     const int row = tid >> 1, half = tid & 1;
     const int key = key_tile * kFlashKeys + row;
-    bool valid = key >= first_key && key <= last_pos;
+    bool valid = key_seen(key, last_pos, first_key, keep);
     int page = 0;
     if (valid) {
       page = table[key / page_tokens];
@@ -135,8 +135,8 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
     copy_async_commit();
   };
 
-  const int tile_begin = first_key / kFlashKeys, tile_end = last_pos / kFlashKeys;
-  load_keys(tile_begin, 0);
+  const KeyWalk walk = key_walk(first_key, last_pos, keep, kFlashKeys);
+  load_keys(walk.tile(0), 0);
 
   // Each warp owns 16 query rows; a thread owns rows g and g + 8 of them.
   const int g = lane >> 2, t = lane & 3;
@@ -162,10 +162,10 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
   }
   __syncthreads();
 
-  for (int kt = tile_begin; kt <= tile_end; ++kt) {
-    const int stage = (kt - tile_begin) & 1;
-    if (kt < tile_end) {
-      load_keys(kt + 1, stage ^ 1);
+  for (int step = 0; step < walk.count; ++step) {
+    const int stage = step & 1, kt = walk.tile(step);
+    if (step + 1 < walk.count) {
+      load_keys(walk.tile(step + 1), stage ^ 1);
       copy_async_wait<1>();
     } else {
       copy_async_wait<0>();
@@ -224,8 +224,8 @@ flash_prefill_kernel(const __nv_bfloat16* __restrict__ q, const __nv_bfloat16* _
 #pragma unroll
         for (int j = 0; j < 2; ++j) {
           const int key = key0 + nb * 8 + 2 * t + j;
-          const bool seen_lo = valid_lo && key <= pos_lo && key >= first_lo;
-          const bool seen_hi = valid_hi && key <= pos_hi && key >= first_hi;
+          const bool seen_lo = valid_lo && key_seen(key, pos_lo, first_lo, keep);
+          const bool seen_hi = valid_hi && key_seen(key, pos_hi, first_hi, keep);
           if (!seen_lo) s[nb][j] = -INFINITY;
           if (!seen_hi) s[nb][2 + j] = -INFINITY;
         }
@@ -319,7 +319,7 @@ template <int HD>
 static int launch_flash(const void* q, const void* cache, void* out, const int* block_tables, int max_pages,
                         const int* tile_request, const int* tile_start, const int* tile_length,
                         const int* positions, int tiles, int heads, int kv_heads, int page_tokens,
-                        int num_pages, int window, int chunk, float scale, const void* gate, long long gate_stride,
+                        int num_pages, int window, int chunk, int keep, float scale, const void* gate, long long gate_stride,
                         float softcap, int has_sink, float sink_score, const float* sink_heads, ScoreBias bias, int* status,
                         cudaStream_t stream) {
   const int shared = 4 * kFlashKeys * HD * 2;
@@ -330,7 +330,7 @@ static int launch_flash(const void* q, const void* cache, void* out, const int* 
   kernel<<<grid, kFlashThreads, shared, stream>>>(
       static_cast<const __nv_bfloat16*>(q), static_cast<const __nv_bfloat16*>(cache),
       static_cast<__nv_bfloat16*>(out), block_tables, max_pages, tile_request, tile_start, tile_length,
-      positions, heads, kv_heads, page_tokens, num_pages, window, chunk, scale, softcap,
+      positions, heads, kv_heads, page_tokens, num_pages, window, chunk, keep, scale, softcap,
       static_cast<const __nv_bfloat16*>(gate), gate_stride, has_sink, sink_score * 1.4426950408889634f, sink_heads, bias, status);
   return static_cast<int>(cudaGetLastError());
 }
@@ -352,7 +352,7 @@ MXB_API int mxb_flash_prefill_tile() { return 2 * kFlashQueries; }
 MXB_API int mxb_flash_prefill(const void* q, const void* cache, void* out, const int* block_tables,
                               int max_pages, const int* tile_request, const int* tile_start,
                               const int* tile_length, const int* positions, int tiles, int heads,
-                              int kv_heads, int head_dim, int page_tokens, int num_pages, int window, int chunk,
+                              int kv_heads, int head_dim, int page_tokens, int num_pages, int window, int chunk, int keep,
                               float scale, int dtype, const void* gate, long long gate_stride, float softcap,
                               int has_sink, float sink_score, const float* sink_heads, const float* bias_table,
                               int bias_far, int* status, cudaStream_t stream) {
@@ -362,9 +362,9 @@ MXB_API int mxb_flash_prefill(const void* q, const void* cache, void* out, const
   const ScoreBias bias = {bias_table, bias_far};
   if (head_dim == 64)
     return launch_flash<64>(q, cache, out, block_tables, max_pages, tile_request, tile_start, tile_length,
-                            positions, tiles, heads, kv_heads, page_tokens, num_pages, window, chunk, scale, gate, gate_stride, softcap, has_sink,
+                            positions, tiles, heads, kv_heads, page_tokens, num_pages, window, chunk, keep, scale, gate, gate_stride, softcap, has_sink,
                             sink_score, sink_heads, bias, status, stream);
   return launch_flash<128>(q, cache, out, block_tables, max_pages, tile_request, tile_start, tile_length,
-                           positions, tiles, heads, kv_heads, page_tokens, num_pages, window, chunk, scale, gate, gate_stride, softcap, has_sink,
+                           positions, tiles, heads, kv_heads, page_tokens, num_pages, window, chunk, keep, scale, gate, gate_stride, softcap, has_sink,
                             sink_score, sink_heads, bias, status, stream);
 }

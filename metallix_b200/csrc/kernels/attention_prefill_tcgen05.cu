@@ -75,7 +75,7 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
                              __nv_bfloat16* __restrict__ out, const int* __restrict__ block_tables, int max_pages,
                              const int* __restrict__ tile_request, const int* __restrict__ tile_start,
                              const int* __restrict__ tile_length, const int* __restrict__ positions, int heads,
-                             int kv_heads, int page_tokens, int num_pages, int window, int chunk, float scale, float softcap,
+                             int kv_heads, int page_tokens, int num_pages, int window, int chunk, int keep, float scale, float softcap,
                              int shared_bytes, float* __restrict__ partial, const __nv_bfloat16* __restrict__ gate,
                              long long gate_stride, int has_sink, float sink_log2, const float* __restrict__ sink_heads,
                              ScoreBias bias, int bias_bytes, int* status) {
@@ -128,11 +128,11 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
   // query tiles with many key tiles each: this way it still fills the GPU);
   // each block then leaves its unnormalised output, maximum and sum in
   // `partial` and a second kernel puts them together. A block's share may be empty.
-  const int all_begin = first_key / kFaKeys, all_end = last_pos / kFaKeys;   // all_end holds the tile's last position
-  const int all_tiles = all_end - all_begin + 1;
+  const KeyWalk walk = key_walk(first_key, last_pos, keep, kFaKeys);
+  const int all_tiles = walk.count, all_end = last_pos / kFaKeys;   // all_end holds the tile's last position
   const int shares = gridDim.z, share = blockIdx.z;
-  const int tile_begin = all_begin + static_cast<int>(static_cast<long long>(share) * all_tiles / shares);
-  const int key_tiles = all_begin + static_cast<int>(static_cast<long long>(share + 1) * all_tiles / shares) - tile_begin;
+  const int step_begin = static_cast<int>(static_cast<long long>(share) * all_tiles / shares);
+  const int key_tiles = static_cast<int>(static_cast<long long>(share + 1) * all_tiles / shares) - step_begin;
 
   if (threadIdx.x == 0) {
     barrier_init(q_full, 1);
@@ -194,9 +194,9 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
     constexpr int kNoPage = -0x40000000;
     const int beyond_cache = num_pages * 2 * kv_heads * page_tokens;
     auto page_of = [&](int i) {
-      const int page_key = (tile_begin + i) * kFaKeys + slot * page_tokens;
-      if (i < key_tiles && lane < copies && page_key <= last_pos && page_key + page_tokens > first_key &&
-          page_key / page_tokens < max_pages)
+      const int page_key = walk.tile(step_begin + i) * kFaKeys + slot * page_tokens;
+      if (i < key_tiles && lane < copies && page_key <= last_pos &&
+          (page_key + page_tokens > first_key || page_key < keep) && page_key / page_tokens < max_pages)
         return table[page_key / page_tokens];
       return kNoPage;
     };
@@ -211,9 +211,10 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
       const int box_row = page == kNoPage ? beyond_cache
                                           : ((page * 2 + (values ? 1 : 0)) * kv_heads + kv) * page_tokens;
       // rows [zero_from, zero_to) of the tile: the last page's rows behind the last position
-      const int zero_from = last_pos + 1 - (tile_begin + i) * kFaKeys;
-      const int zero_to = (last_pos / page_tokens + 1) * page_tokens - (tile_begin + i) * kFaKeys;
-      const bool tail = values && tile_begin + i == all_end && zero_from < zero_to;
+      const int key_tile = walk.tile(step_begin + i);
+      const int zero_from = last_pos + 1 - key_tile * kFaKeys;
+      const int zero_to = (last_pos / page_tokens + 1) * page_tokens - key_tile * kFaKeys;
+      const bool tail = values && key_tile == all_end && zero_from < zero_to;
       uint64_t* landing = tail ? v_tail : &full[stage];
       // K as soon as the scores that read this stage last are done, V when the P V product is.
       if (!barrier_wait(&empty[stage], ((i / stages) & 1) ^ 1, status)) { failed = 1; break; }
@@ -329,11 +330,11 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
 
     for (int i = 0; i < key_tiles; ++i) {
       const int buffer = i & 1;
-      const int key0 = (tile_begin + i) * kFaKeys + part * PART_KEYS;  // first key of this thread's share
+      const int key0 = walk.tile(step_begin + i) * kFaKeys + part * PART_KEYS;  // first key of this thread's share
       if (!barrier_wait(&s_full[buffer], (i >> 1) & 1, status) || failed) { ok = false; break; }
       tc_fence_after_sync();
       const uint32_t tmem_s = tmem_lane + buffer * Config::kScoreColumns + part * PART_KEYS;
-      const bool all_seen = key0 >= key_lo && key0 + PART_KEYS - 1 <= key_hi;
+      const bool all_seen = (key0 >= key_lo || key0 + PART_KEYS <= keep) && key0 + PART_KEYS - 1 <= key_hi;
       uint32_t raw[PART_KEYS];
       tc_load_32(tmem_s, raw);
       float s[PART_KEYS];
@@ -357,10 +358,11 @@ flash_prefill_tcgen05_kernel(const __grid_constant__ CUtensorMap map_q, const __
       if (all_seen) {
 #pragma unroll
         for (int j = 0; j < PART_KEYS; ++j) s[j] = __uint_as_float(raw[j]);
-      } else {
+      } else {   // of this thread's share: lo .. hi, and up to hi those ahead of `kept`
+        const int lo = key_lo - key0, hi = key_hi - key0, kept = keep - key0;
 #pragma unroll
         for (int j = 0; j < PART_KEYS; ++j)
-          s[j] = key0 + j >= key_lo && key0 + j <= key_hi ? __uint_as_float(raw[j]) : -INFINITY;
+          s[j] = j <= hi && (j >= lo || j < kept) ? __uint_as_float(raw[j]) : -INFINITY;
       }
       // Running maximum, already multiplied by scale * log2(e) (scale > 0 keeps the order).
       float max4[4] = {-INFINITY, -INFINITY, -INFINITY, -INFINITY};
@@ -500,7 +502,7 @@ template <int HD>
 static int launch_flash_tc(const void* q, const void* cache, void* out, const int* block_tables, int max_pages,
                            const int* tile_request, const int* tile_start, const int* tile_length,
                            const int* positions, int tokens, int tiles, int heads, int kv_heads, int page_tokens,
-                           int num_pages, int window, int chunk, float scale, int key_shares, float* partial,
+                           int num_pages, int window, int chunk, int keep, float scale, int key_shares, float* partial,
                            const void* gate, long long gate_stride, float softcap, int has_sink, float sink_score, const float* sink_heads,
                            ScoreBias bias, int* status, cudaStream_t stream) {
   using Config = FaConfig<HD>;
@@ -529,7 +531,7 @@ static int launch_flash_tc(const void* q, const void* cache, void* out, const in
   dim3 grid(heads, tiles, shared_out ? key_shares : 1);
   kernel<<<grid, kFaThreads, shared_bytes, stream>>>(
       map_q, map_cache, static_cast<__nv_bfloat16*>(out), block_tables, max_pages, tile_request, tile_start,
-      tile_length, positions, heads, kv_heads, page_tokens, num_pages, window, chunk, scale, softcap, shared_bytes,
+      tile_length, positions, heads, kv_heads, page_tokens, num_pages, window, chunk, keep, scale, softcap, shared_bytes,
       shared_out ? partial : nullptr, static_cast<const __nv_bfloat16*>(gate), gate_stride, has_sink, sink_log2, sink_heads,
       bias, bias_bytes, status);
   e = cudaGetLastError();
@@ -562,7 +564,7 @@ MXB_API int mxb_flash_prefill_tcgen05(const void* q, const void* cache, void* ou
                                       int max_pages, const int* tile_request, const int* tile_start,
                                       const int* tile_length, const int* positions, int tokens, int tiles,
                                       int heads, int kv_heads, int head_dim, int page_tokens, int num_pages,
-                                      int window, int chunk, float scale, int dtype, int key_shares, float* partial,
+                                      int window, int chunk, int keep, float scale, int dtype, int key_shares, float* partial,
                                       const void* gate, long long gate_stride, float softcap, int has_sink,
                                       float sink_score, const float* sink_heads, const float* bias_table, int bias_far,
                                       int* status, cudaStream_t stream) {
@@ -578,9 +580,9 @@ MXB_API int mxb_flash_prefill_tcgen05(const void* q, const void* cache, void* ou
   const ScoreBias bias = {bias_table, bias_far};
   if (head_dim == 64)
     return launch_flash_tc<64>(q, cache, out, block_tables, max_pages, tile_request, tile_start, tile_length,
-                               positions, tokens, tiles, heads, kv_heads, page_tokens, num_pages, window, chunk, scale,
+                               positions, tokens, tiles, heads, kv_heads, page_tokens, num_pages, window, chunk, keep, scale,
                                key_shares, partial, gate, gate_stride, softcap, has_sink, sink_score, sink_heads, bias, status, stream);
   return launch_flash_tc<128>(q, cache, out, block_tables, max_pages, tile_request, tile_start, tile_length,
-                              positions, tokens, tiles, heads, kv_heads, page_tokens, num_pages, window, chunk, scale,
+                              positions, tokens, tiles, heads, kv_heads, page_tokens, num_pages, window, chunk, keep, scale,
                               key_shares, partial, gate, gate_stride, softcap, has_sink, sink_score, sink_heads, bias, status, stream);
 }

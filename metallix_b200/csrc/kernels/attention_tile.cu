@@ -12,8 +12,8 @@
 // Replaces the reference's gather of the whole context plus
 // fast::scaled_dot_product_attention (crates/models/qwen/src/forward/paged.rs:329-342,
 // :1067-1076, :1176-1184): s = (q k^T) * scale, causal with the diagonal at the
-// query's own position, optional window (key > position - window) and chunk (key >= position - position % chunk), softmax
-// over keys, query head j reads key/value head j / (heads / kv_heads).
+// query's own position, optional window (key > position - window) and chunk (key >= position - position % chunk),
+// both widened by the first `keep` positions, softmax over keys, query head j reads key/value head j / (heads / kv_heads).
 //
 // Further parameters, each off by default: `softcap` c bounds a score to
 // (-c, c) ahead of the softmax, s <- c tanh(s / c); the pool may hold one plane
@@ -42,7 +42,7 @@ paged_attention_tile_kernel(const T* __restrict__ q, const T* __restrict__ cache
                             const int* __restrict__ tile_request, const int* __restrict__ tile_start,
                             const int* __restrict__ tile_length, const int* __restrict__ positions,
                             int heads, int kv_heads, int head_dim, int page_tokens, int num_pages,
-                            int window, int chunk, float scale, const T* __restrict__ gate, long long gate_stride,
+                            int window, int chunk, int keep, float scale, const T* __restrict__ gate, long long gate_stride,
                             int planes, int value_dim, float softcap, int gate_per_head, int has_sink, float sink_score, const float* sink_heads,
                             ScoreBias bias, int* status) {
   extern __shared__ float shared[];
@@ -76,15 +76,15 @@ paged_attention_tile_kernel(const T* __restrict__ q, const T* __restrict__ cache
 #pragma unroll
   for (int j = 0; j < DPT; ++j) acc[j] = 0.0f;
 
-  const int tile_begin = first_key / kTileKeys, tile_end = last_pos / kTileKeys;
-  for (int kt = tile_begin; kt <= tile_end; ++kt) {
-    const int key0 = kt * kTileKeys;
+  const KeyWalk walk = key_walk(first_key, last_pos, keep, kTileKeys);
+  for (int step = 0; step < walk.count; ++step) {
+    const int key0 = walk.tile(step) * kTileKeys;
     __syncthreads();  // the previous tile's K, V and P are no longer read
     for (int i = tid; i < kTileKeys * head_dim; i += kTileThreads) {
       const int kk = i / head_dim, d = i - kk * head_dim;
       const int key = key0 + kk;
       float kval = 0.0f, vval = 0.0f;
-      if (key >= first_key && key <= last_pos) {
+      if (key_seen(key, last_pos, first_key, keep)) {
         const int page = table[key / page_tokens];
         if (page < 0 || page >= num_pages) {
           atomicOr(status, kStatusBadPage);
@@ -110,7 +110,7 @@ paged_attention_tile_kernel(const T* __restrict__ q, const T* __restrict__ cache
       const float* qrow = sQ + r * head_dim;
       const float* krow = sK + c * (head_dim + 1);
       for (int d = 0; d < head_dim; ++d) dot = fmaf(qrow[d], krow[d], dot);
-      visible[j] = row_valid && key <= my_pos && key >= my_first;
+      visible[j] = row_valid && key_seen(key, my_pos, my_first, keep);
       dot *= scale;
       if (softcap > 0.0f) dot = softcap * tanhf(dot / softcap);
       if (bias.table != nullptr) dot += bias_at(bias.row(head), my_pos - key, bias.far);
@@ -166,7 +166,7 @@ template <typename T, int DPT>
 static int launch_tile(const void* q, const void* cache, void* out, const int* block_tables,
                        int max_pages, const int* tile_request, const int* tile_start,
                        const int* tile_length, const int* positions, int tiles, int heads,
-                       int kv_heads, int head_dim, int page_tokens, int num_pages, int window, int chunk,
+                       int kv_heads, int head_dim, int page_tokens, int num_pages, int window, int chunk, int keep,
                        float scale, const void* gate, long long gate_stride, int planes, int value_dim, float softcap,
                        int gate_per_head, int has_sink, float sink_score, const float* sink_heads, ScoreBias bias, int* status,
                        cudaStream_t stream) {
@@ -183,7 +183,7 @@ static int launch_tile(const void* q, const void* cache, void* out, const int* b
   kernel<<<grid, kTileThreads, shared, stream>>>(
       static_cast<const T*>(q), static_cast<const T*>(cache), static_cast<T*>(out), block_tables,
       max_pages, tile_request, tile_start, tile_length, positions, heads, kv_heads, head_dim,
-      page_tokens, num_pages, window, chunk, scale, static_cast<const T*>(gate), gate_stride, planes, value_dim, softcap,
+      page_tokens, num_pages, window, chunk, keep, scale, static_cast<const T*>(gate), gate_stride, planes, value_dim, softcap,
       gate_per_head, has_sink, sink_score, sink_heads, bias, status);
   return static_cast<int>(cudaGetLastError());
 }
@@ -200,7 +200,7 @@ MXB_API int mxb_paged_attention_tile(const void* q, const void* cache, void* out
                                      const int* tile_request, const int* tile_start,
                                      const int* tile_length, const int* positions, int tiles,
                                      int heads, int kv_heads, int head_dim, int page_tokens,
-                                     int num_pages, int window, int chunk, float scale, int dtype, const void* gate,
+                                     int num_pages, int window, int chunk, int keep, float scale, int dtype, const void* gate,
                                      long long gate_stride, int planes, int value_dim, float softcap,
                                      int gate_per_head, int has_sink, float sink_score, const float* sink_heads,
                                      const float* bias_table, int bias_far, int* status, cudaStream_t stream) {
@@ -210,7 +210,7 @@ MXB_API int mxb_paged_attention_tile(const void* q, const void* cache, void* out
   const ScoreBias bias = {bias_table, bias_far};
   if ((planes != 1 && planes != 2) || value_dim <= 0 || value_dim > head_dim) return static_cast<int>(cudaErrorInvalidValue);
 #define ARGS q, cache, out, block_tables, max_pages, tile_request, tile_start, tile_length, positions, \
-             tiles, heads, kv_heads, head_dim, page_tokens, num_pages, window, chunk, scale, gate, gate_stride, planes, value_dim, softcap, gate_per_head, has_sink, sink_score, sink_heads, bias, status, stream
+             tiles, heads, kv_heads, head_dim, page_tokens, num_pages, window, chunk, keep, scale, gate, gate_stride, planes, value_dim, softcap, gate_per_head, has_sink, sink_score, sink_heads, bias, status, stream
 #define DISPATCH(T)                                           \
   if (head_dim <= 16) return launch_tile<T, 2>(ARGS);         \
   if (head_dim <= 32) return launch_tile<T, 4>(ARGS);         \

@@ -70,6 +70,9 @@ __device__ __forceinline__ void prefetch_line(const void* p) { asm volatile("pre
 // sigmoid(gate[token * gate_stride + head * head_dim + d]), in float32.
 __device__ __forceinline__ float sigmoid_of(float g) { return 1.0f / (1.0f + expf(-g)); }
 
+// gelu in its exact form: z times the standard normal distribution at z.
+__device__ __forceinline__ float gelu_of(float z) { return 0.5f * z * (1.0f + erff(z * 0.7071067811865476f)); }
+
 // The activation of a gated feed-forward, act(gate) * up: silu(z) = z / (1 + e^-z), or the tanh form of
 // gelu, 0.5 z (1 + tanh(sqrt(2 / pi) (z + 0.044715 z^3))).
 // A third, with clamped halves: g = min(gate, limit), u = clamp(up, -limit, limit), g sigmoid(1.702 g) (u + 1).
@@ -117,6 +120,29 @@ __host__ __device__ __forceinline__ int first_visible_key(int pos, int window, i
     if (chunk_start > first) first = chunk_start;
   }
   return first;
+}
+
+// A third rule widens the first two: the first `keep` positions of a sequence
+// are seen by every query behind them, whatever the window. A query at `pos`
+// whose first key by window and chunk is `first` sees `key` if
+__host__ __device__ __forceinline__ bool key_seen(int key, int pos, int first, int keep) {
+  return key <= pos && (key >= first || key < keep);
+}
+
+// The key tiles of `size` absolute positions that a run of queries walks over: those that hold kept keys (the first
+// `kept` of a sequence), then the window's, up to the tile of the last position. The `skip` tiles between the two
+// are left out, so step i of the walk is tile i + skip from step `kept` on, and tile i before.
+struct KeyWalk {
+  int kept, skip, count;
+  __host__ __device__ __forceinline__ int tile(int i) const { return i < kept ? i : i + skip; }
+};
+__host__ __device__ __forceinline__ KeyWalk key_walk(int first_key, int last_pos, int keep, int size) {
+  const int first_tile = first_key / size;
+  KeyWalk walk;
+  walk.kept = (keep + size - 1) / size;
+  walk.skip = first_tile > walk.kept ? first_tile - walk.kept : 0;
+  walk.count = last_pos / size + 1 - walk.skip;
+  return walk;
 }
 
 // Programmatic dependent launch: a kernel launched through launch_chained()

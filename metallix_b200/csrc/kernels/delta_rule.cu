@@ -1,7 +1,8 @@
 // Matrix-state recurrences over the tokens of a request, the state kept per
 // request in the cache's slots, float32 throughout: the gated delta rule with
-// one decay per head and key channel, the same with one decay per head, and
-// the state-space dual (Mamba-2), which writes without looking first.
+// one decay per head and key channel, the same with one decay per head,
+// the state-space dual (Mamba-2), which writes without looking first, and
+// lightning attention, whose decay per head is a constant.
 //
 // Per head, with key width D and value width V, a request carries a matrix
 // S [D, V]. A token brings q, k (D values each, from one of G groups that
@@ -17,6 +18,10 @@
 // come, dt = softplus(s + bias) in place of beta, g = exp(-a_h dt), and
 //
 //   S <- g S + k (dt v)^T;   o = S^T q + skip_h v
+//
+// Lightning attention takes silu(q), silu(k), silu(v) and nothing else:
+//
+//   S <- g_h S + k v^T;   o = S^T q
 //
 // Every value column of S goes its own way: column j needs only v_j and what
 // all columns share (qn, kn, g, beta). A block owns some of the columns of
@@ -35,7 +40,9 @@
 
 namespace mxb {
 
-enum DeltaMode : int { kDeltaChannel = 0, kDeltaHead = 1, kDeltaDual = 2 };
+enum DeltaMode : int { kDeltaChannel = 0, kDeltaHead = 1, kDeltaDual = 2, kDeltaConstant = 3 };
+// the modes that write without looking at the state first
+__host__ __device__ constexpr bool delta_blind(int mode) { return mode == kDeltaDual || mode == kDeltaConstant; }
 constexpr int kDeltaMaxWarps = 8;     // tokens of a batch: one warp prepares each (a block of fewer warps takes fewer)
 
 // Where channel d of a shared vector lies: every lane's quarter starts 4 floats further than a
@@ -44,12 +51,13 @@ template <int DPT>
 __device__ __forceinline__ int delta_slot(int d) { return d + (d / DPT) * 4; }
 
 template <typename T> struct alignas(4 * sizeof(T)) DeltaFour { T v[4]; };   // four neighbouring values, one access
+__device__ __forceinline__ float delta_silu(float z) { return z * sigmoid_of(z); }
 __device__ __forceinline__ float delta_softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 
 // LANES lanes share a value column, each with DPT of its key channels; COLS neighbouring columns a thread.
 // MODE: see DeltaMode; `step_pre` is float32 [.., heads * dim] with a decay per channel, else of T with one value per head.
 template <typename T, int DPT, int LANES, int COLS, int MODE>
-__global__ void __launch_bounds__(MODE == kDeltaDual ? 256 : 512)   // four columns a thread want more registers each
+__global__ void __launch_bounds__(delta_blind(MODE) ? 256 : 512)   // four columns a thread want more registers each
 delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off, int v_off,
                   const T* __restrict__ beta_pre, long long ldb, int b_off,
                   const void* __restrict__ step_pre, long long lds, const float* __restrict__ step_bias,
@@ -91,7 +99,7 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
 #pragma unroll
   for (int i = 0; i < NL; ++i) {
     const int d = lane + 32 * i;
-    bias[i] = !PER_CHANNEL ? step_bias[head] : (d < dim ? step_bias[head * dim + d] : 0.0f);
+    bias[i] = MODE == kDeltaConstant ? 0.0f : !PER_CHANNEL ? step_bias[head] : (d < dim ? step_bias[head * dim + d] : 0.0f);
   }
   const float head_skip = MODE == kDeltaDual ? skip[head] : 0.0f;
   // this thread's quarter of its columns of S
@@ -142,8 +150,8 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
         raw_k[i] = d < dim ? k_row[d] : none;
         if (PER_CHANNEL) raw_step[PER_CHANNEL ? i : 0] = d < dim ? step_row[d] : 0.0f;
       }
-      if (!PER_CHANNEL) raw_head_step = static_cast<const T*>(step_pre)[t * lds + head];
-      if (MODE != kDeltaDual) raw_beta = beta_pre[t * ldb + b_off + head];
+      if (!PER_CHANNEL && MODE != kDeltaConstant) raw_head_step = static_cast<const T*>(step_pre)[t * lds + head];
+      if (!delta_blind(MODE)) raw_beta = beta_pre[t * ldb + b_off + head];
     }
     const T* v_rows = qkv + (static_cast<long long>(first + base)) * ld + v_off + head * vdim + column;
 #pragma unroll
@@ -167,13 +175,13 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
       float qq = 0.0f, kk = 0.0f, qk = 0.0f, q_in[NL], k_in[NL];
 #pragma unroll
       for (int i = 0; i < NL; ++i) {
-        q_in[i] = to_float(raw_q[i]);
-        k_in[i] = to_float(raw_k[i]);
+        q_in[i] = MODE == kDeltaConstant ? delta_silu(to_float(raw_q[i])) : to_float(raw_q[i]);
+        k_in[i] = MODE == kDeltaConstant ? delta_silu(to_float(raw_k[i])) : to_float(raw_k[i]);
         qq = fmaf(q_in[i], q_in[i], qq); kk = fmaf(k_in[i], k_in[i], kk); qk = fmaf(q_in[i], k_in[i], qk);
       }
       qk = warp_sum(qk);
       float q_unit = 1.0f, k_unit = 1.0f;
-      if (MODE != kDeltaDual) {
+      if (!delta_blind(MODE)) {
         qq = warp_sum(qq); kk = warp_sum(kk);
         q_unit = rsqrtf(qq + 1e-6f) * q_scale;
         k_unit = rsqrtf(kk + 1e-6f);
@@ -189,9 +197,9 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
         }
       }
       if (lane == 0) {
-        const float step = PER_CHANNEL ? 0.0f : delta_softplus(to_float(raw_head_step) + bias[0]);
-        if (!PER_CHANNEL) s_decay[warp] = expf(-head_rate * step);
-        s_beta[warp] = MODE == kDeltaDual ? step : sigmoid_of(to_float(raw_beta));
+        const float step = PER_CHANNEL || MODE == kDeltaConstant ? 0.0f : delta_softplus(to_float(raw_head_step) + bias[0]);
+        if (!PER_CHANNEL) s_decay[warp] = MODE == kDeltaConstant ? head_rate : expf(-head_rate * step);
+        s_beta[warp] = MODE == kDeltaConstant ? 1.0f : MODE == kDeltaDual ? step : sigmoid_of(to_float(raw_beta));
         s_qk[warp] = qk * q_unit * k_unit;
       }
     }
@@ -199,7 +207,8 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
 #pragma unroll
     for (int j = 0; j < kDeltaMaxWarps; ++j)
 #pragma unroll
-      for (int c = 0; c < COLS; ++c) v[j][c] = to_float(next_v[j][c]);
+      for (int c = 0; c < COLS; ++c)
+        v[j][c] = MODE == kDeltaConstant ? delta_silu(to_float(next_v[j][c])) : to_float(next_v[j][c]);
     __syncthreads();
     if (base + warps < length) fetch(base + warps);   // on its way while this batch is walked through
 #pragma unroll
@@ -222,7 +231,7 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
 #pragma unroll
         for (int c = 0; c < COLS; ++c) {
           s[c][i] *= g.x; s[c][i + 1] *= g.y; s[c][i + 2] *= g.z; s[c][i + 3] *= g.w;
-          if (MODE != kDeltaDual) {
+          if (!delta_blind(MODE)) {
             k_dot[c] = fmaf(k.x, s[c][i], k_dot[c]); k_dot[c] = fmaf(k.y, s[c][i + 1], k_dot[c]);
             k_dot[c] = fmaf(k.z, s[c][i + 2], k_dot[c]); k_dot[c] = fmaf(k.w, s[c][i + 3], k_dot[c]);
           }
@@ -233,7 +242,7 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
       float u[COLS];
 #pragma unroll
       for (int c = 0; c < COLS; ++c) {
-        if (MODE != kDeltaDual) {
+        if (!delta_blind(MODE)) {
 #pragma unroll
           for (int offset = 1; offset < LANES; offset <<= 1) {   // over the lanes that share the column
             k_dot[c] += __shfl_xor_sync(0xffffffffu, k_dot[c], offset);
@@ -254,7 +263,7 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
         }
       }
       float* out_row = out + (static_cast<long long>(first + base + j)) * (static_cast<long long>(heads) * vdim) + head * vdim + column;
-      if (MODE == kDeltaDual && COLS == 4) {
+      if (delta_blind(MODE) && COLS == 4) {
         // Four columns over LANES lanes: each exchange halves the columns a lane still adds up, so that a quarter of
         // the lanes ends with each column's sum instead of every lane with all four.
         const bool upper = (part & (LANES / 2)) != 0, odd = (part & (LANES / 4)) != 0;
@@ -312,7 +321,8 @@ MXB_API int mxb_delta_rule_max_dim() { return 256; }
 // mode 0: the above. mode 1: one decay per head; step_pre is [tokens, lds] of `dtype` with one pre-activation per
 // head, step_bias [heads]. mode 2, the state-space dual: as mode 1, with q, k and v taken as they come (C, B, x),
 // softplus(step) in place of sigmoid(beta), no look at the state before the write, and skip (float32 [heads]) times v
-// added to what is read; beta_pre is not read.
+// added to what is read; beta_pre is not read. mode 3, lightning attention: q, k and v pass silu on their way in, the
+// decay is rate[head] itself (in (0, 1]), the write strength 1; beta_pre, step_pre, step_bias and skip are not read.
 MXB_API int mxb_delta_rule(const void* qkv, long long ld, int q_off, int k_off, int v_off, const void* beta_pre,
                            long long ldb, int b_off, const void* step_pre, long long lds, const float* step_bias,
                            const float* rate, const float* skip, int mode, float* state, long long slot_stride, int num_slots,
@@ -320,7 +330,7 @@ MXB_API int mxb_delta_rule(const void* qkv, long long ld, int q_off, int k_off, 
                            int rows, int heads, int groups, int dim, int vdim, int dtype, int longest, int* status,
                            cudaStream_t stream) {
   if (rows <= 0) return 0;
-  if (mode < kDeltaChannel || mode > kDeltaDual || (mode == kDeltaDual) != (skip != nullptr))
+  if (mode < kDeltaChannel || mode > kDeltaConstant || (mode == kDeltaDual) != (skip != nullptr))
     return static_cast<int>(cudaErrorInvalidValue);
   if (heads <= 0 || groups <= 0 || heads % groups != 0 || dim <= 0 || dim > mxb_delta_rule_max_dim() || vdim <= 0)
     return static_cast<int>(cudaErrorInvalidValue);
@@ -331,11 +341,11 @@ MXB_API int mxb_delta_rule(const void* qkv, long long ld, int q_off, int k_off, 
   const int step = 32 / lanes;                                   // columns of a warp
   // The dual has no chain from token to token but the decay, so a thread takes four columns: what is read from shared
   // memory serves four, and the sums over the lanes cost a third of the exchanges.
-  const int cols = mode == kDeltaDual ? 4 : 1;                   // columns of a thread
+  const int cols = delta_blind(mode) ? 4 : 1;                   // columns of a thread
   int columns = ((vdim + cols * step - 1) / (cols * step)) * step;     // ... of a block, in units of `cols`
   // A step of single tokens (`longest`, the most tokens of any row, if the caller knows it; 0: unknown) is one
   // chain of trips to memory per block: small blocks, several of them resident on an SM, overlap their chains.
-  const int most = (longest > 0 && longest < 8 ? 128 : (mode == kDeltaDual ? 256 : 512)) / lanes;
+  const int most = (longest > 0 && longest < 8 ? 128 : (delta_blind(mode) ? 256 : 512)) / lanes;
   if (columns > most) columns = most;
   const int units = (vdim + cols - 1) / cols;
   while (columns > 2 * step && columns >= 32 &&
@@ -344,13 +354,14 @@ MXB_API int mxb_delta_rule(const void* qkv, long long ld, int q_off, int k_off, 
   columns = ((columns + step - 1) / step) * step;
   const dim3 grid(rows, heads, (units + columns - 1) / columns), block(columns * lanes);
 #define LAUNCH_MODE(T, DPT, LANES, MODE)                                                                            \
-  delta_rule_kernel<T, DPT, LANES, MODE == kDeltaDual ? 4 : 1, MODE><<<grid, block, 0, stream>>>(static_cast<const T*>(qkv), ld, q_off, k_off,      \
+  delta_rule_kernel<T, DPT, LANES, delta_blind(MODE) ? 4 : 1, MODE><<<grid, block, 0, stream>>>(static_cast<const T*>(qkv), ld, q_off, k_off,      \
       v_off, static_cast<const T*>(beta_pre), ldb, b_off, step_pre, lds, step_bias, rate, skip, state, slot_stride, \
       num_slots, row_start, row_length, request_slots, out, heads, groups, dim, vdim, status)
 #define LAUNCH(T, DPT, LANES)                                        \
   if (mode == kDeltaChannel) LAUNCH_MODE(T, DPT, LANES, kDeltaChannel);   \
   else if (mode == kDeltaHead) LAUNCH_MODE(T, DPT, LANES, kDeltaHead);    \
-  else LAUNCH_MODE(T, DPT, LANES, kDeltaDual)
+  else if (mode == kDeltaDual) LAUNCH_MODE(T, DPT, LANES, kDeltaDual);    \
+  else LAUNCH_MODE(T, DPT, LANES, kDeltaConstant)
 #define BY_DIM(T)                                                   \
   if (lanes == 4 && per_lane == 4) { LAUNCH(T, 4, 4); }             \
   else if (lanes == 4) { LAUNCH(T, 8, 4); }                         \

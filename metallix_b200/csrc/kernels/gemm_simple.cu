@@ -168,22 +168,26 @@ MXB_API int mxb_silu_mul(void* out, const void* gate_up, int dtype, long long to
 }
 
 namespace mxb {
-// out = max(x, 0)^2: the activation of a feed-forward without a gate, float32 inside.
+// The activation of a feed-forward without a gate, float32 inside: max(x, 0)^2, or gelu in its exact form.
+__device__ __forceinline__ float plain_activation(float x, int gelu) {
+  if (gelu) return gelu_of(x);
+  const float v = fmaxf(x, 0.0f);
+  return v * v;
+}
 template <typename T>
-__global__ void relu_squared_kernel(T* __restrict__ out, const T* __restrict__ x, size_t count) {
+__global__ void plain_activation_kernel(T* __restrict__ out, const T* __restrict__ x, size_t count, int gelu) {
   chain_release();
   for (size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < count;
-       i += static_cast<size_t>(gridDim.x) * blockDim.x) {
-    const float v = fmaxf(to_float(x[i]), 0.0f);
-    out[i] = from_float<T>(v * v);
-  }
+       i += static_cast<size_t>(gridDim.x) * blockDim.x)
+    out[i] = from_float<T>(plain_activation(to_float(x[i]), gelu));
 }
 }  // namespace mxb
 
 namespace mxb {
 // Eight bfloat16 values per thread (16-byte loads and stores).
-__global__ void relu_squared_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ x,
-                                           size_t groups) {
+template <int GELU>
+__global__ void plain_activation_bf16x8_kernel(__nv_bfloat16* __restrict__ out, const __nv_bfloat16* __restrict__ x,
+                                               size_t groups) {
   chain_release();
   for (size_t i = static_cast<size_t>(blockIdx.x) * blockDim.x + threadIdx.x; i < groups;
        i += static_cast<size_t>(gridDim.x) * blockDim.x) {
@@ -192,8 +196,8 @@ __global__ void relu_squared_bf16x8_kernel(__nv_bfloat16* __restrict__ out, cons
     uint32_t ow[4];
 #pragma unroll
     for (int j = 0; j < 4; ++j) {
-      const float a = fmaxf(__uint_as_float(in[j] << 16), 0.0f), b = fmaxf(__uint_as_float(in[j] & 0xffff0000u), 0.0f);
-      __nv_bfloat162 packed = __floats2bfloat162_rn(a * a, b * b);
+      __nv_bfloat162 packed = __floats2bfloat162_rn(plain_activation(__uint_as_float(in[j] << 16), GELU),
+                                                    plain_activation(__uint_as_float(in[j] & 0xffff0000u), GELU));
       ow[j] = *reinterpret_cast<uint32_t*>(&packed);
     }
     *reinterpret_cast<uint4*>(out + i * 8) = make_uint4(ow[0], ow[1], ow[2], ow[3]);
@@ -201,25 +205,27 @@ __global__ void relu_squared_bf16x8_kernel(__nv_bfloat16* __restrict__ out, cons
 }
 }  // namespace mxb
 
-MXB_API int mxb_relu_squared(void* out, const void* x, long long count, int dtype, cudaStream_t stream) {
+// gelu 0: max(x, 0)^2; 1: gelu(x) in its exact form.
+MXB_API int mxb_plain_activation(void* out, const void* x, long long count, int dtype, int gelu, cudaStream_t stream) {
   if (count <= 0) return 0;
   if (dtype == mxb::kBF16 && count % 8 == 0 && reinterpret_cast<uintptr_t>(out) % 16 == 0 &&
       reinterpret_cast<uintptr_t>(x) % 16 == 0) {
     const size_t groups = static_cast<size_t>(count) / 8;
     size_t wide = (groups + 255) / 256;
     if (wide > 148 * 32) wide = 148 * 32;
-    mxb::relu_squared_bf16x8_kernel<<<static_cast<unsigned>(wide), 256, 0, stream>>>(
+    auto kernel = gelu ? mxb::plain_activation_bf16x8_kernel<1> : mxb::plain_activation_bf16x8_kernel<0>;
+    kernel<<<static_cast<unsigned>(wide), 256, 0, stream>>>(
         static_cast<__nv_bfloat16*>(out), static_cast<const __nv_bfloat16*>(x), groups);
     return static_cast<int>(cudaGetLastError());
   }
   long long blocks = (count + 255) / 256;
   if (blocks > 148 * 16) blocks = 148 * 16;
   if (dtype == mxb::kF32)
-    mxb::relu_squared_kernel<float><<<static_cast<unsigned>(blocks), 256, 0, stream>>>(
-        static_cast<float*>(out), static_cast<const float*>(x), static_cast<size_t>(count));
+    mxb::plain_activation_kernel<float><<<static_cast<unsigned>(blocks), 256, 0, stream>>>(
+        static_cast<float*>(out), static_cast<const float*>(x), static_cast<size_t>(count), gelu);
   else if (dtype == mxb::kBF16)
-    mxb::relu_squared_kernel<__nv_bfloat16><<<static_cast<unsigned>(blocks), 256, 0, stream>>>(
-        static_cast<__nv_bfloat16*>(out), static_cast<const __nv_bfloat16*>(x), static_cast<size_t>(count));
+    mxb::plain_activation_kernel<__nv_bfloat16><<<static_cast<unsigned>(blocks), 256, 0, stream>>>(
+        static_cast<__nv_bfloat16*>(out), static_cast<const __nv_bfloat16*>(x), static_cast<size_t>(count), gelu);
   else
     return static_cast<int>(cudaErrorInvalidValue);
   return static_cast<int>(cudaGetLastError());

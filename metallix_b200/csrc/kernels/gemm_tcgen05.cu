@@ -22,7 +22,7 @@ constexpr int kTcM = 128;     // rows of a tile
 constexpr int kTcK = 64;      // k per stage: 64 bfloat16 = one 128-byte swizzle row
 constexpr int kTcThreads = 192;
 
-enum TcEpilogue : int { kTcStoreBf16 = 0, kTcStoreF32 = 1, kTcSwiGLU = 2, kTcReluSquared = 3, kTcGeGLU = 4, kTcClampedGLU = 5 };
+enum TcEpilogue : int { kTcStoreBf16 = 0, kTcStoreF32 = 1, kTcSwiGLU = 2, kTcReluSquared = 3, kTcGeGLU = 4, kTcClampedGLU = 5, kTcGelu = 6 };
 // the epilogues that take a tile of gate rows beside a tile of up rows: act(gate) * up (silu, or the tanh form of gelu), or the product of clamped halves
 __host__ __device__ constexpr bool tc_gated(int epilogue) { return epilogue == kTcSwiGLU || epilogue == kTcGeGLU || epilogue == kTcClampedGLU; }
 
@@ -46,12 +46,13 @@ template <int BN, int STAGES_> struct TcConfig {
 // tile_group[i]; a row tile whose entry is negative is left out by every warp
 // alike. The rows of A are then tokens sorted by the expert they go to, each
 // expert's rows padded to whole tiles. kTcReluSquared stores max(c, 0)^2 in
-// bfloat16.
+// bfloat16, kTcGelu gelu(s c) in its exact form, s being row_scale[row] (1
+// without the array): the weight of an expert's input.
 template <int BN, int EPI, int STAGES_>
 __global__ void __launch_bounds__(kTcThreads)
 gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
                     void* __restrict__ out, int m, int n, int k, long long ldo, const int* __restrict__ tile_group,
-                    int group_rows, float limit, int* status) {
+                    int group_rows, float limit, const float* __restrict__ row_scale, int* status) {
   using Config = TcConfig<BN, STAGES_>;
   constexpr int STAGES = Config::kStages;
   constexpr int OUT_COLUMNS = tc_gated(EPI) ? BN / 2 : BN;  // output columns of a tile
@@ -163,6 +164,7 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
       if (failed) break;
       asm volatile("tcgen05.fence::after_thread_sync;\n" ::: "memory");
       const int row = m0 + lane_base + lane;
+      const float scale = EPI == kTcGelu && row_scale != nullptr && row < m ? row_scale[row] : 1.0f;
       const uint32_t tmem_row = tmem_base + buffer * BN + (static_cast<uint32_t>(lane_base) << 16);
 #pragma unroll 1
       for (int c = 0; c < OUT_COLUMNS; c += 32) {
@@ -185,6 +187,9 @@ gemm_tcgen05_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_cons
             const float u = fmaxf(__uint_as_float(acc[i]), 0.0f);
             values[i] = u * u;
           }
+        } else if (EPI == kTcGelu) {
+#pragma unroll
+          for (int i = 0; i < 32; ++i) values[i] = gelu_of(scale * __uint_as_float(acc[i]));
         } else {
 #pragma unroll
           for (int i = 0; i < 32; ++i) values[i] = __uint_as_float(acc[i]);
@@ -246,8 +251,8 @@ int g_tc_bn = 0, g_tc_deep = -1;  // tuning overrides: tile width, deep (1) or s
 
 template <int BN, int EPI, int STAGES_>
 static int launch_tc_staged(const CUtensorMap& map_a, const CUtensorMap& map_b, void* out, int m, int n, int k,
-                            long long ldo, const int* tile_group, int group_rows, float limit, int* status,
-                            cudaStream_t stream) {
+                            long long ldo, const int* tile_group, int group_rows, float limit, const float* row_scale,
+                            int* status, cudaStream_t stream) {
   using Config = TcConfig<BN, STAGES_>;
   auto kernel = gemm_tcgen05_kernel<BN, EPI, STAGES_>;
   cudaError_t e = cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, Config::kSharedBytes);
@@ -262,7 +267,7 @@ static int launch_tc_staged(const CUtensorMap& map_a, const CUtensorMap& map_b, 
   }
   dim3 grid(tiles < sm_count ? tiles : sm_count);  // one block per SM walks over the tiles
   kernel<<<grid, kTcThreads, Config::kSharedBytes, stream>>>(map_a, map_b, out, m, n, k, ldo, tile_group, group_rows,
-                                                             limit, status);
+                                                             limit, row_scale, status);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -271,12 +276,12 @@ static int launch_tc_staged(const CUtensorMap& map_a, const CUtensorMap& map_b, 
 template <int BN, int EPI>
 static int launch_tc(const CUtensorMap& map_a, const CUtensorMap& map_b, void* out, int m, int n, int k,
                      long long ldo, int* status, cudaStream_t stream, const int* tile_group = nullptr,
-                     int group_rows = 0, float limit = 0.0f) {
+                     int group_rows = 0, float limit = 0.0f, const float* row_scale = nullptr) {
   constexpr int deep = BN >= 256 ? 4 : (BN >= 128 ? 6 : 8);
   const bool shallow = g_tc_deep == 0;
   if (shallow)
-    return launch_tc_staged<BN, EPI, deep / 2>(map_a, map_b, out, m, n, k, ldo, tile_group, group_rows, limit, status, stream);
-  return launch_tc_staged<BN, EPI, deep>(map_a, map_b, out, m, n, k, ldo, tile_group, group_rows, limit, status, stream);
+    return launch_tc_staged<BN, EPI, deep / 2>(map_a, map_b, out, m, n, k, ldo, tile_group, group_rows, limit, row_scale, status, stream);
+  return launch_tc_staged<BN, EPI, deep>(map_a, map_b, out, m, n, k, ldo, tile_group, group_rows, limit, row_scale, status, stream);
 }
 
 }  // namespace mxb
@@ -291,7 +296,7 @@ MXB_API int mxb_gemm_tcgen05_supported(int m, int n, int k, long long lda, long 
 
 // epilogue: 0 bfloat16 out[m, n], 1 float32 out[m, n], 2 SwiGLU: w is
 // [2 * n, k] (gate rows, then up rows) and out is bfloat16 [m, n]; 4 the same
-// with the tanh form of gelu in place of silu; 5 min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, -limit, limit) + 1).
+// with the tanh form of gelu in place of silu; 6 bfloat16 gelu(c) in its exact form; 5 min(g, limit) sigmoid(1.702 min(g, limit)) (clamp(u, -limit, limit) + 1).
 MXB_API int mxb_gemm_tcgen05(void* out, const void* a, const void* w, int m, int n, int k, long long lda,
                              long long ldw, long long ldo, int epilogue, float limit, int* status, cudaStream_t stream) {
   if (!mxb_gemm_tcgen05_supported(m, n, k, lda, ldw)) return static_cast<int>(cudaErrorInvalidValue);
@@ -335,6 +340,11 @@ MXB_API int mxb_gemm_tcgen05(void* out, const void* a, const void* w, int m, int
     if (bn == 128) return launch_tc<128, kTcStoreF32>(map_a, map_b, out, m, n, k, ldo, status, stream);
     return launch_tc<64, kTcStoreF32>(map_a, map_b, out, m, n, k, ldo, status, stream);
   }
+  if (epilogue == kTcGelu) {
+    if (bn == 256) return launch_tc<256, kTcGelu>(map_a, map_b, out, m, n, k, ldo, status, stream);
+    if (bn == 128) return launch_tc<128, kTcGelu>(map_a, map_b, out, m, n, k, ldo, status, stream);
+    return launch_tc<64, kTcGelu>(map_a, map_b, out, m, n, k, ldo, status, stream);
+  }
   if (epilogue != kTcStoreBf16) return static_cast<int>(cudaErrorInvalidValue);
   if (bn == 256) return launch_tc<256, kTcStoreBf16>(map_a, map_b, out, m, n, k, ldo, status, stream);
   if (bn == 128) return launch_tc<128, kTcStoreBf16>(map_a, map_b, out, m, n, k, ldo, status, stream);
@@ -348,10 +358,10 @@ MXB_API int mxb_gemm_tcgen05(void* out, const void* a, const void* w, int m, int
 // tile is left out); out is [m, n] with n <= group_rows. epilogue: 1 float32,
 // 3 bfloat16 max(c, 0)^2, 0 bfloat16, 2 SwiGLU: every group's matrix is
 // [2 * n, k], its gate rows and then its up rows (group_rows = 2 n), and out is
-// bfloat16 silu(gate) * up.
+// bfloat16 silu(gate) * up; 6 bfloat16 gelu(row_scale[row] * c), row_scale being float32 [m] or null (1).
 MXB_API int mxb_gemm_tcgen05_grouped(void* out, const void* a, const void* w, const int* tile_group, int m, int n,
                                      int k, int groups, int group_rows, long long lda, long long ldw, long long ldo,
-                                     int epilogue, int* status, cudaStream_t stream) {
+                                     int epilogue, const float* row_scale, int* status, cudaStream_t stream) {
   if (!mxb_gemm_tcgen05_supported(m, n, k, lda, ldw) || groups < 1 || n > group_rows || tile_group == nullptr)
     return static_cast<int>(cudaErrorInvalidValue);
   if ((reinterpret_cast<uintptr_t>(a) & 15) || (reinterpret_cast<uintptr_t>(w) & 15)) return static_cast<int>(cudaErrorInvalidValue);
@@ -365,11 +375,12 @@ MXB_API int mxb_gemm_tcgen05_grouped(void* out, const void* a, const void* w, co
       !make_map(&map_b, w, static_cast<int>(w_rows), k, ldw, epilogue == kTcSwiGLU ? bn / 2 : bn))
     return static_cast<int>(cudaErrorInvalidValue);
 #define GROUPED(EPI)                                                                                             \
-  if (bn == 256) return launch_tc<256, EPI>(map_a, map_b, out, m, n, k, ldo, status, stream, tile_group, group_rows); \
-  if (bn == 128) return launch_tc<128, EPI>(map_a, map_b, out, m, n, k, ldo, status, stream, tile_group, group_rows); \
-  return launch_tc<64, EPI>(map_a, map_b, out, m, n, k, ldo, status, stream, tile_group, group_rows);
+  if (bn == 256) return launch_tc<256, EPI>(map_a, map_b, out, m, n, k, ldo, status, stream, tile_group, group_rows, 0.0f, row_scale); \
+  if (bn == 128) return launch_tc<128, EPI>(map_a, map_b, out, m, n, k, ldo, status, stream, tile_group, group_rows, 0.0f, row_scale); \
+  return launch_tc<64, EPI>(map_a, map_b, out, m, n, k, ldo, status, stream, tile_group, group_rows, 0.0f, row_scale);
   if (epilogue == kTcStoreF32) { GROUPED(kTcStoreF32) }
   if (epilogue == kTcReluSquared) { GROUPED(kTcReluSquared) }
+  if (epilogue == kTcGelu) { GROUPED(kTcGelu) }
   if (epilogue == kTcStoreBf16) { GROUPED(kTcStoreBf16) }
   if (epilogue == kTcSwiGLU) { GROUPED(kTcSwiGLU) }
 #undef GROUPED

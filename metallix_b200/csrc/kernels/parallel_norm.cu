@@ -2,13 +2,14 @@
 // both sublayers' norms of the new x in one pass over the row. The two norms
 // share the row's mean square (they differ in their weights only):
 //
-//   x += m * (a + b)                    float32, in place (a, b optional)
+//   x += m * (a + b) + c                float32, in place (a, b, c optional)
 //   r = rsqrt(mean(x^2) + eps)
 //   y1 = x r w1,   y2 = x r w2          (y2 optional)
 //
 // a and b are what the previous layer's mixer and feed-forward left (float32
 // or bfloat16, each in its own type); the sum a + b is formed in float32
-// before it is scaled. One block per row, four values a thread at a time; the
+// before it is scaled; c is float32 (the embedding output, where a pass over the layers
+// begins with it). One block per row, four values a thread at a time; the
 // thread's first four values stay in registers between the two passes.
 #include "common.cuh"
 
@@ -31,7 +32,7 @@ __device__ __forceinline__ void pn_store4(__nv_bfloat16* p, float4 v) {
 template <typename TOut>
 __global__ void __launch_bounds__(256)
 pair_add_rmsnorm_kernel(float* __restrict__ x, const void* __restrict__ a, int a_code, const void* __restrict__ b,
-                        int b_code, float m, const float* __restrict__ w1, const float* __restrict__ w2,
+                        int b_code, float m, const float* __restrict__ c, const float* __restrict__ w1, const float* __restrict__ w2,
                         TOut* __restrict__ y1, TOut* __restrict__ y2, const int* __restrict__ rows_index, int size,
                         float eps) {
   __shared__ float scratch[33];
@@ -47,10 +48,11 @@ pair_add_rmsnorm_kernel(float* __restrict__ x, const void* __restrict__ a, int a
   float* row = behind_wait(x) + src * size;
   a = behind_wait(a);
   b = behind_wait(b);
+  c = behind_wait(c);
   float sum = 0.0f;
   for (int i = first; i < size; i += blockDim.x * 4) {
     float4 v = *reinterpret_cast<const float4*>(row + i);
-    if (a != nullptr || b != nullptr) {
+    if (a != nullptr || b != nullptr || c != nullptr) {
       float4 d = make_float4(0.0f, 0.0f, 0.0f, 0.0f);
       if (a != nullptr) d = pn_load4(a, a_code, src * size + i);
       if (b != nullptr) {
@@ -58,6 +60,10 @@ pair_add_rmsnorm_kernel(float* __restrict__ x, const void* __restrict__ a, int a
         d.x += e.x; d.y += e.y; d.z += e.z; d.w += e.w;
       }
       v.x = fmaf(m, d.x, v.x); v.y = fmaf(m, d.y, v.y); v.z = fmaf(m, d.z, v.z); v.w = fmaf(m, d.w, v.w);
+      if (c != nullptr) {
+        const float4 e = *reinterpret_cast<const float4*>(c + src * size + i);
+        v.x += e.x; v.y += e.y; v.z += e.z; v.w += e.w;
+      }
       *reinterpret_cast<float4*>(row + i) = v;
     }
     if (i == first) held = v;
@@ -114,28 +120,29 @@ add_bias_by8_kernel(const TIn* __restrict__ in, long long ldi, const float* __re
 using namespace mxb;
 
 // x: float32 [rows_of_x, size], updated in place when a or b is given (then rows_index must be null and the
-// grid covers every row). a, b: [rows, size] of their own types (kF32 / kBF16), or null. y1, y2: [rows, size] of
+// grid covers every row). a, b: [rows, size] of their own types (kF32 / kBF16), or null; c: float32 [rows, size], or
+// null. y1, y2: [rows, size] of
 // y_dtype; y2 with w2 or neither; y1 null: only the sum is made. size a multiple of 4 (8 for a bfloat16 operand),
 // everything 16-byte aligned.
-MXB_API int mxb_pair_add_rmsnorm(float* x, const void* a, int a_dtype, const void* b, int b_dtype, float m,
+MXB_API int mxb_pair_add_rmsnorm(float* x, const void* a, int a_dtype, const void* b, int b_dtype, float m, const float* c,
                                  const float* w1, const float* w2, void* y1, void* y2, int y_dtype,
                                  const int* rows_index, int rows, int size, float eps, cudaStream_t stream) {
   if (rows <= 0) return 0;
   auto aligned = [](const void* p) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0; };
   const bool halves = (a != nullptr && a_dtype == kBF16) || (b != nullptr && b_dtype == kBF16) || y_dtype == kBF16;
   if (size <= 0 || size % (halves ? 8 : 4) != 0 || !aligned(x) || !aligned(a) || !aligned(b) || !aligned(w1) ||
-      !aligned(w2) || !aligned(y1) || !aligned(y2) || (y1 != nullptr && w1 == nullptr) ||
-      ((y2 != nullptr) != (w2 != nullptr)) || (rows_index != nullptr && (a != nullptr || b != nullptr)))
+      !aligned(w2) || !aligned(c) || !aligned(y1) || !aligned(y2) || (y1 != nullptr && w1 == nullptr) ||
+      ((y2 != nullptr) != (w2 != nullptr)) || (rows_index != nullptr && (a != nullptr || b != nullptr || c != nullptr)))
     return static_cast<int>(cudaErrorInvalidValue);
   int threads = ((size / 4 + 31) / 32) * 32;
   if (threads > 256) threads = 256;
   if (y_dtype == kF32)
     return static_cast<int>(launch_chained(pair_add_rmsnorm_kernel<float>, dim3(rows), dim3(threads), 0, stream, x, a,
-                                           a_dtype, b, b_dtype, m, w1, w2, static_cast<float*>(y1),
+                                           a_dtype, b, b_dtype, m, c, w1, w2, static_cast<float*>(y1),
                                            static_cast<float*>(y2), rows_index, size, eps));
   if (y_dtype == kBF16)
     return static_cast<int>(launch_chained(pair_add_rmsnorm_kernel<__nv_bfloat16>, dim3(rows), dim3(threads), 0, stream,
-                                           x, a, a_dtype, b, b_dtype, m, w1, w2, static_cast<__nv_bfloat16*>(y1),
+                                           x, a, a_dtype, b, b_dtype, m, c, w1, w2, static_cast<__nv_bfloat16*>(y1),
                                            static_cast<__nv_bfloat16*>(y2), rows_index, size, eps));
   return static_cast<int>(cudaErrorInvalidValue);
 }

@@ -4,7 +4,7 @@
 // outputs (or, as a switch, s = sigmoid(z) for each output on its own; the
 // outputs may also form equal groups of neighbours of which only the best few,
 // by the sum of a group's two largest s + correction, can be chosen from; and
-// the weights may be multiplied by a constant; or, as a third form, s = z + correction itself decides and
+// the weights may be multiplied by a constant, or left as the chosen scores are, undivided; or, as a third form, s = z + correction itself decides and
 // weighs: the largest are chosen and their weights are the softmax over the chosen alone); the `top` outputs with the largest s + correction are chosen (ties
 // go to the lower index); their weights are their s, divided by the sum of
 // the chosen s (+ 1e-20). The sum s + correction is formed and compared in
@@ -19,7 +19,7 @@
 // of weights over the real experts (zeros for those not chosen) and the sum of
 // the weights that fell on identity experts.
 //
-// Two ways through the experts W_down act(W_up h), act(u) = relu(u)^2, with
+// Two ways through the experts W_down act(W_up h), act(u) = relu(u)^2 or u times the normal distribution at u, with
 // W_up stacked [experts * ff, hidden] and W_down stacked [experts * hidden, ff]:
 // * grouped, for steps of many tokens: expert_rows_kernel gives every
 //   (token, choice) pair a row in an array sorted by expert, each expert's
@@ -33,12 +33,15 @@
 //   warp per row of a chosen expert's W_up) and routed_down_kernel (a warp
 //   per output value, over the chosen experts' W_down), so that a decode step
 //   reads `top` experts' weights and not all of them.
+// A pair's weight multiplies what its expert leaves or (`weigh_input`) what it
+// takes, act(w W_up h): the product's rows are scaled ahead of the activation.
 // Both add weight_identity * h at the end (combine_rows_kernel, or inside
 // routed_down_kernel).
 #include "common.cuh"
 
 namespace mxb {
 
+enum ExpertForm : int { kExpertReluSquared = 0, kExpertGated = 1, kExpertGelu = 2 };
 enum RouteScores : int { kScoreSoftmax = 0, kScoreSigmoid = 1, kScoreChosen = 2 };
 constexpr int kRouteThreads = 128;   // four tokens a block, a warp each
 
@@ -46,7 +49,7 @@ __global__ void __launch_bounds__(kRouteThreads)
 route_kernel(const float* __restrict__ logits, const float* __restrict__ correction, int* __restrict__ chosen,
              float* __restrict__ weights, float* __restrict__ dense, float* __restrict__ identity_weight,
              int tokens, int outputs, int experts, int top, int scores, int group_count, int group_keep,
-             float weight_scale, long long ld, int always) {
+             float weight_scale, long long ld, int always, int undivided) {
   extern __shared__ double shared[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int t = blockIdx.x * (kRouteThreads / 32) + warp;
@@ -150,7 +153,7 @@ route_kernel(const float* __restrict__ logits, const float* __restrict__ correct
     picked_sum += score[where];
     __syncwarp();
   }
-  const float scale = weight_scale / (picked_sum + 1e-20f);
+  const float scale = undivided ? weight_scale : weight_scale / (picked_sum + 1e-20f);
   if (lane == 0) {
     float on_identity = 0.0f;
     for (int k = 0; k < top; ++k) {
@@ -231,15 +234,17 @@ expert_rows_kernel(const int* __restrict__ chosen, int* __restrict__ position, i
   }
 }
 
-// sorted[position[p], :] = h[p / top, :], 16 bytes a thread at a time (hidden * sizeof(T) a multiple of 16)
+// sorted[position[p], :] = h[p / top, :], 16 bytes a thread at a time (hidden * sizeof(T) a multiple of 16), and the
+// pair's weight into row_weight[position[p]] where the products scale their rows by it
 template <typename T>
 __global__ void __launch_bounds__(256)
 gather_rows_kernel(const T* __restrict__ h, const int* __restrict__ position, T* __restrict__ sorted, int pairs,
-                   int hidden, int top) {
+                   int hidden, int top, const float* __restrict__ weights, float* __restrict__ row_weight) {
   const int p = blockIdx.x * 8 + (threadIdx.x >> 5), lane = threadIdx.x & 31;
   if (p >= pairs) return;
   const int row = position[p];
   if (row < 0) return;
+  if (row_weight != nullptr && lane == 0) row_weight[row] = weights[p];
   const uint4* src = reinterpret_cast<const uint4*>(h + static_cast<size_t>(p / top) * hidden);
   uint4* dst = reinterpret_cast<uint4*>(sorted + static_cast<size_t>(row) * hidden);
   const int vectors = hidden * static_cast<int>(sizeof(T)) / 16;
@@ -247,6 +252,7 @@ gather_rows_kernel(const T* __restrict__ h, const int* __restrict__ position, T*
 }
 
 // y[t, c] = sum_k weights[t, k] * rows[position[t, k], c] + identity_weight[t] * h[t, c]; four columns a thread
+// (no weights: 1 for every row)
 template <typename T>
 __global__ void __launch_bounds__(256)
 combine_rows_kernel(const float* __restrict__ rows, const int* __restrict__ position,
@@ -259,7 +265,7 @@ combine_rows_kernel(const float* __restrict__ rows, const int* __restrict__ posi
     for (int k = 0; k < top; ++k) {
       const int row = position[static_cast<size_t>(t) * top + k];
       if (row < 0) continue;
-      const float w = weights[static_cast<size_t>(t) * top + k];
+      const float w = weights != nullptr ? weights[static_cast<size_t>(t) * top + k] : 1.0f;
       const float4 v = *reinterpret_cast<const float4*>(rows + static_cast<size_t>(row) * hidden + c);
       sum[0] = fmaf(w, v.x, sum[0]); sum[1] = fmaf(w, v.y, sum[1]);
       sum[2] = fmaf(w, v.z, sum[2]); sum[3] = fmaf(w, v.w, sum[3]);
@@ -299,33 +305,35 @@ __device__ __forceinline__ float dot_rows(const T* __restrict__ row, const U* __
 
 constexpr int kRoutedThreads = 256;   // eight warps, a row of a weight each
 
-// act[(t, k), f] = relu(W_up[e * ff + f, :] . h[t, :])^2 * weight[t, k] for e = chosen[t, k] < experts; or, `gated`,
-// with an expert's matrix [2 * ff, hidden] holding gate rows and then up rows,
-// silu(W_gate[f, :] . h) * (W_up[f, :] . h) * weight
+// act[(t, k), f] = relu(W_up[e * ff + f, :] . h[t, :])^2 * weight[t, k] for e = chosen[t, k] < experts; or, form
+// kExpertGated, with an expert's matrix [2 * ff, hidden] holding gate rows and then up rows,
+// silu(W_gate[f, :] . h) * (W_up[f, :] . h) * weight; or, form kExpertGelu, gelu(W_up[e * ff + f, :] . h) in its exact
+// form. weigh_input: the weight multiplies h instead of the result.
 template <typename T>
 __global__ void __launch_bounds__(kRoutedThreads)
 routed_up_kernel(const T* __restrict__ h, const T* __restrict__ w_up, const int* __restrict__ chosen,
                  const float* __restrict__ weights, float* __restrict__ act, int hidden, int experts, int ff, int top,
-                 int gated) {
+                 int form, int weigh_input) {
   const int pair = blockIdx.x;                    // token * top + k
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
   const int f = blockIdx.y * (kRoutedThreads / 32) + warp;
   const int e = chosen[pair];
   if (f >= ff || e >= experts || e < 0) return;
   const T* x = h + static_cast<size_t>(pair / top) * hidden;
-  if (gated) {
+  const float before = weigh_input ? weights[pair] : 1.0f, after = weigh_input ? 1.0f : weights[pair];
+  if (form == kExpertGated) {
     const T* gate_row = w_up + (static_cast<size_t>(e) * 2 * ff + f) * hidden;
-    const float gate = warp_sum(dot_rows(gate_row, x, hidden, lane));
-    const float up = warp_sum(dot_rows(gate_row + static_cast<size_t>(ff) * hidden, x, hidden, lane));
-    if (lane == 0) act[static_cast<size_t>(pair) * ff + f] = gate / (1.0f + expf(-gate)) * up * weights[pair];
+    const float gate = before * warp_sum(dot_rows(gate_row, x, hidden, lane));
+    const float up = before * warp_sum(dot_rows(gate_row + static_cast<size_t>(ff) * hidden, x, hidden, lane));
+    if (lane == 0) act[static_cast<size_t>(pair) * ff + f] = gate / (1.0f + expf(-gate)) * up * after;
     return;
   }
   const T* row = w_up + (static_cast<size_t>(e) * ff + f) * hidden;
   float sum = dot_rows(row, x, hidden, lane);
-  sum = warp_sum(sum);
+  sum = before * warp_sum(sum);
   if (lane == 0) {
     const float u = fmaxf(sum, 0.0f);
-    act[static_cast<size_t>(pair) * ff + f] = u * u * weights[pair];
+    act[static_cast<size_t>(pair) * ff + f] = (form == kExpertGelu ? gelu_of(sum) : u * u) * after;
   }
 }
 
@@ -362,11 +370,12 @@ using namespace mxb;
 // logits: float32 [tokens, outputs]; correction: float32 [outputs]; chosen: int32 [tokens, top + always];
 // weights: float32 [tokens, top + always]; dense: float32 [tokens, experts]; identity_weight: float32 [tokens].
 // scores: 0 s = softmax(z), 1 s = sigmoid(z), 2 z + correction chooses and the softmax over the chosen weighs. group_count > 1: the outputs form that many equal groups of
-// neighbours, and only outputs of the group_keep best groups can be chosen. weight_scale multiplies the weights.
+// neighbours, and only outputs of the group_keep best groups can be chosen. weight_scale multiplies the weights; undivided: they are
+// the chosen scores as they are.
 MXB_API int mxb_route_experts(const float* logits, const float* correction, int* chosen, float* weights, float* dense,
                               float* identity_weight, int tokens, int outputs, int experts, int top,
                               int scores, int group_count, int group_keep, float weight_scale,
-                              long long ld, int always, cudaStream_t stream) {
+                              long long ld, int always, int undivided, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (always < 0 || (always > 0 && experts != outputs)) return static_cast<int>(cudaErrorInvalidValue);
   if (scores < kScoreSoftmax || scores > kScoreChosen) return static_cast<int>(cudaErrorInvalidValue);
@@ -380,7 +389,7 @@ MXB_API int mxb_route_experts(const float* logits, const float* correction, int*
   if (shared > 48 * 1024) return static_cast<int>(cudaErrorInvalidValue);
   route_kernel<<<ceil_div(tokens, kRouteThreads / 32), kRouteThreads, shared, stream>>>(
       logits, correction, chosen, weights, dense, identity_weight, tokens, outputs, experts, top, scores,
-      group_count, group_keep, weight_scale, ld < outputs ? outputs : ld, always);
+      group_count, group_keep, weight_scale, ld < outputs ? outputs : ld, always, undivided);
   return static_cast<int>(cudaGetLastError());
 }
 
@@ -399,25 +408,26 @@ MXB_API int mxb_experts_add_identity(float* y, const void* h, const float* ident
   return static_cast<int>(cudaGetLastError());
 }
 
-// h: [tokens, hidden]; w_up: [experts * ff, hidden] (gated: [experts * 2 * ff, hidden], every expert's gate rows
-// and then its up rows, the activation silu instead of relu^2); w_down: [experts * hidden, ff]; act: float32
+// h: [tokens, hidden]; w_up: [experts * ff, hidden] (form 1: [experts * 2 * ff, hidden], every expert's gate rows
+// and then its up rows, the activation silu instead of relu^2; form 2: gelu instead of relu^2); weigh_input: a pair's
+// weight multiplies its expert's input; w_down: [experts * hidden, ff]; act: float32
 // scratch [tokens * top, ff]; y: float32 [tokens, hidden].
 MXB_API int mxb_experts_routed(const void* h, const void* w_up, const void* w_down, const int* chosen,
                                const float* weights, float* act, float* y, int tokens, int hidden, int experts, int ff,
-                               int top, int dtype, int gated, cudaStream_t stream) {
+                               int top, int dtype, int form, int weigh_input, cudaStream_t stream) {
   if (tokens <= 0) return 0;
-  if (hidden <= 0 || ff <= 0 || top <= 0) return static_cast<int>(cudaErrorInvalidValue);
+  if (hidden <= 0 || ff <= 0 || top <= 0 || form < kExpertReluSquared || form > kExpertGelu) return static_cast<int>(cudaErrorInvalidValue);
   const int per_block = kRoutedThreads / 32;
   dim3 up_grid(tokens * top, ceil_div(ff, per_block)), down_grid(tokens, ceil_div(hidden, per_block));
   if (dtype == kF32) {
     routed_up_kernel<float><<<up_grid, kRoutedThreads, 0, stream>>>(
-        static_cast<const float*>(h), static_cast<const float*>(w_up), chosen, weights, act, hidden, experts, ff, top, gated);
+        static_cast<const float*>(h), static_cast<const float*>(w_up), chosen, weights, act, hidden, experts, ff, top, form, weigh_input);
     routed_down_kernel<float><<<down_grid, kRoutedThreads, 0, stream>>>(
         act, static_cast<const float*>(w_down), static_cast<const float*>(h), chosen, weights, y, hidden, experts, ff, top);
   } else if (dtype == kBF16) {
     routed_up_kernel<__nv_bfloat16><<<up_grid, kRoutedThreads, 0, stream>>>(
         static_cast<const __nv_bfloat16*>(h), static_cast<const __nv_bfloat16*>(w_up), chosen, weights, act, hidden,
-        experts, ff, top, gated);
+        experts, ff, top, form, weigh_input);
     routed_down_kernel<__nv_bfloat16><<<down_grid, kRoutedThreads, 0, stream>>>(
         act, static_cast<const __nv_bfloat16*>(w_down), static_cast<const __nv_bfloat16*>(h), chosen, weights, y,
         hidden, experts, ff, top);
@@ -460,26 +470,29 @@ MXB_API int mxb_expert_rows(const int* chosen, int* position, int* tile_group, i
 }
 
 // sorted[position[p], :] = h[p / top, :] for the pairs with a position; hidden * the element's size a multiple of 16.
+// row_weight (float32, one per sorted row, or null) takes the pairs' weights.
 MXB_API int mxb_expert_gather_rows(const void* h, const int* position, void* sorted, int pairs, int hidden, int top,
-                                   int dtype, cudaStream_t stream) {
+                                   int dtype, const float* weights, float* row_weight, cudaStream_t stream) {
   if (pairs <= 0) return 0;
   const int size = dtype == kF32 ? 4 : 2;
   if (hidden <= 0 || top <= 0 || (hidden * size) % 16 != 0 || (reinterpret_cast<uintptr_t>(h) & 15) ||
-      (reinterpret_cast<uintptr_t>(sorted) & 15))
+      (reinterpret_cast<uintptr_t>(sorted) & 15) || (row_weight != nullptr && weights == nullptr))
     return static_cast<int>(cudaErrorInvalidValue);
   const unsigned blocks = static_cast<unsigned>(ceil_div(pairs, 8));
   if (dtype == kF32)
     gather_rows_kernel<float><<<blocks, 256, 0, stream>>>(static_cast<const float*>(h), position,
-                                                         static_cast<float*>(sorted), pairs, hidden, top);
+                                                         static_cast<float*>(sorted), pairs, hidden, top, weights, row_weight);
   else if (dtype == kBF16)
     gather_rows_kernel<__nv_bfloat16><<<blocks, 256, 0, stream>>>(static_cast<const __nv_bfloat16*>(h), position,
-                                                                 static_cast<__nv_bfloat16*>(sorted), pairs, hidden, top);
+                                                                 static_cast<__nv_bfloat16*>(sorted), pairs, hidden, top, weights,
+                                                               row_weight);
   else
     return static_cast<int>(cudaErrorInvalidValue);
   return static_cast<int>(cudaGetLastError());
 }
 
-// rows: float32 [sorted rows, hidden]; y: float32 [tokens, hidden]; hidden a multiple of 4.
+// rows: float32 [sorted rows, hidden]; weights: one per pair, or null (1 each); y: float32 [tokens, hidden]; hidden a
+// multiple of 4.
 MXB_API int mxb_expert_combine_rows(const float* rows, const int* position, const float* weights,
                                     const float* identity_weight, const void* h, float* y, int tokens, int hidden,
                                     int top, int dtype, cudaStream_t stream) {

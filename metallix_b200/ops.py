@@ -35,25 +35,25 @@ _SIGNATURES = {
     "mxb_copy_units": [_P, _I, _I, _L, _P, _I, _P, _P],
     "mxb_qk_norm_rope_cache": [_P, _P, _P, _L, _L, _L, _P, _P, _P, _P, _P, _P, _P, _P,
                                _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _I, _P, _P],
-    "mxb_paged_attention_tile": [_P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I,
+    "mxb_paged_attention_tile": [_P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I,
                                  _F, _I, _P, _L, _I, _I, _F, _I, _I, _F, _P, _P, _I, _P, _P],
     "mxb_short_conv": [_P, _L, _P, _P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _P, _P],
     "mxb_selective_scan": [_P, _L, _P, _L, _P, _P, _P, _P, _L, _P, _P, _L, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I,
                            _I, _P, _P],
-    "mxb_route_experts": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _L, _I, _P],
+    "mxb_route_experts": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _F, _L, _I, _I, _P],
     "mxb_expert_rows": [_P, _P, _P, _I, _I, _I, _P],
     "mxb_expert_rows_tile": [],
     "mxb_expert_rows_experts": [],
-    "mxb_expert_gather_rows": [_P, _P, _P, _I, _I, _I, _I, _P],
+    "mxb_expert_gather_rows": [_P, _P, _P, _I, _I, _I, _I, _P, _P, _P],
     "mxb_expert_combine_rows": [_P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _P],
     "mxb_experts_add_identity": [_P, _P, _P, _I, _I, _I, _P],
-    "mxb_experts_routed": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _P],
+    "mxb_experts_routed": [_P, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _P],
     "mxb_add_gated_rows": [_P, _P, _P, _L, _I, _I, _I, _P],
-    "mxb_pair_add_rmsnorm": [_P, _P, _I, _P, _I, _F, _P, _P, _P, _P, _I, _P, _I, _I, _F, _P],
+    "mxb_pair_add_rmsnorm": [_P, _P, _I, _P, _I, _F, _P, _P, _P, _P, _P, _I, _P, _I, _I, _F, _P],
     "mxb_pair_norm_max_size": [],
     "mxb_pair_norm": [_P, _P, _I, _I, _P, _I, _P, _P, _P, _P, _F, _F, _F, _F, _P, _I, _P, _I, _I, _F, _P],
     "mxb_gated_norm_max_part": [],
-    "mxb_gated_norm": [_P, _P, _L, _I, _P, _P, _I, _I, _I, _I, _I, _F, _P],
+    "mxb_gated_norm": [_P, _P, _L, _I, _P, _P, _I, _I, _I, _I, _I, _I, _F, _P],
     "mxb_join_rows": [_P, _P, _I, _P, _P, _I, _I, _I, _P],
     "mxb_add_bias": [_P, _L, _I, _P, _P, _L, _I, _I, _I, _P],
     "mxb_delta_rule_max_dim": [],
@@ -71,23 +71,23 @@ _SIGNATURES = {
     "mxb_latent_heads": [_P, _L, _P, _L, _P, _L, _I, _P, _P, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I,
                          _I, _P, _P],
     "mxb_rotate_into": [_P, _L, _I, _I, _P, _I, _I, _I, _I, _I, _I, _P, _P, _I, _P, _I, _I, _P, _P],
-    "mxb_relu_squared": [_P, _P, _L, _I, _P],
-    "mxb_paged_attention_decode": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I,
+    "mxb_plain_activation": [_P, _P, _L, _I, _I, _P],
+    "mxb_paged_attention_decode": [_P, _P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I,
                                    _F, _I, _P, _L, _F, _I, _F, _P, _P, _I, _P, _P],
     "mxb_postnorm_add_rmsnorm": [_P, _P, _I, _I, _P, _F, _P, _I, _P, _F, _I, _I, _P],
     "mxb_sigmoid_gate": [_P, _P, _P, _L, _L, _L, _I, _I, _I, _P],
     "mxb_softcap": [_P, _F, _L, _P],
     "mxb_paged_attention_decode_supported": [_I, _I, _I, _I],
     "mxb_paged_attention_decode_project_supported": [_I, _I, _I, _I, _I, _P, _L],
-    "mxb_paged_attention_decode_project": [_P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I,
+    "mxb_paged_attention_decode_project": [_P, _P, _P, _P, _I, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I,
                                            _F, _P, _L, _I, _P, _P, _L, _F, _I, _F, _P, _P, _I, _P, _P],
     "mxb_paged_attention_split_keys": [],
     "mxb_set_decode_resident_blocks": [_I, _I],
-    "mxb_flash_prefill": [_P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _L, _F, _I, _F,
+    "mxb_flash_prefill": [_P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _P, _L, _F, _I, _F,
                           _P, _P, _I, _P, _P],
     "mxb_flash_prefill_supported": [_I, _I, _I, _I],
     "mxb_flash_prefill_tile": [],
-    "mxb_flash_prefill_tcgen05": [_P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P,
+    "mxb_flash_prefill_tcgen05": [_P, _P, _P, _P, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _I, _I, _I, _I, _F, _I, _I, _P,
                                   _P, _L, _F, _I, _F, _P, _P, _I, _P, _P],
     "mxb_flash_prefill_tcgen05_supported": [_I, _I, _I, _I, _I],
     "mxb_flash_prefill_tcgen05_tile": [],
@@ -98,7 +98,7 @@ _SIGNATURES = {
     "mxb_gemm_stream_supported": [_I, _I, _I, _L, _L, _I],
     "mxb_gemm_tcgen05": [_P, _P, _P, _I, _I, _I, _L, _L, _L, _I, _F, _P, _P],
     "mxb_gemm_tcgen05_supported": [_I, _I, _I, _L, _L],
-    "mxb_gemm_tcgen05_grouped": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _L, _L, _L, _I, _P, _P],
+    "mxb_gemm_tcgen05_grouped": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _L, _L, _L, _I, _P, _P, _P],
     "mxb_silu_mul": [_P, _P, _I, _L, _I, _I, _F, _P],
     "mxb_argmax": [_P, _L, _I, _I, _P, _P, _P, _P],
     "mxb_argmax_pieces": [_I, _I],
@@ -350,9 +350,10 @@ def add_(x: torch.Tensor, delta: torch.Tensor) -> torch.Tensor:
 
 def pair_add_rmsnorm(x: torch.Tensor, a: Optional[torch.Tensor], b: Optional[torch.Tensor], scale: float,
                      weight: Optional[torch.Tensor], second_weight: Optional[torch.Tensor], eps: float,
-                     out_dtype: torch.dtype, rows_index: Optional[torch.Tensor] = None):
-    """x += scale * (a + b) in float32 (in place; ``a`` and ``b`` are optional,
-    each float32 or bfloat16), then RMSNorm(x) * weight and, with
+                     out_dtype: torch.dtype, rows_index: Optional[torch.Tensor] = None,
+                     c: Optional[torch.Tensor] = None):
+    """x += scale * (a + b) + c in float32 (in place; ``a``, ``b`` and ``c`` are
+    optional, a and b each float32 or bfloat16, c float32), then RMSNorm(x) * weight and, with
     ``second_weight``, RMSNorm(x) * second_weight from the same pass over the
     row: what a layer needs whose two sublayers read the same input. Returns
     the one result, or the two as a pair; None without ``weight`` (the sum
@@ -363,10 +364,13 @@ def pair_add_rmsnorm(x: torch.Tensor, a: Optional[torch.Tensor], b: Optional[tor
         if delta is not None:
             _check(delta, name, tuple(_CODES), 2)
             _need(delta.shape == x.shape, f"{name} and x differ in shape")
+    if c is not None:
+        _check(c, "c", (torch.float32,), 2)
+        _need(c.shape == x.shape, "c and x differ in shape")
     rows = x.shape[0]
     if rows_index is not None:
         _check(rows_index, "rows_index", (torch.int32,), 1)
-        _need(a is None and b is None, "rows are picked only where nothing is added")
+        _need(a is None and b is None and c is None, "rows are picked only where nothing is added")
         rows = rows_index.numel()
     first = second = None
     if weight is not None:
@@ -381,7 +385,7 @@ def pair_add_rmsnorm(x: torch.Tensor, a: Optional[torch.Tensor], b: Optional[tor
         _need(second_weight is None, "a second weight without a first")
     _need(out_dtype in _CODES, "out_dtype must be float32 or bfloat16")
     _call("mxb_pair_add_rmsnorm", x.data_ptr(), _ptr(a), _CODES[a.dtype] if a is not None else F32, _ptr(b),
-          _CODES[b.dtype] if b is not None else F32, float(scale), _ptr(weight), _ptr(second_weight), _ptr(first),
+          _CODES[b.dtype] if b is not None else F32, float(scale), _ptr(c), _ptr(weight), _ptr(second_weight), _ptr(first),
           _ptr(second), _CODES[out_dtype], _ptr(rows_index), rows, size, float(eps), _stream())
     if weight is None:
         return None
@@ -583,9 +587,18 @@ def weighted_sum(x: torch.Tensor, y: torch.Tensor, a: float, b: float) -> torch.
 
 def relu_squared(x: torch.Tensor) -> torch.Tensor:
     """max(x, 0)^2, float32 inside."""
+    return _plain_activation(x, 0)
+
+
+def gelu(x: torch.Tensor) -> torch.Tensor:
+    """x times the standard normal distribution at x (gelu's exact form), float32 inside."""
+    return _plain_activation(x, 1)
+
+
+def _plain_activation(x: torch.Tensor, code: int) -> torch.Tensor:
     _check(x, "x", tuple(_CODES))
     out = torch.empty_like(x)
-    _call("mxb_relu_squared", out.data_ptr(), x.data_ptr(), x.numel(), _CODES[x.dtype], _stream())
+    _call("mxb_plain_activation", out.data_ptr(), x.data_ptr(), x.numel(), _CODES[x.dtype], code, _stream())
     return out
 
 
@@ -676,14 +689,16 @@ def selective_scan(x: torch.Tensor, step: torch.Tensor, step_bias: torch.Tensor,
 
 # ------------------------------------------------------------ routed experts
 ROUTE_SCORES = {"softmax": 0, "sigmoid": 1, "chosen": 2}
+EXPERT_FORMS = {"relu_squared": 0, "swiglu": 1, "gelu": 2}
 ROUTER_OUTPUTS = 1024   # the most router outputs the routing kernel keeps in shared memory
 
 
 def route_experts(logits: torch.Tensor, correction: torch.Tensor, experts: int, top: int, scores: str = "softmax",
-                  groups: Optional[tuple] = None, scale: float = 1.0, always: int = 0):
+                  groups: Optional[tuple] = None, scale: float = 1.0, always: int = 0, normalized: bool = True):
     """Scores over all router outputs (``scores``: "softmax" over the row, or
     "sigmoid" of each logit on its own), the ``top`` largest score + correction
-    chosen, weights = the chosen scores over their sum, times ``scale``. With
+    chosen, weights = the chosen scores over their sum (not ``normalized``: as
+    they are), times ``scale``. With
     "chosen" the ``top`` largest logit + correction (a bias of the router's) are
     chosen and their weights are the softmax over these sums alone. ``always``: that
     many choices more per token, the experts from index ``experts`` on with weight
@@ -715,7 +730,7 @@ def route_experts(logits: torch.Tensor, correction: torch.Tensor, experts: int, 
     on_identity = torch.empty((tokens,), dtype=torch.float32, device=device)
     _call("mxb_route_experts", logits.data_ptr(), correction.data_ptr(), chosen.data_ptr(), weights.data_ptr(),
           dense.data_ptr(), on_identity.data_ptr(), tokens, outputs, experts, top, ROUTE_SCORES[scores],
-          count, keep, float(scale), logits.stride(0), int(always), _stream())
+          count, keep, float(scale), logits.stride(0), int(always), 0 if normalized else 1, _stream())
     return chosen, weights, dense, on_identity
 
 
@@ -741,31 +756,38 @@ def expert_rows_tile() -> int:
     return int(_fn("mxb_expert_rows_tile")())
 
 
-def expert_gather_rows(h: torch.Tensor, position: torch.Tensor, rows: int) -> torch.Tensor:
+def expert_gather_rows(h: torch.Tensor, position: torch.Tensor, rows: int, weights: Optional[torch.Tensor] = None):
     """``[rows, hidden]`` with h[t] at position[t, k] for every pair that has
-    a position; the other rows are left as they are found."""
+    a position; the other rows are left as they are found. With ``weights``
+    (float32, one per pair) the rows come with each row's weight, ``[rows]``."""
     _check(h, "h", tuple(_CODES), 2)
     _check(position, "position", (torch.int32,), 2)
     _need(position.shape[0] == h.shape[0], "a row of positions per token")
     out = torch.empty((rows, h.shape[1]), dtype=h.dtype, device=h.device)
+    row_weight = None
+    if weights is not None:
+        _check(weights, "weights", (torch.float32,), 2)
+        _need(weights.shape == position.shape, "one weight per pair")
+        row_weight = torch.empty((rows,), dtype=torch.float32, device=h.device)
     _call("mxb_expert_gather_rows", h.data_ptr(), position.data_ptr(), out.data_ptr(), position.numel(), h.shape[1],
-          position.shape[1], _CODES[h.dtype], _stream())
-    return out
+          position.shape[1], _CODES[h.dtype], _ptr(weights), _ptr(row_weight), _stream())
+    return out if weights is None else (out, row_weight)
 
 
-def expert_combine_rows(rows: torch.Tensor, position: torch.Tensor, weights: torch.Tensor, on_identity: torch.Tensor,
-                        h: torch.Tensor) -> torch.Tensor:
-    """y[t] = sum_k weights[t, k] rows[position[t, k]] + on_identity[t] h[t], float32."""
+def expert_combine_rows(rows: torch.Tensor, position: torch.Tensor, weights: Optional[torch.Tensor],
+                        on_identity: torch.Tensor, h: torch.Tensor) -> torch.Tensor:
+    """y[t] = sum_k weights[t, k] rows[position[t, k]] + on_identity[t] h[t], float32; without ``weights`` every row counts 1."""
     _check(rows, "rows", (torch.float32,), 2)
     _check(position, "position", (torch.int32,), 2)
-    _check(weights, "weights", (torch.float32,), 2)
+    if weights is not None:
+        _check(weights, "weights", (torch.float32,), 2)
     _check(on_identity, "on_identity", (torch.float32,), 1)
     _check(h, "h", tuple(_CODES), 2)
     tokens, hidden = h.shape
-    _need(rows.shape[1] == hidden and position.shape == weights.shape and position.shape[0] == tokens
+    _need(rows.shape[1] == hidden and (weights is None or position.shape == weights.shape) and position.shape[0] == tokens
           and on_identity.numel() == tokens, "rows, positions, weights and h do not fit")
     y = torch.empty((tokens, hidden), dtype=torch.float32, device=h.device)
-    _call("mxb_expert_combine_rows", rows.data_ptr(), position.data_ptr(), weights.data_ptr(), on_identity.data_ptr(),
+    _call("mxb_expert_combine_rows", rows.data_ptr(), position.data_ptr(), _ptr(weights), on_identity.data_ptr(),
           h.data_ptr(), y.data_ptr(), tokens, hidden, position.shape[1], _CODES[h.dtype], _stream())
     return y
 
@@ -782,14 +804,19 @@ def experts_add_identity(y: torch.Tensor, h: torch.Tensor, on_identity: torch.Te
 
 
 def experts_routed(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, chosen: torch.Tensor,
-                   weights: torch.Tensor, experts: int, ff: int, gated: bool = False) -> torch.Tensor:
+                   weights: torch.Tensor, experts: int, ff: int, activation: str = "relu_squared",
+                   weigh_input: bool = False) -> torch.Tensor:
     """sum_k weight[t, k] W_down[e] relu(W_up[e] h_t)^2 over a token's chosen
     experts e = chosen[t, k] < experts, plus h_t times the weights of chosen
     indices from ``experts`` on; float32 ``[tokens, hidden]``. Only the chosen
     experts' weights are read. w_up ``[experts * ff, hidden]``, w_down
-    ``[experts * hidden, ff]``. ``gated``: an expert is W_down (silu(W_gate h) *
-    (W_up h)) and w_up holds, expert by expert, its gate rows and then its up
-    rows, ``[experts * 2 * ff, hidden]``."""
+    ``[experts * hidden, ff]``. ``activation`` "swiglu": an expert is W_down
+    (silu(W_gate h) * (W_up h)) and w_up holds, expert by expert, its gate rows
+    and then its up rows, ``[experts * 2 * ff, hidden]``; "gelu": gelu in its
+    exact form instead of the squared relu. ``weigh_input``: the weights
+    multiply the experts' inputs, not their outputs."""
+    _need(activation in EXPERT_FORMS, f"unknown activation {activation!r}")
+    gated = activation == "swiglu"
     dtype = h.dtype
     _check(h, "h", tuple(_CODES), 2)
     _check(w_up, "w_up", (dtype,), 2)
@@ -805,7 +832,7 @@ def experts_routed(h: torch.Tensor, w_up: torch.Tensor, w_down: torch.Tensor, ch
     y = torch.empty((tokens, hidden), dtype=torch.float32, device=h.device)
     _call("mxb_experts_routed", h.data_ptr(), w_up.data_ptr(), w_down.data_ptr(), chosen.data_ptr(),
           weights.data_ptr(), act.data_ptr(), y.data_ptr(), tokens, hidden, experts, ff, top, _CODES[dtype],
-          1 if gated else 0, _stream())
+          EXPERT_FORMS[activation], 1 if weigh_input else 0, _stream())
     return y
 
 
@@ -918,11 +945,11 @@ def head_norm_gate(x: torch.Tensor, weight: torch.Tensor, gate: Optional[torch.T
 
 
 def gated_norm(x: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, parts: int, eps: float, out_dtype: torch.dtype,
-               activation: str = "silu") -> torch.Tensor:
+               activation: str = "silu", behind: bool = False) -> torch.Tensor:
     """u = x * act(gate) for x float32 ``[tokens, width]``, each of the row's
     ``parts`` equal parts over its own root mean square, times ``weight``
     (``[width]``). ``gate`` has x's shape (rows may be strided); act is "silu" or
-    "sigmoid"."""
+    "sigmoid". ``behind``: act(gate) multiplies what the norm leaves instead."""
     _check(x, "x", (torch.float32,), 2)
     _check(weight, "weight", (torch.float32,), 1)
     tokens, width = x.shape
@@ -932,8 +959,8 @@ def gated_norm(x: torch.Tensor, weight: torch.Tensor, gate: torch.Tensor, parts:
     _need(activation in ("silu", "sigmoid") and out_dtype in _CODES, "unknown activation or out_dtype")
     out = torch.empty((tokens, width), dtype=out_dtype, device=x.device)
     _call("mxb_gated_norm", x.data_ptr(), gate.data_ptr(), gate.stride(0), _CODES[gate.dtype], weight.data_ptr(),
-          out.data_ptr(), _CODES[out_dtype], tokens, parts, width // parts, 1 if activation == "silu" else 0, float(eps),
-          _stream())
+          out.data_ptr(), _CODES[out_dtype], tokens, parts, width // parts, 1 if activation == "silu" else 0, 1 if behind else 0,
+          float(eps), _stream())
     return out
 
 
@@ -984,6 +1011,19 @@ def state_space_dual(xbc: torch.Tensor, offsets, step: torch.Tensor, step_bias: 
                          heads, groups, dim, vdim, longest)
 
 
+def lightning_attention(qkv: torch.Tensor, offsets, decay: torch.Tensor, state: torch.Tensor, row_start: torch.Tensor,
+                        row_length: torch.Tensor, request_slots: torch.Tensor, heads: int, dim: int, vdim: int,
+                        longest: int = 0) -> torch.Tensor:
+    """Linear attention with a constant decay per head over a step's tokens.
+    ``qkv`` holds, from the column ``offsets`` (q, k, v) on, heads * dim queries and
+    keys and heads * vdim values, all ahead of their silu, which happens in the
+    kernel; ``decay`` float32 ``[heads]``. Per head S <- decay S + k v^T, o = S^T q.
+    ``state`` float32 ``[slots, heads, vdim, dim]`` is advanced in place; rows and
+    slots as in ``delta_rule``. Returns float32 ``[tokens, heads * vdim]``."""
+    return _matrix_state(3, qkv, offsets, None, None, None, decay, None, state, row_start, row_length, request_slots,
+                         heads, heads, dim, vdim, longest)
+
+
 def _matrix_state(mode: int, qkv, offsets, beta, step, step_bias, rate, skip, state, row_start, row_length, request_slots,
                   heads: int, groups: int, dim: int, vdim: int, longest: int) -> torch.Tensor:
     _need(qkv.is_cuda and qkv.dtype in _CODES and qkv.dim() == 2 and qkv.stride(1) == 1,
@@ -991,16 +1031,17 @@ def _matrix_state(mode: int, qkv, offsets, beta, step, step_bias, rate, skip, st
     tokens = qkv.shape[0]
     per_head = lambda tensor: (tensor.is_cuda and tensor.dtype == qkv.dtype and tensor.dim() == 2
                                and (tensor.stride(1) == 1 or heads == 1) and tensor.shape == (tokens, heads))
-    _need(mode == 2 or per_head(beta), "beta must be [tokens, heads] of qkv's type")
+    _need(mode >= 2 or per_head(beta), "beta must be [tokens, heads] of qkv's type")
     if mode == 0:
         _need(step.is_cuda and step.dtype == torch.float32 and step.dim() == 2 and step.stride(1) == 1
               and step.shape == (tokens, heads * dim), "step must be float32 [tokens, heads * dim]")
-    else:
+    elif mode != 3:
         _need(per_head(step), "step must be [tokens, heads] of qkv's type")
-    _check(step_bias, "step_bias", (torch.float32,), 1)
+    if mode != 3:
+        _check(step_bias, "step_bias", (torch.float32,), 1)
+        _need(step_bias.numel() == (heads * dim if mode == 0 else heads), "step_bias has the wrong size")
     _check(rate, "rate", (torch.float32,), 1)
-    _need(step_bias.numel() == (heads * dim if mode == 0 else heads) and rate.numel() == heads,
-          "step_bias or rate has the wrong size")
+    _need(rate.numel() == heads, "rate has the wrong size")
     if mode == 2:
         _check(skip, "skip", (torch.float32,), 1)
         _need(skip.numel() == heads, "skip has the wrong size")
@@ -1016,7 +1057,7 @@ def _matrix_state(mode: int, qkv, offsets, beta, step, step_bias, rate, skip, st
           "the column offsets reach beyond qkv")
     out = torch.empty((tokens, heads * vdim), dtype=torch.float32, device=qkv.device)
     _call("mxb_delta_rule", qkv.data_ptr(), qkv.stride(0), q_off, k_off, v_off, _ptr(beta),
-          beta.stride(0) if beta is not None else 0, 0, step.data_ptr(), step.stride(0), step_bias.data_ptr(),
+          beta.stride(0) if beta is not None else 0, 0, _ptr(step), step.stride(0) if step is not None else 0, _ptr(step_bias),
           rate.data_ptr(), _ptr(skip), mode, state.data_ptr(), state.stride(0),
           state.shape[0], row_start.data_ptr(), row_length.data_ptr(), request_slots.data_ptr(), out.data_ptr(), rows,
           heads, groups, dim, vdim, _CODES[qkv.dtype], int(longest), status_word(qkv.device).data_ptr(), _stream())
@@ -1239,6 +1280,12 @@ def _sink(sink, heads: int):
     return 1, float(sink), None
 
 
+def _kept(keep) -> int:
+    """The number of first positions that stay visible beside a window or chunk."""
+    _need(int(keep or 0) >= 0, "the number of kept positions cannot be negative")
+    return int(keep or 0)
+
+
 def _score_bias(bias, heads: int):
     """(pointer, far) as the attention kernels take a bias per head and distance:
     None for none, or a contiguous float32 tensor ``[heads, far + 1]`` whose entry
@@ -1257,7 +1304,7 @@ def paged_attention_tile(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor
                          tile_start: torch.Tensor, tile_length: torch.Tensor,
                          positions: torch.Tensor, scale: float, window: int = 0, chunk: int = 0,
                          gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                         gate_per_head: bool = False, sink=None, bias=None) -> torch.Tensor:
+                         gate_per_head: bool = False, sink=None, bias=None, keep: int = 0) -> torch.Tensor:
     """Attention of every query token over its request's cached keys (itself
     included) in float32; q is [tokens, heads, head_dim], out
     [tokens, heads, value_dim] with value_dim at most head_dim (the first
@@ -1266,6 +1313,7 @@ def paged_attention_tile(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor
     values, one plane holds rows that are keys and values at once. ``window``:
     only the last that many positions are seen; ``chunk``: only the keys of the
     query's own chunk of that many positions, counted from position 0;
+    ``keep``: the first that many positions are seen beside either;
     ``softcap`` c: scores pass c tanh(s / c) ahead of the softmax;
     ``gate`` ([tokens, heads * value_dim], or [tokens, heads] with
     ``gate_per_head``; rows may be strided): the output is multiplied by
@@ -1301,7 +1349,7 @@ def paged_attention_tile(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor
     _call("mxb_paged_attention_tile", q.data_ptr(), cache.data_ptr(), out.data_ptr(),
           block_tables.data_ptr(), block_tables.shape[1], tile_request.data_ptr(),
           tile_start.data_ptr(), tile_length.data_ptr(), positions.data_ptr(), tiles, heads,
-          kv_heads, head_dim, page_tokens, num_pages, int(window or 0), int(chunk or 0), float(scale), _CODES[dtype],
+          kv_heads, head_dim, page_tokens, num_pages, int(window or 0), int(chunk or 0), _kept(keep), float(scale), _CODES[dtype],
           _ptr(gate), gate_stride, planes, value_dim, float(softcap), 1 if gate_per_head else 0,
           *_sink(sink, heads), *_score_bias(bias, heads), status_word(q.device).data_ptr(), _stream())
     return out
@@ -1352,7 +1400,7 @@ def flash_prefill(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block
                   tile_request: torch.Tensor, tile_start: torch.Tensor, tile_length: torch.Tensor,
                   positions: torch.Tensor, scale: float, window: int = 0, kernel: str = "auto",
                   longest_context: int = 0, chunk: int = 0, gate: Optional[torch.Tensor] = None,
-                  softcap: float = 0.0, sink=None, bias=None) -> torch.Tensor:
+                  softcap: float = 0.0, sink=None, bias=None, keep: int = 0) -> torch.Tensor:
     """Causal attention of prompt portions on the tensor cores (bfloat16,
     float32 softmax and accumulation); tiles hold up to 128 consecutive tokens
     of one request. ``kernel``: "tcgen05" (TMA, tensor memory), "mma" (the
@@ -1362,7 +1410,8 @@ def flash_prefill(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block
     the tiles alone would leave most of the GPU idle. ``softcap`` c: scores
     pass c tanh(s / c) ahead of the softmax. ``sink``: the score of one more
     key that has no value and that every query sees. ``bias`` (float32
-    ``[heads, far + 1]``): joins the scores by head and distance."""
+    ``[heads, far + 1]``): joins the scores by head and distance. ``keep``: the
+    first that many positions are seen beside the window or chunk."""
     _need(softcap >= 0.0, "the cap on the scores cannot be negative")
     _check(q, "q", (torch.bfloat16,), 3)
     _check(out, "out", (torch.bfloat16,), 3)
@@ -1398,7 +1447,7 @@ def flash_prefill(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block
         _call("mxb_flash_prefill_tcgen05", q.data_ptr(), cache.data_ptr(), out.data_ptr(),
               block_tables.data_ptr(), block_tables.shape[1], tile_request.data_ptr(), tile_start.data_ptr(),
               tile_length.data_ptr(), positions.data_ptr(), tokens, tiles, heads, kv_heads, head_dim,
-              page_tokens, num_pages, int(window or 0), int(chunk or 0), float(scale), _CODES[q.dtype], shares, _ptr(partial),
+              page_tokens, num_pages, int(window or 0), int(chunk or 0), _kept(keep), float(scale), _CODES[q.dtype], shares, _ptr(partial),
               _ptr(gate), gate_stride, float(softcap), *_sink(sink, heads), *_score_bias(bias, heads),
               status_word(q.device).data_ptr(), _stream())
         if shares > 1:
@@ -1408,7 +1457,7 @@ def flash_prefill(q: torch.Tensor, cache: torch.Tensor, out: torch.Tensor, block
     _call("mxb_flash_prefill", q.data_ptr(), cache.data_ptr(), out.data_ptr(), block_tables.data_ptr(),
           block_tables.shape[1], tile_request.data_ptr(), tile_start.data_ptr(), tile_length.data_ptr(),
           positions.data_ptr(), tiles, heads, kv_heads, head_dim, page_tokens, num_pages,
-          int(window or 0), int(chunk or 0), float(scale), _CODES[q.dtype], _ptr(gate), gate_stride, float(softcap),
+          int(window or 0), int(chunk or 0), _kept(keep), float(scale), _CODES[q.dtype], _ptr(gate), gate_stride, float(softcap),
           *_sink(sink, heads), *_score_bias(bias, heads), status_word(q.device).data_ptr(), _stream())
     return out
 
@@ -1441,7 +1490,7 @@ def paged_attention_decode(q: torch.Tensor, cache: torch.Tensor, out: torch.Tens
                            longest_context: int, window: int = 0,
                            partial: Optional[torch.Tensor] = None, chunk: int = 0,
                            gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                           sink=None, bias=None) -> torch.Tensor:
+                           sink=None, bias=None, keep: int = 0) -> torch.Tensor:
     """Attention of single tokens over their requests' cached keys, split
     along the keys. ``row_token[i]`` is the token (row of q and out) of the
     i-th decoded request, negative for a padding row; ``row_request[i]`` its
@@ -1453,7 +1502,8 @@ def paged_attention_decode(q: torch.Tensor, cache: torch.Tensor, out: torch.Tens
     scores pass c tanh(s / c) ahead of the softmax. ``sink``: the score of one
     more key that has no value and that every query sees (it joins the
     denominator where the splits are put together). ``bias`` (float32
-    ``[heads, far + 1]``): joins the scores by head and distance."""
+    ``[heads, far + 1]``): joins the scores by head and distance. ``keep``: the
+    first that many positions are seen beside the window or chunk."""
     dtype = q.dtype
     _need(softcap >= 0.0, "the cap on the scores cannot be negative")
     _check(q, "q", tuple(_CODES), 3)
@@ -1480,7 +1530,7 @@ def paged_attention_decode(q: torch.Tensor, cache: torch.Tensor, out: torch.Tens
     _call("mxb_paged_attention_decode", q.data_ptr(), cache.data_ptr(), out.data_ptr(), partial.data_ptr(),
           block_tables.data_ptr(), block_tables.shape[1], row_token.data_ptr(), row_request.data_ptr(),
           positions.data_ptr(), rows, heads, kv_heads, head_dim, page_tokens, num_pages, splits,
-          int(window or 0), int(chunk or 0), float(scale), _CODES[dtype], _ptr(gate), gate_stride, float(softcap),
+          int(window or 0), int(chunk or 0), _kept(keep), float(scale), _CODES[dtype], _ptr(gate), gate_stride, float(softcap),
           *_sink(sink, heads), *_score_bias(bias, heads), status_word(q.device).data_ptr(), _stream())
     return out
 
@@ -1510,7 +1560,7 @@ def paged_attention_decode_project(q: torch.Tensor, cache: torch.Tensor, block_t
                                    scale: float, longest_context: int, weight: torch.Tensor,
                                    window: int = 0, chunk: int = 0,
                                    gate: Optional[torch.Tensor] = None, softcap: float = 0.0,
-                                   sink=None, bias=None) -> torch.Tensor:
+                                   sink=None, bias=None, keep: int = 0) -> torch.Tensor:
     """``paged_attention_decode`` followed at once by the output projection
     ``weight`` ``[hidden, heads * head_dim]``, for steps of up to 64 tokens in
     bfloat16. Returns float32 ``[heads, tokens, hidden]``: the projection's sum
@@ -1537,7 +1587,7 @@ def paged_attention_decode_project(q: torch.Tensor, cache: torch.Tensor, block_t
     _call("mxb_paged_attention_decode_project", q.data_ptr(), cache.data_ptr(), partial.data_ptr(),
           block_tables.data_ptr(), block_tables.shape[1], row_token.data_ptr(), row_request.data_ptr(),
           positions.data_ptr(), rows, tokens, heads, kv_heads, head_dim, page_tokens, num_pages, splits,
-          int(window or 0), int(chunk or 0), float(scale), weight.data_ptr(), weight.stride(0), hidden, summands.data_ptr(),
+          int(window or 0), int(chunk or 0), _kept(keep), float(scale), weight.data_ptr(), weight.stride(0), hidden, summands.data_ptr(),
           _ptr(gate), gate_stride, float(softcap), *_sink(sink, heads), *_score_bias(bias, heads),
           status_word(q.device).data_ptr(), _stream())
     return summands

@@ -10,14 +10,18 @@ Variants, each a parameter: the norms of q and k may run over a token's whole
 projection instead of head by head (``qk_norm_scope="projection"``); a model
 without a value projection reuses the key projection's raw output (ahead of
 its norm and rotation) as the values (no ``v_proj``); ``chunk`` lets a query
-reach back only to the last absolute multiple of that many positions;
+reach back only to the last absolute multiple of that many positions; the
+first ``keep_first`` positions of a sequence are seen beside a window or chunk
+(the cache keeps their pages);
 ``gate_proj`` multiplies the concatenated heads by sigmoid(a Wg^T) ahead of the
 output projection (``gate_scope="head"``: Wg has one row per head, and a
 head's whole output is multiplied by one number); ``softcap`` c bounds the
 scores, s <- c tanh(s / c), ahead of the softmax; ``value_dim`` lets the
 values be wider or narrower than the keys (a page then holds rows as wide as
 the wider of the two, the others padded with zeros). Values of another width
-than the keys run on the general kernel only; a per-head gate is spread over
+than the keys run on the general kernel only, unless ``pad_heads`` says that
+heads of up to 128 values are to be padded with zeros to a size the tensor-core
+kernels take (``padded_heads``, bfloat16 only); a per-head gate is spread over
 the head's values for the tensor-core kernels. ``sink`` adds one more key
 without a value to every query's softmax, with that score (0.0: the
 denominator is 1 + the sum); a tensor's name instead of a number gives every
@@ -175,7 +179,7 @@ def tiles_of(ctx: StepContext) -> Dict[str, object]:
 def attend_cached(q_heads: torch.Tensor, cache: CacheView, ctx: StepContext, *, scale: float, window: int = 0,
                   chunk: int = 0, softcap: float = 0.0, gate: Optional[torch.Tensor] = None, gate_per_head: bool = False,
                   split_decode: bool = False, flash: bool = False, project=None, sink: Optional[float] = None,
-                  bias: Optional[torch.Tensor] = None):
+                  bias: Optional[torch.Tensor] = None, keep: int = 0):
     """Attention of a step's queries ``[tokens, heads, head_dim]`` over what the
     cache entry holds (this step's rows included), each kind of request on the
     kernel made for it: single tokens split along the keys, portions of prompts
@@ -198,20 +202,20 @@ def attend_cached(q_heads: torch.Tensor, cache: CacheView, ctx: StepContext, *, 
         return ops.paged_attention_decode_project(
             q_heads, cache.pool, cache.block_tables, tiles["decode_token"], tiles["decode_request"],
             ctx.positions, scale, tiles["longest_context"], project.weight, window, chunk, gate=gate,
-            softcap=softcap, sink=sink, bias=bias), True
+            softcap=softcap, sink=sink, bias=bias, keep=keep), True
     out = torch.empty_like(q_heads)
     if split:
         # Requests that bring one token: split along the keys.
         ops.paged_attention_decode(q_heads, cache.pool, out, cache.block_tables, tiles["decode_token"],
                                    tiles["decode_request"], ctx.positions, scale, tiles["longest_context"], window,
-                                   chunk=chunk, gate=gate, softcap=softcap, sink=sink, bias=bias)
+                                   chunk=chunk, gate=gate, softcap=softcap, sink=sink, bias=bias, keep=keep)
     if flash:
         # Requests that bring several tokens: tensor cores, tiles of 128.
         if tiles["wide_request"].numel():
             ops.flash_prefill(q_heads, cache.pool, out, cache.block_tables, tiles["wide_request"],
                               tiles["wide_start"], tiles["wide_length"], ctx.positions, scale, window,
                               longest_context=tiles["longest_keys"], chunk=chunk, gate=gate, softcap=softcap,
-                              sink=sink, bias=bias)
+                              sink=sink, bias=bias, keep=keep)
         rest = None if split else slice(multi_tiles, None)   # single tokens not yet served
     else:
         rest = slice(0, multi_tiles) if split else slice(0, None)
@@ -219,8 +223,65 @@ def attend_cached(q_heads: torch.Tensor, cache: CacheView, ctx: StepContext, *, 
         ops.paged_attention_tile(q_heads, cache.pool, out, cache.block_tables, tiles["tile_request"][rest],
                                  tiles["tile_start"][rest], tiles["tile_length"][rest], ctx.positions,
                                  scale, window, chunk, gate=gate, softcap=softcap, gate_per_head=gate_per_head,
-                                 sink=sink, bias=bias)
+                                 sink=sink, bias=bias, keep=keep)
     return out, False
+
+
+def padded_heads(spec: PartSpec, weights: WeightStore, runtime: Runtime):
+    """The same attention with heads of 64 or 128 values, the further ones zero:
+    (spec, weights), or the given ones where nothing is gained (float32, heads
+    that are such a size already or do not fit one, parts that need the given
+    size). Rows of zeros in the projections make the further values; columns of
+    zeros in the output projection take them. A norm over a whole projection
+    divides by the number of its values, so with c = D / (padded D) its weights
+    become sqrt(c) w and its epsilon c eps:
+    x rsqrt(S / (H D) + eps) w = x rsqrt(c (S / (H D) + eps)) sqrt(c) w."""
+    dim, value_dim = spec["head_dim"], spec.get("value_dim") or spec["head_dim"]
+    size = next((n for n in (64, 128) if n >= max(dim, value_dim)), 0)
+    norms = [spec.get("q_norm"), spec.get("k_norm")]
+    if (runtime.dtype != torch.bfloat16 or not size or (dim == value_dim == size) or spec.get("shared_kv")
+            or spec.get("v_proj") is None or spec.get("value_position") is not None or spec.get("gate_scope") == "head"
+            or any(norm is not None and (norm.kind != "rmsnorm" or norm.get("weight") is None) for norm in norms)):
+        return spec, weights
+    heads, groups = spec["num_heads"], spec["num_kv_heads"]
+    store, params, share = {}, dict(spec.params), dim / size
+
+    def rows(name, count, width):
+        if spec.get(name) is None:
+            return
+        tensor = weights.take(spec[name]).to(runtime.device)
+        wide = torch.zeros((count, size) + tuple(tensor.shape[1:]), dtype=tensor.dtype, device=tensor.device)
+        wide[:, :width] = tensor.reshape((count, width) + tuple(tensor.shape[1:]))
+        store[spec[name]] = wide.reshape((count * size,) + tuple(tensor.shape[1:]))
+
+    for name, count, width in (("q_proj", heads, dim), ("k_proj", groups, dim), ("v_proj", groups, value_dim),
+                               ("q_bias", heads, dim), ("k_bias", groups, dim), ("v_bias", groups, value_dim),
+                               ("gate_proj", heads, value_dim)):
+        rows(name, count, width)
+    out = weights.take(spec["o_proj"]).to(runtime.device)
+    wide = torch.zeros((out.shape[0], heads, size), dtype=out.dtype, device=out.device)
+    wide[:, :, :value_dim] = out.reshape(out.shape[0], heads, value_dim)
+    store[spec["o_proj"]] = wide.reshape(out.shape[0], heads * size)
+    per_head = (spec.get("qk_norm_scope") or "head") == "head"
+    for key, count in (("q_norm", heads), ("k_norm", groups)):
+        norm = spec.get(key)
+        if norm is None:
+            continue
+        given = weights.take(norm["weight"]).to(device=runtime.device, dtype=torch.float32)
+        given = (given + 1.0 if norm.get("one_plus") else given).reshape(1 if per_head else count, dim)
+        wide = torch.zeros((given.shape[0], size), dtype=torch.float32, device=given.device)
+        wide[:, :dim] = given * math.sqrt(share)
+        store[norm["weight"]] = wide.reshape(-1)
+        params[key] = PartSpec("rmsnorm", {"size": wide.numel(), "eps": norm["eps"] * share, "weight": norm["weight"]})
+    if spec.get("position") is not None:
+        params["position"] = PartSpec(spec["position"].kind, dict(spec["position"].params, head_dim=size))
+    for key in ("out_bias", "sink"):
+        if isinstance(spec.get(key), str):
+            store[spec[key]] = weights.take(spec[key])
+    if spec.get("distance_bias") is not None:
+        store[spec["distance_bias"]["weight"]] = weights.take(spec["distance_bias"]["weight"])
+    params.update(head_dim=size, value_dim=size, pad_heads=False)
+    return PartSpec(spec.kind, params), WeightStore(store)
 
 
 class GQAttention:
@@ -237,6 +298,8 @@ class GQAttention:
         self.scale = float(spec["scale"])
         self.window = spec.get("window") or 0
         self.chunk = spec.get("chunk") or 0
+        # kept positions matter only where something else ends what a query sees
+        self.keep = int(spec.get("keep_first") or 0) if self.window or self.chunk else 0
         self.norm_scope = spec.get("qk_norm_scope") or "head"
         if self.norm_scope not in ("head", "projection"):
             raise ValueError(f"qk_norm_scope must be 'head' or 'projection', got {self.norm_scope!r}")
@@ -347,7 +410,7 @@ class GQAttention:
 
     def cache_need(self) -> CacheNeed:
         return CacheNeed(kind="kv_pages", kv_heads=self.num_kv_heads, head_dim=self.row_dim,
-                         window=self.window or None, chunk=self.chunk or None)
+                         window=self.window or None, chunk=self.chunk or None, keep=self.keep)
 
     def parts(self):
         return [self.q_norm, self.k_norm, self.position, self.value_position]
@@ -451,7 +514,7 @@ class GQAttention:
             q_heads, cache, ctx, scale=self.scale, window=self.window, chunk=self.chunk, softcap=self.softcap, gate=gate,
             gate_per_head=per_head_gate, split_decode=self.split_decode, flash=self.flash,
             project=self.o if summands and self.value_position is None else None, sink=self.sink,
-            bias=self.distance_bias)
+            bias=self.distance_bias, keep=self.keep)
         if projected:
             return out
         if self.value_position is not None:
@@ -496,7 +559,8 @@ class GQAttention:
         ops.paged_attention_tile(q_rows, cache.pool, out, cache.block_tables, tiles["tile_request"],
                                  tiles["tile_start"], tiles["tile_length"], ctx.positions, self.scale, self.window,
                                  self.chunk, gate=gate, softcap=self.softcap,
-                                 gate_per_head=self.gate_scope == "head", sink=self.sink, bias=self.distance_bias)
+                                 gate_per_head=self.gate_scope == "head", sink=self.sink, bias=self.distance_bias,
+                                 keep=self.keep)
         if self.value_position is not None:
             out = self._turn_values(out.view(tokens, self.out_size), ctx, back=True)
         return self.o.forward(out.view(tokens, self.out_size), out_dtype=out_dtype)
@@ -505,4 +569,10 @@ class GQAttention:
         return self.qkv.weight_bytes() + self.o.weight_bytes()
 
 
-register_part("mixer", "gqa_attention", lambda spec, weights, runtime: GQAttention(spec, weights, runtime))
+def _build(spec: PartSpec, weights: WeightStore, runtime: Runtime) -> GQAttention:
+    if spec.get("pad_heads"):
+        spec, weights = padded_heads(spec, weights, runtime)
+    return GQAttention(spec, weights, runtime)
+
+
+register_part("mixer", "gqa_attention", _build)

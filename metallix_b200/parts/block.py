@@ -32,8 +32,9 @@ x <- x + norm(input(x, token)).
 
 ``parallel_residual`` lets both sublayers read the same input:
 x' = x + m (mixer(norm1(x)) + feed_forward(norm2(x))) with a constant m, the
-feed-forward being optional. What the layer leaves is a ``PairSum`` (the two
-results and m); the next layer's first kernel adds it to the stream and makes
+feed-forward being optional; with ``shared_norm`` both read the output of the one
+norm there is. What the layer leaves is a ``PairSum`` (the two results and m, and
+whatever else joins the stream ahead of the next layer); the next layer's first kernel adds it to the stream and makes
 both of that layer's norms from one pass over the row (two RMS norms of the
 same row share its mean square).
 """
@@ -304,18 +305,20 @@ register_part("block", "conv_prenorm_residual",
 
 @dataclass
 class PairSum:
-    """Two sublayers' results on their way into the residual stream: x += scale * (first + second)."""
+    """Two sublayers' results on their way into the residual stream: x += scale * (first + second) + extra."""
 
-    first: torch.Tensor
+    first: Optional[torch.Tensor]
     second: Optional[torch.Tensor]
     scale: float
+    extra: Optional[torch.Tensor] = None      # float32
 
     def settle(self, residual: torch.Tensor) -> None:
-        ops.pair_add_rmsnorm(residual, self.first, self.second, self.scale, None, None, 0.0, torch.float32)
+        ops.pair_add_rmsnorm(residual, self.first, self.second, self.scale, None, None, 0.0, torch.float32, c=self.extra)
 
 
 class ParallelResidualBlock:
-    """x <- x + m (mixer(norm1(x)) + feed_forward(norm2(x))): both sublayers on the same x."""
+    """x <- x + m (mixer(norm1(x)) + feed_forward(norm2(x))): both sublayers on the same x, or (``shared_norm``) on the
+    same norm1(x)."""
 
     kind = "parallel_residual"
 
@@ -327,7 +330,7 @@ class ParallelResidualBlock:
         self.mixer = build_part("mixer", layer.mixer, weights, runtime)
         self.feed_forward = build_part("feed_forward", layer.feed_forward, weights, runtime)
         self.feed_forward_norm = None
-        if self.feed_forward is not None:
+        if self.feed_forward is not None and not layer.block.get("shared_norm"):
             if layer.feed_forward_norm is None:
                 raise ValueError(f"{layer.name}: a feed-forward needs its norm")
             self.feed_forward_norm = build_part("norm", layer.feed_forward_norm, weights, runtime)
@@ -342,20 +345,20 @@ class ParallelResidualBlock:
         return [self.mixer_norm, self.mixer, self.feed_forward_norm, self.feed_forward]
 
     def forward(self, residual: torch.Tensor, pending, ctx: StepContext, cache: CacheView):
-        first = second = None
+        first = second = extra = None
         scale = 1.0
         if isinstance(pending, PairSum) and self.fused:
-            first, second, scale = pending.first, pending.second, pending.scale
+            first, second, scale, extra = pending.first, pending.second, pending.scale, pending.extra
         elif pending is not None:
             settle(residual, pending)
         if self.fused:
             second_weight = self.feed_forward_norm.weight if self.feed_forward_norm is not None else None
             normed = ops.pair_add_rmsnorm(residual, first, second, scale, self.mixer_norm.weight, second_weight,
-                                          self.mixer_norm.eps, self.dtype)
-            mixer_in, feed_in = normed if second_weight is not None else (normed, None)
+                                          self.mixer_norm.eps, self.dtype, c=extra)
+            mixer_in, feed_in = normed if second_weight is not None else (normed, normed)
         else:
             mixer_in = self.mixer_norm.forward(residual, self.dtype)
-            feed_in = self.feed_forward_norm.forward(residual, self.dtype) if self.feed_forward is not None else None
+            feed_in = self.feed_forward_norm.forward(residual, self.dtype) if self.feed_forward_norm is not None else mixer_in
         mixed = self.mixer.forward(mixer_in, ctx, cache)
         fed = self.feed_forward.forward(feed_in, ctx) if self.feed_forward is not None else None
         return PairSum(mixed, fed, self.scale)

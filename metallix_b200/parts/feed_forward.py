@@ -7,7 +7,7 @@ gelu in SiLU's place, in every kernel that holds the activation;
 and u = clamp(up, -limit, limit), g sigmoid(1.702 g) (u + 1).
 
 ``dense_ff`` is the feed-forward without a gate: d = act(m Wu^T) Wd^T, the
-activation a parameter (``relu_squared``: max(z, 0)^2).
+activation a parameter (``relu_squared``: max(z, 0)^2; ``gelu``: its exact form).
 
 ``routed_experts`` is a mixture of such feed-forwards: a router picks ``top``
 of ``experts`` (+ ``identity`` outputs that stand for experts returning their
@@ -20,7 +20,10 @@ groups of neighbouring experts; ``scale`` multiplies the weights;
 down(silu(gate(h)) * up(h)); ``shared`` names a gated feed-forward that every
 token uses, added behind a sigmoid gate of one number per token, or as it is
 without ``shared_gate``; ``scores="chosen"`` chooses by the logits plus
-``logit_bias`` and weighs by the softmax over the chosen ones alone."""
+``logit_bias`` and weighs by the softmax over the chosen ones alone;
+``normalized=False`` takes the chosen scores as weights as they are;
+``weigh_input`` lets a weight multiply what its expert reads, expert(w h),
+instead of what it leaves."""
 from __future__ import annotations
 
 import torch
@@ -85,7 +88,7 @@ register_part("feed_forward", "swiglu", lambda spec, weights, runtime: SwiGLU(sp
 
 class DenseFeedForward:
     kind = "dense_ff"
-    ACTIVATIONS = {"relu_squared": ops.relu_squared}
+    ACTIVATIONS = {"relu_squared": ops.relu_squared, "gelu": ops.gelu}
 
     def __init__(self, spec: PartSpec, weights: WeightStore, runtime: Runtime):
         hidden, inter = spec["hidden_size"], spec["intermediate_size"]
@@ -100,6 +103,10 @@ class DenseFeedForward:
         self.intermediate_size = inter
 
     def forward(self, x: torch.Tensor, ctx: StepContext) -> torch.Tensor:
+        if self.up.dtype == torch.bfloat16 and self.activation is ops.gelu and x.shape[0] >= FUSED_ACTIVATION_ROWS:
+            from .. import tensor_core
+            if tensor_core.supports(x, self.up.weight, torch.bfloat16):
+                return self.down.forward(tensor_core.gemm_gelu(x, self.up.weight))     # in the product's epilogue
         return self.down.forward(self.activation(self.up.forward(x)))
 
     def weight_bytes(self) -> int:
@@ -121,7 +128,8 @@ class RoutedExperts:
 
     kind = "routed_experts"
     ROUTED_TOKENS = 1     # from two tokens on experts are shared often enough for the grouped products to read less
-    ACTIVATIONS = ("relu_squared", "swiglu")
+    ACTIVATIONS = ("relu_squared", "swiglu", "gelu")
+    SHARED_WASTE = 1.5    # at most this many rows computed per row of a shared expert that is cut into experts
 
     def __init__(self, spec: PartSpec, weights: WeightStore, runtime: Runtime):
         hidden, ff = spec["hidden_size"], spec["intermediate_size"]
@@ -131,29 +139,42 @@ class RoutedExperts:
             raise ValueError(f"top {self.top} of {outputs} router outputs (at most {ops.ROUTER_OUTPUTS}) cannot be chosen")
         if spec["activation"] not in self.ACTIVATIONS:
             raise ValueError(f"activation {spec['activation']!r}; one of {self.ACTIVATIONS}")
-        self.gated = spec["activation"] == "swiglu"
+        self.activation = spec["activation"]
+        self.gated = self.activation == "swiglu"
+        self.normalized, self.weigh_input = bool(spec.get("normalized", True)), bool(spec.get("weigh_input", False))
         self.scores = spec.get("scores") or "softmax"
         self.groups = tuple(int(v) for v in spec["groups"]) if spec.get("groups") else None
         self.weight_scale = float(spec.get("scale") or 1.0)
+        if self.weigh_input and (self.activation != "gelu" or self.identity):
+            raise ValueError("weights on the experts' inputs are built for gelu experts without identity outputs")
         if self.scores not in ops.ROUTE_SCORES:
             raise ValueError(f"scores {self.scores!r}; one of {sorted(ops.ROUTE_SCORES)}")
         if self.groups is not None:
             count, keep = self.groups
             if count < 1 or outputs % count or not 1 <= keep <= count or keep * (outputs // count) < self.top:
                 raise ValueError(f"{count} groups of which {keep} are kept do not fit {outputs} outputs and top {self.top}")
-        # A shared expert without a gate that looks like the others is one more of them, chosen by every token with
-        # weight 1: its work then rides in the same launches.
+        # A shared expert without a gate, of the others' form, is as many more of them as its width takes (the sum over
+        # its inner values cut into runs of ff, the last one filled up with zeros, which the activations leave zero),
+        # chosen by every token with weight 1: its work then rides in the same launches.
         shared = spec.get("shared")
-        self.always = int(shared is not None and spec.get("shared_gate") is None and self.identity == 0 and not self.gated
-                          and shared.kind == "dense_ff" and shared["activation"] == spec["activation"]
-                          and shared["intermediate_size"] == ff)
-        names = [(spec["up_proj"].format(index), spec["down_proj"].format(index)) for index in range(self.experts)]
+        self.always = 0
+        if (shared is not None and spec.get("shared_gate") is None and self.identity == 0 and not self.gated
+                and shared.kind == "dense_ff" and shared["activation"] == spec["activation"]):
+            pieces = -(-shared["intermediate_size"] // ff)
+            if pieces * ff <= self.SHARED_WASTE * shared["intermediate_size"]:
+                self.always = pieces
+        pairs = [(weights.take(spec["up_proj"].format(index)), weights.take(spec["down_proj"].format(index)))
+                 for index in range(self.experts)]
         if self.always:
-            names.append((shared["up_proj"], shared["down_proj"]))
-        self.stacked = len(names)
+            up, down = weights.take(shared["up_proj"]), weights.take(shared["down_proj"])
+            if tuple(up.shape) != (shared["intermediate_size"], hidden) or tuple(down.shape) != (hidden, shared["intermediate_size"]):
+                raise ValueError(f"shared expert: up is {tuple(up.shape)}, down is {tuple(down.shape)}")
+            extra = self.always * ff - shared["intermediate_size"]
+            up, down = torch.nn.functional.pad(up, (0, 0, 0, extra)), torch.nn.functional.pad(down, (0, extra))
+            pairs += [(up[i * ff:(i + 1) * ff], down[:, i * ff:(i + 1) * ff]) for i in range(self.always)]
+        self.stacked = len(pairs)
         ups, downs = [], []
-        for index, (up_name, down_name) in enumerate(names):
-            up, down = weights.take(up_name), weights.take(down_name)
+        for index, (up, down) in enumerate(pairs):
             if tuple(up.shape) != (ff, hidden) or tuple(down.shape) != (hidden, ff):
                 raise ValueError(f"expert {index}: up is {tuple(up.shape)}, down is {tuple(down.shape)}; "
                                  f"expected {(ff, hidden)} and {(hidden, ff)}")
@@ -205,18 +226,25 @@ class RoutedExperts:
     def _routed(self, x: torch.Tensor, logits: torch.Tensor) -> torch.Tensor:
         chosen, weights, dense, on_identity = ops.route_experts(logits, self.correction, self.experts, self.top,
                                                                 scores=self.scores, groups=self.groups,
-                                                                scale=self.weight_scale, always=self.always)
+                                                                scale=self.weight_scale, always=self.always,
+                                                                normalized=self.normalized)
         if self.up is None:     # identity experts only
             return ops.experts_add_identity(torch.zeros(x.shape, dtype=torch.float32, device=x.device), x, on_identity)
         if x.shape[0] > self.ROUTED_TOKENS and self.grouped(x):
             from .. import tensor_core
             position, tile_group, rows = ops.expert_rows(chosen, self.stacked)
-            act = tensor_core.gemm_grouped(ops.expert_gather_rows(x, position, rows), self.up.weight, tile_group,
-                                           self.stacked, tensor_core.SWIGLU if self.gated else tensor_core.RELU_SQUARED)
+            row_scale = None
+            if self.weigh_input:    # the rows of the first product are scaled ahead of the activation
+                gathered, row_scale = ops.expert_gather_rows(x, position, rows, weights)
+            else:
+                gathered = ops.expert_gather_rows(x, position, rows)
+            epilogue = {"swiglu": tensor_core.SWIGLU, "gelu": tensor_core.GELU, "relu_squared": tensor_core.RELU_SQUARED}
+            act = tensor_core.gemm_grouped(gathered, self.up.weight, tile_group, self.stacked, epilogue[self.activation],
+                                           row_scale=row_scale)
             out = tensor_core.gemm_grouped(act, self.down.weight, tile_group, self.stacked, tensor_core.STORE_F32)
-            return ops.expert_combine_rows(out, position, weights, on_identity, x)
+            return ops.expert_combine_rows(out, position, None if self.weigh_input else weights, on_identity, x)
         return ops.experts_routed(x, self.up.weight, self.down.weight, chosen, weights, self.stacked,
-                                  self.intermediate_size, gated=self.gated)
+                                  self.intermediate_size, activation=self.activation, weigh_input=self.weigh_input)
 
     def grouped(self, x: torch.Tensor) -> bool:
         """Whether the grouped tensor-core products take this step."""

@@ -24,6 +24,11 @@ positions (its own included), ``sink`` adds one more key without a value to
 every query's softmax, with one score for all heads (a number) or a learned
 score per head (a tensor's name); both reach whichever kernel serves the step.
 
+``gate_proj`` multiplies the concatenated heads by sigmoid(a Wg^T) ahead of the
+output projection: inside the attention kernels with per-head rows, behind the
+widening with latent ones. Whatever is projected straight from the input is one
+product.
+
 ``cache_mode="heads"`` keeps the equations in their first order instead: every
 position's latent is widened once, when it arrives, to each head's key
 [k_h | rot(kr)] and value v_h, and those rows are cached per head (padded
@@ -39,7 +44,8 @@ import torch
 from .. import ops
 from ..config.spec import CacheNeed, PartSpec
 from .attention import attend_cached, attention_tiles, tiles_of
-from .linear import Linear
+from .linear import Linear, stacked_rows
+from .norm import RMSNorm
 from .registry import CacheView, Runtime, StepContext, WeightStore, build_part, register_part
 
 
@@ -66,13 +72,13 @@ class LatentAttention:
             return weight
 
         if self.q_rank:
-            self.dq = Linear(matrix("q_down_proj", (self.q_rank, hidden)), runtime)
+            query = matrix("q_down_proj", (self.q_rank, hidden))
             self.uq = Linear(matrix("q_up_proj", (H * (D + R), self.q_rank)), runtime)
             self.q_norm = build_part("norm", spec["q_norm"], weights, runtime)
         else:   # queries straight from the mixer's input
-            self.dq, self.q_norm = None, None
-            self.uq = Linear(matrix("q_proj", (H * (D + R), hidden)), runtime)
-        self.dkv = Linear(matrix("kv_down_proj", (self.width, hidden)), runtime)
+            query, self.uq, self.q_norm = matrix("q_proj", (H * (D + R), hidden)), None, None
+        down = matrix("kv_down_proj", (self.width, hidden))
+        gate = matrix("gate_proj", (H * V, hidden)) if spec.get("gate_proj") else None
         self.window = int(spec.get("window") or 0)
         sink = spec.get("sink")
         if isinstance(sink, str):
@@ -99,6 +105,19 @@ class LatentAttention:
         if mode == "heads" and not self.head_size:
             raise ValueError(f"keys of {D + R} and values of {V} do not fit a head of up to 256 values")
         self.per_head = mode == "heads" or (mode == "auto" and bool(self.head_size))
+        # One product of the input: the gate's rows (one per value of the attention kernel's heads, so that it can
+        # read them as they lie), the latent's, the queries'.
+        self.gate_rows = 0
+        stacked = [down, query]
+        if gate is not None:
+            wide = self.head_size if self.per_head else V
+            rows = torch.zeros((H, wide, hidden), dtype=gate.dtype, device=gate.device)
+            rows[:, :V] = gate.view(H, V, hidden)
+            stacked.insert(0, rows.view(H * wide, hidden))
+            self.gate_rows = H * wide
+        self.query_at = self.gate_rows + self.width
+        self.query_rows = query.shape[0]
+        self.inputs = stacked_rows(stacked, runtime)
         if self.per_head:
             hd = self.head_size
             # keys and values from the latent in one product: rows of uk, then rows of uv
@@ -116,11 +135,15 @@ class LatentAttention:
             return CacheNeed(kind="kv_pages", kv_heads=self.heads, head_dim=self.head_size, window=self.window or None)
         return CacheNeed(kind="kv_pages", kv_heads=1, head_dim=self.width, planes=1, window=self.window or None)
 
-    def _queries(self, x: torch.Tensor) -> torch.Tensor:
+    def _queries(self, proj: torch.Tensor, positions: torch.Tensor) -> torch.Tensor:
         """[tokens, H * (D + R)]: through their own normed latent, or straight from the input."""
-        if self.dq is None:
-            return self.uq.forward(x)
-        return self.uq.forward(self.q_norm.forward(self.dq.forward(x), self.dtype))
+        query = proj[:, self.query_at:self.query_at + self.query_rows]
+        if self.uq is None:
+            return query
+        if isinstance(self.q_norm, RMSNorm):     # rows of the wider product, read where they lie
+            return self.uq.forward(ops.latent_cache(query, self.q_norm.weight, self.q_norm.eps, self.q_rank, None, None,
+                                                    positions, None, None, False))
+        return self.uq.forward(self.q_norm.forward(query.contiguous(), self.dtype))
 
     def parts(self):
         return [self.q_norm, self.kv_norm, self.position]
@@ -132,12 +155,14 @@ class LatentAttention:
         paired = bool(getattr(self.position, "interleaved", False))
         if self.per_head:
             return self._forward_per_head(x, ctx, cache, cos, sin, paired)
+        proj = self.inputs.forward(x)
+        latent = proj[:, self.gate_rows:self.query_at]
         # the position's cache row: normed latent, rotated shared key part
         if cache.write and cache.slots is not None:
-            ops.latent_cache(self.dkv.forward(x), self.kv_norm.weight, self.kv_norm.eps, r, cache.pool, cache.slots,
+            ops.latent_cache(latent, self.kv_norm.weight, self.kv_norm.eps, r, cache.pool, cache.slots,
                              ctx.positions, cos, sin, paired)
         # queries: through their own latent, then onto the cache's side
-        q = self._queries(x)                                                            # [tokens, H * (D + R)]
+        q = self._queries(proj, ctx.positions)                                          # [tokens, H * (D + R)]
         q_heads = q.view(tokens, H, D + R)
         q_cache = torch.empty((tokens, H, self.width), dtype=self.dtype, device=x.device)
         if self.dtype == torch.float32:
@@ -158,30 +183,32 @@ class LatentAttention:
                 ops.gemm_simple(mixed[:, h, :], self.uv[h], out=values[:, h * V:(h + 1) * V])
         else:
             values = torch.bmm(mixed.transpose(0, 1), self.uv.transpose(1, 2)).transpose(0, 1).reshape(tokens, H * V)
+        if self.gate_rows:
+            values = ops.sigmoid_gate(values, proj[:, :self.gate_rows])
         return self.o.forward(values)
 
     def _forward_per_head(self, x, ctx: StepContext, cache: CacheView, cos, sin, paired: bool) -> torch.Tensor:
         tokens, H, D, R, V, r, hd = x.shape[0], self.heads, self.dim, self.rot, self.vdim, self.rank, self.head_size
+        proj = self.inputs.forward(x)
         # [normed latent | rotated shared key part] of this step's tokens, then every head's keys and values
-        rows = ops.latent_cache(self.dkv.forward(x), self.kv_norm.weight, self.kv_norm.eps, r, None, None,
+        rows = ops.latent_cache(proj[:, self.gate_rows:self.query_at], self.kv_norm.weight, self.kv_norm.eps, r, None, None,
                                 ctx.positions, cos, sin, paired)
         widened = self.kv_up.forward(rows[:, :r])                                       # [tokens, H * D + H * V]
-        q = self._queries(x)                                                            # [tokens, H * (D + R)]
+        q = self._queries(proj, ctx.positions)                                          # [tokens, H * (D + R)]
         q_heads = torch.empty((tokens, H, hd), dtype=self.dtype, device=x.device)
         write = cache.write and cache.slots is not None
         ops.latent_heads(q, widened, rows, r, q_heads, cache.pool if write else None, cache.slots if write else None,
                          ctx.positions, cos, sin, paired, D, R, V)
         out, _ = attend_cached(q_heads, cache, ctx, scale=self.scale, window=self.window, split_decode=self.split_decode,
-                               flash=self.flash, sink=self.sink)
+                               flash=self.flash, sink=self.sink, gate=proj[:, :self.gate_rows] if self.gate_rows else None)
         return self.o.forward(out.view(tokens, H * hd))
 
     def weight_bytes(self) -> int:
-        queries = self.uq.weight_bytes() + (self.dq.weight_bytes() if self.dq is not None else 0)
+        inputs = self.inputs.weight_bytes() + (self.uq.weight_bytes() if self.uq is not None else 0)
         if self.per_head:
-            return queries + self.dkv.weight_bytes() + self.o.weight_bytes() + self.kv_up.weight_bytes()
+            return inputs + self.o.weight_bytes() + self.kv_up.weight_bytes()
         element = self.uk.element_size()
-        return (queries + self.dkv.weight_bytes() + self.o.weight_bytes()
-                + (self.uk.numel() + self.uv.numel()) * element)
+        return (inputs + self.o.weight_bytes() + (self.uk.numel() + self.uv.numel()) * element)
 
 
 register_part("mixer", "latent_attention", lambda spec, weights, runtime: LatentAttention(spec, weights, runtime))

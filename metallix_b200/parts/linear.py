@@ -47,3 +47,14 @@ class Linear:
 
     def weight_bytes(self) -> int:
         return self.weight.numel() * self.weight.element_size()
+
+
+def stacked_rows(matrices: Sequence[torch.Tensor], runtime: Runtime, multiple: int = 8) -> Linear:
+    """One product over the same input, with rows of zeros at the end so that a
+    row of the result starts on the boundary that vector accesses need."""
+    rows = sum(m.shape[0] for m in matrices)
+    extra = -rows % multiple
+    if extra:
+        matrices = list(matrices) + [torch.zeros((extra, matrices[0].shape[1]), dtype=matrices[0].dtype,
+                                                 device=matrices[0].device)]
+    return Linear.stacked(matrices, runtime)

@@ -3,7 +3,8 @@ directly (crates/models/qwen/src/forward.rs:2442-2449). Sum of squares and
 scale are float32 in both precisions. A checkpoint may store the weight around
 zero (``one_plus``): the factor is then 1 + w, formed once in float32 when the
 part is built. It may also store one number for all coordinates (``scalar``)
-or none at all (the row over its root mean square).
+or none at all (the row over its root mean square). ``scale`` multiplies the
+factor by a constant.
 
 Dynamic Tanh: y = tanh(alpha * x) * w + b with a scalar alpha, computed value
 by value in float32; it takes no mean or variance of the row, so it has no
@@ -23,9 +24,11 @@ class RMSNorm:
     kind = "rmsnorm"
     adds_summands = True   # add_forward also takes [parts, rows, size]: a sum its producer left in parts
 
-    def __init__(self, weight: torch.Tensor, eps: float, runtime: Runtime, one_plus: bool = False):
+    def __init__(self, weight: torch.Tensor, eps: float, runtime: Runtime, one_plus: bool = False,
+                 scale: float = 1.0):
         weight = weight.to(device=runtime.device, dtype=torch.float32)
-        self.weight = (weight + 1.0 if one_plus else weight).contiguous()
+        weight = weight + 1.0 if one_plus else weight
+        self.weight = (weight * scale if scale != 1.0 else weight).contiguous()
         self.size = self.weight.numel()
         self.eps = float(eps)
 
@@ -62,8 +65,9 @@ class RMSNorm:
 def _build(spec: PartSpec, weights: WeightStore, runtime: Runtime) -> RMSNorm:
     """``weight`` None: the row over its root mean square and nothing else;
     ``scalar``: the stored weight is one number for all coordinates."""
+    scale = float(spec.get("scale", 1.0))
     if spec.get("weight") is None:
-        return RMSNorm(torch.ones(spec["size"]), spec["eps"], runtime)
+        return RMSNorm(torch.ones(spec["size"]), spec["eps"], runtime, scale=scale)
     weight = weights.take(spec["weight"])
     if spec.get("scalar"):
         if weight.numel() != 1:
@@ -71,7 +75,7 @@ def _build(spec: PartSpec, weights: WeightStore, runtime: Runtime) -> RMSNorm:
         weight = weight.to(torch.float32).reshape(1).expand(spec["size"])
     if weight.numel() != spec["size"]:
         raise ValueError(f"{spec['weight']} has {weight.numel()} values, the norm is over {spec['size']}")
-    return RMSNorm(weight, spec["eps"], runtime, one_plus=bool(spec.get("one_plus", False)))
+    return RMSNorm(weight, spec["eps"], runtime, one_plus=bool(spec.get("one_plus", False)), scale=scale)
 
 
 register_part("norm", "rmsnorm", _build)

@@ -31,7 +31,7 @@ import torch
 
 from .. import ops
 from ..config.spec import CacheNeed, PartSpec
-from .linear import Linear
+from .linear import Linear, stacked_rows
 from .registry import CacheView, Prepared, Runtime, StepContext, StepPlan, WeightStore, register_part
 
 
@@ -333,17 +333,6 @@ def _named(spec: PartSpec, weights: WeightStore, runtime: Runtime):
     return matrix, vector
 
 
-def _stacked_rows(matrices, runtime: Runtime, multiple: int = 8) -> Linear:
-    """One product over the same input, with rows of zeros at the end so that a
-    row of the result starts on the boundary that vector accesses need."""
-    rows = sum(m.shape[0] for m in matrices)
-    extra = -rows % multiple
-    if extra:
-        matrices = list(matrices) + [torch.zeros((extra, matrices[0].shape[1]), dtype=matrices[0].dtype,
-                                                 device=matrices[0].device)]
-    return Linear.stacked(matrices, runtime)
-
-
 class HeadDelta:
     """The gated delta rule with one decay per head. As ``ChannelDelta``, but
 
@@ -378,7 +367,7 @@ class HeadDelta:
             stacked.append(matrix(name, (rows, hidden)))
             self.offsets[name] = cursor
             cursor += rows
-        self.inputs = _stacked_rows(stacked, runtime)
+        self.inputs = stacked_rows(stacked, runtime)
         self.step_bias = vector("step_bias", H)
         self.rate = torch.exp(vector("a_log", H)).contiguous()
         self.norm_weight = vector("norm", V).repeat(H).contiguous()       # one weight over V, the same for every head
@@ -454,7 +443,7 @@ class StateSpaceDual:
             raise ValueError(f"{N} states per value column; the recurrence takes up to {ops.delta_rule_max_dim()}")
         matrix, vector = _named(spec, weights, runtime)
         self.conv_channels = self.inner + 2 * G * N
-        self.inputs = _stacked_rows([matrix("in_proj", (2 * self.inner + 2 * G * N + H, hidden))], runtime)
+        self.inputs = stacked_rows([matrix("in_proj", (2 * self.inner + 2 * G * N + H, hidden))], runtime)
         self.conv = ShortConv(PartSpec("short_conv", {
             "channels": self.conv_channels, "taps": int(spec["conv_taps"]), "weight": spec["conv_weight"],
             "bias": spec["conv_bias"], "activation": "silu"}), weights, runtime)
@@ -491,3 +480,60 @@ class StateSpaceDual:
 
 
 register_part("mixer", "state_space_dual", lambda spec, weights, runtime: StateSpaceDual(spec, weights, runtime))
+
+
+class Lightning:
+    """Linear attention with a constant decay per head (lightning attention):
+
+        q = silu(a Wq^T), k = silu(a Wk^T)  (H x D),   v = silu(a Wv^T)  (H x V)
+        S <- decay_h S + k v^T,   o = S^T q                                per head
+
+    The heads side by side over their common root mean square, times a weight,
+    times sigmoid(a Wg^T), then Wo. S (float32, kept transposed as ``[H, V, D]``)
+    is kept per request in the cache's state slots. One product gives q, k, v and
+    the gate ahead of their activations; the silus, the recurrence and the norm
+    are float32 in both precisions."""
+
+    kind = "lightning"
+    graph_safe = True
+    step_key = "request_rows"
+    prepare_step = staticmethod(request_rows)
+
+    def __init__(self, spec: PartSpec, weights: WeightStore, runtime: Runtime):
+        hidden = spec["hidden_size"]
+        self.heads, self.dim, self.vdim = int(spec["num_heads"]), int(spec["head_dim"]), int(spec["value_dim"])
+        self.eps = float(spec["eps"])
+        H, D, V = self.heads, self.dim, self.vdim
+        if not 0 < D <= ops.delta_rule_max_dim():
+            raise ValueError(f"keys of {D} channels; the recurrence takes up to {ops.delta_rule_max_dim()}")
+        decay = [float(value) for value in spec["decay"]]
+        if len(decay) != H or not all(0.0 <= value <= 1.0 for value in decay):
+            raise ValueError(f"decay must hold one number in [0, 1] per head ({H}), got {decay}")
+        self.decay = torch.tensor(decay, dtype=torch.float32).to(runtime.device)
+        matrix, vector = _named(spec, weights, runtime)
+        self.inputs = stacked_rows([matrix("q_proj", (H * D, hidden)), matrix("k_proj", (H * D, hidden)),
+                                    matrix("v_proj", (H * V, hidden)), matrix("gate_proj", (H * V, hidden))], runtime)
+        self.norm_weight = vector("norm", H * V)
+        self.o = Linear(matrix("o_proj", (hidden, H * V)), runtime)
+        self.dtype = runtime.dtype
+
+    def cache_need(self) -> CacheNeed:
+        return CacheNeed(kind="state", state_shape=(self.heads, self.vdim, self.dim), state_dtype="float32")
+
+    def forward(self, x: torch.Tensor, ctx: StepContext, cache: CacheView) -> torch.Tensor:
+        if cache.state is None:
+            raise ValueError("the lightning mixer needs a state entry of the cache")
+        rows = request_rows_of(ctx)
+        H, D, V = self.heads, self.dim, self.vdim
+        proj = self.inputs.forward(x)       # every later step reads column ranges of it in place
+        mixed = ops.lightning_attention(proj, (0, H * D, 2 * H * D), self.decay, cache.state, rows["row_start"],
+                                        rows["row_length"], ctx.request_slots, H, D, V, longest=rows.get("longest", 0))
+        at = 2 * H * D + H * V
+        return self.o.forward(ops.gated_norm(mixed, self.norm_weight, proj[:, at:at + H * V], 1, self.eps, self.dtype,
+                                             activation="sigmoid", behind=True))
+
+    def weight_bytes(self) -> int:
+        return self.inputs.weight_bytes() + self.o.weight_bytes()
+
+
+register_part("mixer", "lightning", lambda spec, weights, runtime: Lightning(spec, weights, runtime))

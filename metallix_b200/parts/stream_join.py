@@ -5,7 +5,11 @@ x0 being the stream as the embedding left it, and (optional) a learned vector of
 the turn is added, x <- x + step[t]. A model whose layers run several times in a
 row does this once per pass, so that a pass knows which one it is. The product's
 result is the new stream (float32); the vector rides into the next layer's first
-kernel as what is still to be added to every row."""
+kernel as what is still to be added to every row.
+
+``add_first`` adds the embedding output to the stream, x <- x + x0, with what is
+still pending in the same pass: the sum rides into the next layer's first kernel
+as a third summand."""
 from __future__ import annotations
 
 from typing import Optional
@@ -14,6 +18,7 @@ import torch
 
 from .. import ops
 from ..config.spec import PartSpec
+from .block import PairSum
 from .linear import Linear
 from .registry import Runtime, WeightStore, register_part, settle
 
@@ -48,4 +53,23 @@ class MixFirst:
         return self.mix.weight_bytes()
 
 
+class AddFirst:
+    kind = "add_first"
+
+    def __init__(self, spec: PartSpec, weights: WeightStore, runtime: Runtime):
+        pass
+
+    def forward(self, residual: torch.Tensor, pending, first: torch.Tensor, turn: int):
+        if first.data_ptr() == residual.data_ptr():      # the stream is still the embedding output itself
+            residual = residual.clone()
+        if isinstance(pending, PairSum) and pending.extra is None:
+            return residual, PairSum(pending.first, pending.second, pending.scale, extra=first)
+        settle(residual, pending)
+        return residual, PairSum(None, None, 1.0, extra=first)
+
+    def weight_bytes(self) -> int:
+        return 0
+
+
+register_part("join", "add_first", lambda spec, weights, runtime: AddFirst(spec, weights, runtime))
 register_part("join", "mix_first", lambda spec, weights, runtime: MixFirst(spec, weights, runtime))

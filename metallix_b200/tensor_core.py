@@ -8,7 +8,7 @@ import torch
 
 from . import ops
 
-STORE_BF16, STORE_F32, SWIGLU, RELU_SQUARED, GEGLU, CLAMPED_GLU = 0, 1, 2, 3, 4, 5
+STORE_BF16, STORE_F32, SWIGLU, RELU_SQUARED, GEGLU, CLAMPED_GLU, GELU = 0, 1, 2, 3, 4, 5, 6
 
 
 def why_not(a: torch.Tensor, w: torch.Tensor, out_dtype: torch.dtype) -> str:
@@ -68,11 +68,23 @@ def gemm_swiglu(a: torch.Tensor, gate_up: torch.Tensor, out: Optional[torch.Tens
     return _launch(out, a, gate_up, inter, {"silu": SWIGLU, "gelu_tanh": GEGLU, "clamped": CLAMPED_GLU}[activation], limit)
 
 
-def gemm_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, groups: int, epilogue: int) -> torch.Tensor:
+def gemm_gelu(a: torch.Tensor, w: torch.Tensor) -> torch.Tensor:
+    """gelu(a w^T) in its exact form, bfloat16 [m, n], the activation in the product's epilogue."""
+    reason = why_not(a, w, torch.bfloat16)
+    if reason:
+        raise ops.KernelError("the tcgen05 kernel does not take this call: " + reason)
+    out = torch.empty((a.shape[0], w.shape[0]), dtype=torch.bfloat16, device=a.device)
+    return _launch(out, a, w, w.shape[0], GELU)
+
+
+def gemm_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, groups: int, epilogue: int,
+                 row_scale: Optional[torch.Tensor] = None) -> torch.Tensor:
     """Row tile i of a ``[m, k]`` (128 rows a tile, m a whole number of them)
     times matrix tile_group[i] of w ``[groups * n, k]`` transposed; tiles with a
     negative entry are left out, and their rows of the result are not written.
-    ``epilogue``: STORE_BF16, STORE_F32, RELU_SQUARED (bfloat16 max(c, 0)^2) or
+    ``epilogue``: STORE_BF16, STORE_F32, RELU_SQUARED (bfloat16 max(c, 0)^2), GELU
+    (bfloat16 gelu(row_scale[row] c) in its exact form, ``row_scale`` float32
+    ``[m]`` or None for 1) or
     SWIGLU (every matrix of w holds its gate rows and then as many up rows;
     the result is bfloat16 silu(gate) * up, half as wide as a matrix has rows)."""
     reason = why_not(a, w, torch.bfloat16)
@@ -82,9 +94,12 @@ def gemm_grouped(a: torch.Tensor, w: torch.Tensor, tile_group: torch.Tensor, gro
               and tile_group.numel() >= a.shape[0] // 128, "the groups do not fit")
     m, group_rows = a.shape[0], w.shape[0] // groups
     ops._need(epilogue != SWIGLU or group_rows % 2 == 0, "gate and up rows must pair up")
+    if row_scale is not None:
+        ops._check(row_scale, "row_scale", (torch.float32,), 1)
+        ops._need(epilogue == GELU and row_scale.numel() == m, "row_scale is one float32 per row, for the GELU epilogue")
     n = group_rows // 2 if epilogue == SWIGLU else group_rows
     out = torch.empty((m, n), dtype=torch.float32 if epilogue == STORE_F32 else torch.bfloat16, device=a.device)
     ops._call("mxb_gemm_tcgen05_grouped", out.data_ptr(), a.data_ptr(), w.data_ptr(), tile_group.data_ptr(), m, n,
               a.shape[1], groups, group_rows, a.stride(0), w.stride(0), out.stride(0), epilogue,
-              ops.status_word(a.device).data_ptr(), ops._stream())
+              ops._ptr(row_scale), ops.status_word(a.device).data_ptr(), ops._stream())
     return out
