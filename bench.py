@@ -10,6 +10,7 @@
     python bench.py --design sadosun                              the Sadosun decoder beside Qwen3 and Zitezen at equal width and active weights
     python bench.py --design dimorax                              the Dimorax decoder beside Qwen3 and Sadosun at equal width and active weights
     python bench.py --design kokolorn                             the Kokolorn decoder beside Qwen3 and Dimorax at equal width and active weights
+    python bench.py --design mekuvik                              the Mekuvik decoder beside Qwen3 and Kokolorn at equal width and active weights
 
 Default workload: a Qwen3-0.6B-shaped model (28 layers,
 hidden 1024, 16 query and 8 key/value heads of 128, SwiGLU 3072, vocabulary
@@ -672,6 +673,9 @@ def workload(args):
             config = parse_config(dict(other, layers=other["layers"][:4] if layers <= 4 else other["layers"][:layers]))
         elif args.design == "kokolorn":   # all eight layer runs (two layers of them looped), or its first layers without the loop
             other = _kokolorn(hidden, heads, kv_heads, dim, inter, {"0.6b": "0.6b-layers", "8b": "8b-layers"}[args.shape])
+            config = parse_config(other if layers >= DESIGN_LAYERS else dict(other, loop=None, layers=other["layers"][:layers]))
+        elif args.design == "mekuvik":   # all eight layer runs (two layers of them looped), or its first layers without the loop
+            other = _mekuvik(hidden, heads, kv_heads, dim, inter, {"0.6b": "0.6b-layers", "8b": "8b-layers"}[args.shape])
             config = parse_config(other if layers >= DESIGN_LAYERS else dict(other, loop=None, layers=other["layers"][:layers]))
         elif args.design == "sadosun":   # its layers come in twos
             other = _sadosun(hidden, heads, kv_heads, dim, inter, {"0.6b": "0.6b-layers", "8b": "8b-layers"}[args.shape],
@@ -1807,6 +1811,220 @@ def design_kokolorn(args):
     return 0
 
 
+# Mekuvik layers at the two sizes: lightning's (heads, key channels, value columns), the latent attention's (heads,
+# unrotated and rotated key values, value width, query rank, latent width), the experts' (count, top, ff) with a shared
+# expert of the same ff, as Kokolorn's; the attention's window and kept positions. Six layers, of which the first two
+# run twice: eight layer runs.
+MEKUVIK_SIZES = {"0.6b-layers": ((16, 128, 128), (16, 96, 32, 128, 512, 256), (12, 2, 1536), (1024, 16)),
+                 "8b-layers": ((32, 128, 128), (32, 96, 32, 128, 1536, 512), (12, 2, 6144), (1024, 16))}
+
+
+def _mekuvik(hidden, heads, kv_heads, dim, inter, size):
+    (lh, ld, lv), (ch, cd, cr, cv, q_rank, rank), (count, top, ff), (window, keep) = MEKUVIK_SIZES[size]
+    experts = {"kind": "moe", "expert": {"ff": ff}, "shared": {"ff": ff}, "router": {"experts": count, "top": top}}
+    dense = {"kind": "dense", "ff": inter}
+    lightning = {"type": "lightning", "mixer": {"heads": lh, "dim": ld, "vdim": lv,
+                                                "decay": [1.0 - 0.5 ** (1.0 + 9.0 * i / (lh - 1)) for i in range(lh)]}}
+    latent = {"type": "latent_attention",
+              "mixer": {"heads": ch, "dim": cd, "rot_dim": cr, "vdim": cv, "q_rank": q_rank, "kv_rank": rank,
+                        "scale": (cd + cr) ** -0.5,
+                        "rot": {"base": 1.0e5, "dims": cr,
+                                "scaling": {"factor": 16.0, "original": 2048, "fast": 24.0, "slow": 1.0}}}}
+    attention = {"type": "attention",
+                 "mixer": {"heads": heads, "kv_heads": kv_heads, "dim": dim, "vdim": dim, "scale": dim ** -0.5,
+                           "rot": {"base": 1.0e6, "dims": dim // 2}, "mask": {"size": window, "keep_first": keep}}}
+    return {"architecture": "Mekuvik", "vocab": DESIGN_VOCAB, "width": hidden, "norm": {"eps": 1e-6}, "logit_scale": 0.5,
+            "loop": {"start": 0, "stop": 2, "times": 2},
+            "layers": [dict(lightning, mlp=experts), dict(latent, mlp=dense), dict(attention, mlp=experts),
+                       dict(lightning, mlp=dense), dict(attention, mlp=dense), dict(latent, mlp=experts)]}
+
+
+def design_mekuvik(args):
+    """Prompt and decode throughput of the Mekuvik decoder beside the Qwen3
+    decoder (equal width, heads and active feed-forward weights) and the
+    Kokolorn decoder (the other model with passes, matrix states and experts
+    beside a shared one), random weights, bfloat16, 8 layer runs; then each
+    kernel the design adds beside the like kernel of those models: bytes that
+    must move over time against the measured copy bandwidth, or arithmetic over
+    time against the measured bf16 matrix peak. One JSON line."""
+    import numpy as np
+    import torch
+    from metallix_b200 import ops, parse_config
+    from metallix_b200.config.kokolorn import ChosenExperts
+    from metallix_b200.config.mekuvik import WeighedExperts
+    from metallix_b200.parts.registry import Runtime, WeightStore, build_part
+
+    peak, peak_source = peaks()
+    warmup, steps = max(args.warmup, 3), min(max(args.steps, 1), 64)
+    rng = np.random.default_rng(0)
+    out = {"design": "mekuvik", "beside": ["qwen3", "kokolorn"], "dtype": "bf16", "layers": DESIGN_LAYERS,
+           "vocab": DESIGN_VOCAB, "prompt_len": args.prompt_len, "peaks": peak_source, "sizes": {}}
+    for size, (hidden, heads, kv_heads, dim, inter) in ({} if args.kernels_only else DESIGN_SIZES).items():
+        configs = {"mekuvik": parse_config(_mekuvik(hidden, heads, kv_heads, dim, inter, size)),
+                   "qwen3": parse_config(dict(_qwen3(DESIGN_LAYERS, hidden, heads, kv_heads, inter, False),
+                                              vocab_size=DESIGN_VOCAB, head_dim=dim)),
+                   "kokolorn": parse_config(_kokolorn(hidden, heads, kv_heads, dim, inter, size))}
+        out["sizes"][size] = {family: _engine_numbers(config, args, peak, rng, warmup, steps)
+                              for family, config in configs.items()}
+
+    def measure(function):
+        for _ in range(3):
+            function()
+        flush = torch.empty(192 << 20, dtype=torch.uint8, device="cuda")
+        times = []
+        for _ in range(7):
+            flush.zero_()    # a buffer larger than L2 between the timed launches
+            times.append(timed(torch, "cuda", lambda _: function(), 1))
+        return statistics.median(times)
+
+    def gbs(bytes_moved, function):
+        ms = measure(function)
+        return {"us": ms * 1e3, "gb_s": bytes_moved / (ms * 1e-3) / 1e9,
+                "frac_of_copy_bandwidth": bytes_moved / (ms * 1e-3) / 1e9 / peak["hbm_gbs"]}
+
+    def tflops(flops, function):
+        ms = measure(function)
+        return {"us": ms * 1e3, "tflop_s": flops / (ms * 1e-3) / 1e12,
+                "frac_of_bf16_matrix_peak": flops / (ms * 1e-3) / 1e12 / peak["bf16_tflops"]}
+
+    ops.require_cuda()
+    kernels = {}
+    size = "8b-layers"
+    hidden, heads, kv_heads, dim, inter = DESIGN_SIZES[size]
+    (lh, ld, lv), (ch, cd, cr, cv, q_rank, rank), (count, top, ff), (window, keep) = MEKUVIK_SIZES[size]
+    _, (sh, sv, states, groups, parts, _), _, _ = KOKOLORN_SIZES[size]
+    bf16, f32 = torch.bfloat16, torch.float32
+    ints = lambda values: torch.tensor(values, dtype=torch.int32, device="cuda")
+    normal = lambda *shape: torch.randn(*shape, device="cuda")
+    prompt = args.prompt_len
+    runtime = Runtime(device=torch.device("cuda"), dtype=bf16, max_positions=args.context, gemm_backend=args.gemm)
+
+    def weights_of(shapes):
+        return WeightStore({name: (normal(*shape) * 0.02).to(bf16) for name, shape in shapes.items()})
+
+    # ---- into the residual stream and out of it; a recurrence's output; queries, keys and the cache
+    ones, inner = torch.ones(hidden, device="cuda"), lh * lv
+    for tokens in (8, prompt * 4):
+        x, a, b, first = normal(tokens, hidden), normal(tokens, hidden).to(bf16), normal(tokens, hidden).to(bf16), normal(tokens, hidden)
+        kernels[f"sublayer_input_{tokens}"] = {
+            "mekuvik: x += a + b; one norm of x": gbs(
+                tokens * hidden * (4 + 4 + 2 + 2 + 2), lambda: ops.pair_add_rmsnorm(x, a, b, 1.0, ones, None, 1e-6, bf16)),
+            "mekuvik: x += a + b + x0; one norm of x": gbs(
+                tokens * hidden * (4 + 4 + 2 + 2 + 4 + 2),
+                lambda: ops.pair_add_rmsnorm(x, a, b, 1.0, ones, None, 1e-6, bf16, c=first)),
+            "dimorax: x += m (a + b); two norms of x": gbs(
+                tokens * hidden * (4 + 4 + 2 + 2 + 2 + 2), lambda: ops.pair_add_rmsnorm(x, a, b, 0.5, ones, ones, 1e-6, bf16)),
+            "kokolorn: [x + d | x0] rounded": gbs(tokens * hidden * (4 + 2 + 4 + 4), lambda: ops.join_rows(x, a, first, bf16)),
+            "qwen3: x += d; y = norm(x)": gbs(tokens * hidden * (4 + 4 + 2 + 2), lambda: ops.add_rmsnorm(x, a, ones, 1e-6, bf16))}
+        wide, product, weight = normal(tokens, inner), normal(tokens, 2 * inner).to(bf16), torch.ones(inner, device="cuda")
+        kernels[f"recurrent_output_{tokens}"] = {
+            "mekuvik: norm of %d values, times sigmoid(gate)" % inner: gbs(
+                tokens * inner * (4 + 2 + 2), lambda: ops.gated_norm(wide, weight, product[:, :inner], 1, 1e-6, bf16,
+                                                                   activation="sigmoid", behind=True)),
+            "kokolorn: x silu(gate), then its norm": gbs(
+                tokens * inner * (4 + 2 + 2), lambda: ops.gated_norm(wide, weight, product[:, :inner], 1, 1e-6, bf16))}
+        q_width, k_width = heads * dim, kv_heads * dim
+        pages = -(-tokens // 16)
+        qk, pool = normal(tokens, q_width + k_width).to(bf16), torch.zeros(pages, 2, kv_heads, 16, dim, dtype=bf16, device="cuda")
+        q_out, at = torch.empty(tokens, heads, dim, dtype=bf16, device="cuda"), torch.arange(tokens, dtype=torch.int32, device="cuda")
+        gain, q_gain, k_gain = (torch.ones(n, device="cuda") for n in (dim, q_width, k_width))
+        half, quarter = (torch.ones(max(tokens, 8), n, device="cuda") for n in (dim // 2, dim // 4))
+        moved, keys = tokens * (2 * q_width + 4 * k_width) * 2, qk[:, q_width:]
+        kernels[f"queries_and_cache_{tokens}"] = {
+            "mekuvik: norms over the projections, pairs of half a head turned, the cache": gbs(
+                moved + tokens * dim * 2, lambda: ops.qk_norm_rope_cache(
+                    qk[:, :q_width], keys, keys, q_out, pool, at, at, q_gain, k_gain, quarter, quarter, 1e-6, interleaved=True,
+                    norm_scope="projection")),
+            "qwen3: norms of the heads, rotation, the cache": gbs(
+                moved + tokens * dim * 4, lambda: ops.qk_norm_rope_cache(qk[:, :q_width], keys, keys, q_out, pool, at, at, gain,
+                                                                         gain, half, half, 1e-6))}
+        del pool, qk, q_out
+
+    # ---- the feed-forward: experts weighed at their input, with a shared one, beside Kokolorn's
+    built = {}
+    for name, typed in (("mekuvik", WeighedExperts(ff=ff, experts=count, top=top, shared_ff=ff)),
+                        ("kokolorn", ChosenExperts(ff=ff, experts=count, top=top, shared_ff=ff))):
+        built[name] = build_part("feed_forward", typed.part("m", hidden), weights_of(typed.shapes("m", hidden)), runtime)
+    for tokens in (8, prompt * 4):
+        h, label = normal(tokens, hidden).to(bf16), f"feed_forward_{tokens}"
+        kernels[label] = {}
+        for name, part in built.items():
+            logits = part.router.forward(h, out_dtype=f32)
+            picked = ops.route_experts(logits[:, :count], part.correction, count, top, scores=part.scores)[0]
+            distinct = int(torch.unique(picked).numel())
+            if tokens == 8:     # a decode step: the weights that must be read
+                kernels[label][name + ": router, choice, %d distinct experts of %d, the shared one" % (distinct, count)] = gbs(
+                    (distinct + 1) * 2 * ff * hidden * 2 + count * hidden * 2, lambda: part.forward(h, None))
+            else:               # a prompt: the products that must be made
+                kernels[label][name + ": router, choice, the chosen experts, the shared one"] = tflops(
+                    (top + 1) * tokens * 4.0 * ff * hidden + tokens * 2.0 * count * hidden, lambda: part.forward(h, None))
+    del built, part
+
+    # ---- the mixers: a decode step of 8 requests, then a prompt in one step
+    decay = torch.linspace(0.6, 0.999, lh, device="cuda")
+    s_bias, s_rate, skip = normal(sh) - 3.0, torch.exp(normal(sh) * 0.3), normal(sh)
+
+    def recurrences(tokens, rows, lengths, slots, longest):
+        """(name, bytes of rows, bytes of state, call)."""
+        l_state, s_state = (torch.zeros(rows.numel(), *shape, device="cuda") for shape in ((lh, lv, ld), (sh, sv, states)))
+        l_in, s_in = normal(tokens, 2 * lh * ld + lh * lv).to(bf16), normal(tokens, 2 * groups * states + sh * sv).to(bf16)
+        s_side = normal(tokens, sh).to(bf16)
+        return [
+            ("mekuvik: lightning attention, %d heads of %d by %d" % (lh, ld, lv), tokens * (l_in.shape[1] * 2 + lh * lv * 4),
+             2 * l_state.numel() * 4,
+             lambda: ops.lightning_attention(l_in, (0, lh * ld, 2 * lh * ld), decay, l_state, rows, lengths, slots, lh, ld, lv,
+                                             longest=longest)),
+            ("kokolorn: state-space dual, %d heads of %d, %d states" % (sh, sv, states),
+             tokens * (s_in.shape[1] * 2 + sh * 2 + sh * sv * 4), 2 * s_state.numel() * 4,
+             lambda: ops.state_space_dual(s_in, (sh * sv + groups * states, sh * sv, 0), s_side, s_bias, s_rate, skip, s_state, rows,
+                                          lengths, slots, sh, groups, states, sv, longest=longest))]
+
+    batch, context = 8, prompt
+    rows, one_each, label = ints(range(batch)), ints([1] * batch), "decode_step_mixer_8_requests"
+    kernels[label] = {name + ", state read and written": gbs(state, call)
+                      for name, _, state, call in recurrences(batch, rows, one_each, rows, 1)}
+    pages = batch * (-(-context // 16))
+    table = torch.arange(pages, dtype=torch.int32, device="cuda").view(batch, -1)
+    positions = ints([context - 1] * batch)
+    cache, q = normal(pages, 2, kv_heads, 16, dim).to(bf16), normal(batch, heads, dim).to(bf16)
+    attended = torch.empty_like(q)
+    row_bytes = batch * 2 * kv_heads * dim * 2
+    for name, size_of, kept in (("qwen3: split-key attention over %d cached positions" % context, 0, 0),
+                                ("qwen3: the same in a window of %d" % window, window, 0),
+                                ("mekuvik: in a window of %d beside %d kept positions" % (window, keep), window, keep)):
+        kernels[label][name] = gbs(row_bytes * min(context, (size_of or context) + kept), lambda: ops.paged_attention_decode(
+            q, cache, attended, table, rows, rows, positions, dim ** -0.5, context, window=size_of, keep=kept))
+    del cache
+
+    tokens, label = prompt, f"prompt_mixer_{prompt}"
+    one_row, length = ints([0]), ints([tokens])
+    kernels[label] = {name + ", one request (rows read and written)": gbs(moved, call)
+                      for name, moved, _, call in recurrences(tokens, one_row, length, one_row, tokens)}
+    four = ints([tokens * n for n in range(4)]), ints([tokens] * 4), ints(range(4))
+    kernels[label].update({name + ", four requests (rows read and written)": gbs(moved, call)
+                           for name, moved, _, call in recurrences(4 * tokens, *four, tokens)})
+    pages = -(-tokens // 16)
+    table = torch.arange(pages, dtype=torch.int32, device="cuda").view(1, -1)
+    positions = torch.arange(tokens, dtype=torch.int32, device="cuda")
+    cache, q = normal(pages, 2, kv_heads, 16, dim).to(bf16), normal(tokens, heads, dim).to(bf16)
+    attended = torch.empty_like(q)
+    gate = normal(tokens, heads * dim).to(bf16)
+    tile = ops.flash_prefill_tile()
+    starts = list(range(0, tokens, tile))[::-1]
+    tiles = (ints([0] * len(starts)), ints(starts), ints([min(tile, tokens - s) for s in starts]))
+    for name, size_of, kept, gated in (("qwen3: tensor-core attention", 0, 0, None),
+                                       ("qwen3: the same in a window of %d" % window, window, 0, None),
+                                       ("mekuvik: in a window of %d beside %d kept positions" % (window, keep), window, keep, None),
+                                       ("mekuvik: all positions, a gate per value", 0, 0, gate)):
+        seen = sum(min(p + 1, (size_of or tokens) + kept) for p in range(tokens))
+        kernels[label][name] = tflops(4.0 * dim * heads * seen, lambda: ops.flash_prefill(
+            q, cache, attended, table, *tiles, positions, dim ** -0.5, longest_context=tokens, window=size_of, keep=kept, gate=gated))
+    ops.check_status("cuda")
+    out["kernels"] = kernels
+    print(json.dumps(out))
+    return 0
+
+
 def main():
     parser = argparse.ArgumentParser(description=__doc__.split("\n\n")[0])
     parser.add_argument("--gpus", type=int, default=1)
@@ -1845,7 +2063,7 @@ def main():
     parser.add_argument("--kernel", default="both", choices=("both", "tcgen05", "mma"))
     parser.add_argument("--page-tokens", type=int, default=16, help="workloads: tokens per cache page")
     parser.add_argument("--max-context", type=int, default=0, help="workloads: the engine's context limit")
-    parser.add_argument("--design", choices=("mekazen", "zitezen", "sadosun", "dimorax", "kokolorn"),
+    parser.add_argument("--design", choices=("mekazen", "zitezen", "sadosun", "dimorax", "kokolorn", "mekuvik"),
                         help="another decoder design beside Qwen3 at equal layer sizes, and its kernels beside their like")
     parser.add_argument("--chunk", type=int, default=0, help="--design: positions per chunk of the mask (0: the context)")
     parser.add_argument("--kernels-only", action="store_true",
@@ -1869,6 +2087,8 @@ def main():
         return design_dimorax(args)
     if args.design == "kokolorn" and not args.workload:
         return design_kokolorn(args)
+    if args.design == "mekuvik" and not args.workload:
+        return design_mekuvik(args)
     if args.design and not args.workload:
         return design(args)
     if args.workload:

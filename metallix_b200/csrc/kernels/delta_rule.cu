@@ -19,7 +19,7 @@
 //
 //   S <- g S + k (dt v)^T;   o = S^T q + skip_h v
 //
-// Lightning attention takes silu(q), silu(k), silu(v) and nothing else:
+// Lightning attention (prompts have a chunked form in lightning.cu) takes silu(q), silu(k), silu(v) and nothing else:
 //
 //   S <- g_h S + k v^T;   o = S^T q
 //
@@ -51,7 +51,11 @@ template <int DPT>
 __device__ __forceinline__ int delta_slot(int d) { return d + (d / DPT) * 4; }
 
 template <typename T> struct alignas(4 * sizeof(T)) DeltaFour { T v[4]; };   // four neighbouring values, one access
-__device__ __forceinline__ float delta_silu(float z) { return z * sigmoid_of(z); }
+// silu, rounded to the type of the projection it activates (what the chunked form of lightning.cu multiplies)
+template <typename T> __device__ __forceinline__ float delta_silu(T x) {
+  const float z = to_float(x);
+  return to_float(from_float<T>(z * sigmoid_of(z)));
+}
 __device__ __forceinline__ float delta_softplus(float z) { return z > 20.0f ? z : log1pf(expf(z)); }
 
 // LANES lanes share a value column, each with DPT of its key channels; COLS neighbouring columns a thread.
@@ -175,8 +179,8 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
       float qq = 0.0f, kk = 0.0f, qk = 0.0f, q_in[NL], k_in[NL];
 #pragma unroll
       for (int i = 0; i < NL; ++i) {
-        q_in[i] = MODE == kDeltaConstant ? delta_silu(to_float(raw_q[i])) : to_float(raw_q[i]);
-        k_in[i] = MODE == kDeltaConstant ? delta_silu(to_float(raw_k[i])) : to_float(raw_k[i]);
+        q_in[i] = MODE == kDeltaConstant ? delta_silu(raw_q[i]) : to_float(raw_q[i]);
+        k_in[i] = MODE == kDeltaConstant ? delta_silu(raw_k[i]) : to_float(raw_k[i]);
         qq = fmaf(q_in[i], q_in[i], qq); kk = fmaf(k_in[i], k_in[i], kk); qk = fmaf(q_in[i], k_in[i], qk);
       }
       qk = warp_sum(qk);
@@ -208,7 +212,7 @@ delta_rule_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off,
     for (int j = 0; j < kDeltaMaxWarps; ++j)
 #pragma unroll
       for (int c = 0; c < COLS; ++c)
-        v[j][c] = MODE == kDeltaConstant ? delta_silu(to_float(next_v[j][c])) : to_float(next_v[j][c]);
+        v[j][c] = MODE == kDeltaConstant ? delta_silu(next_v[j][c]) : to_float(next_v[j][c]);
     __syncthreads();
     if (base + warps < length) fetch(base + warps);   // on its way while this batch is walked through
 #pragma unroll

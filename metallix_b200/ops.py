@@ -59,6 +59,9 @@ _SIGNATURES = {
     "mxb_delta_rule_max_dim": [],
     "mxb_delta_rule": [_P, _L, _I, _I, _I, _P, _L, _I, _P, _L, _P, _P, _P, _I, _P, _L, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I,
                        _I, _I, _P, _P],
+    "mxb_lightning_chunks_supported": [_P, _L, _I, _I, _I, _I, _I, _I],
+    "mxb_silu_columns": [_P, _L, _I, _I, _P],
+    "mxb_lightning_chunks": [_P, _L, _I, _I, _I, _P, _P, _L, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     "mxb_add_cast": [_P, _P, _I, _P, _I, _L, _P],
     "mxb_gelu_gate_rows": [_P, _P, _P, _P, _I, _I, _I, _I, _I, _I, _P, _P],
     "mxb_stream_mix": [_P, _P, _P, _L, _L, _F, _F, _I, _P, _P, _P, _P, _P, _P, _P, _P, _I, _P, _I, _I, _I, _I, _P],
@@ -1011,15 +1014,56 @@ def state_space_dual(xbc: torch.Tensor, offsets, step: torch.Tensor, step_bias: 
                          heads, groups, dim, vdim, longest)
 
 
+def silu_columns_(x: torch.Tensor) -> torch.Tensor:
+    """x <- silu(x), rounded once, for bfloat16 x ``[tokens, width]`` whose rows may be strided (a column range)."""
+    _need(x.is_cuda and x.dtype == torch.bfloat16 and x.dim() == 2 and x.stride(1) == 1, "x must be bfloat16 [tokens, width]")
+    _call("mxb_silu_columns", x.data_ptr(), x.stride(0), x.shape[0], x.shape[1], _stream())
+    return x
+
+
+LIGHTNING_CHUNK_TOKENS = 8    # steps whose longest row brings this many tokens or more take the chunked form
+
+
 def lightning_attention(qkv: torch.Tensor, offsets, decay: torch.Tensor, state: torch.Tensor, row_start: torch.Tensor,
                         row_length: torch.Tensor, request_slots: torch.Tensor, heads: int, dim: int, vdim: int,
-                        longest: int = 0) -> torch.Tensor:
+                        longest: int = 0, form: str = "auto") -> torch.Tensor:
     """Linear attention with a constant decay per head over a step's tokens.
     ``qkv`` holds, from the column ``offsets`` (q, k, v) on, heads * dim queries and
-    keys and heads * vdim values, all ahead of their silu, which happens in the
-    kernel; ``decay`` float32 ``[heads]``. Per head S <- decay S + k v^T, o = S^T q.
+    keys and heads * vdim values, all ahead of their silu (in the chunked form qkv
+    itself takes it, so that these columns are used up); ``decay`` float32 ``[heads]``. Per head S <- decay S + k v^T, o = S^T q.
     ``state`` float32 ``[slots, heads, vdim, dim]`` is advanced in place; rows and
-    slots as in ``delta_rule``. Returns float32 ``[tokens, heads * vdim]``."""
+    slots as in ``delta_rule``. Returns float32 ``[tokens, heads * vdim]``. ``form``:
+    "tokens" walks token by token, "chunks" takes 64 tokens at a time on the
+    tensor cores (bfloat16, up to 128 key channels), "auto" the second where it
+    takes the layout and the longest row brings ``LIGHTNING_CHUNK_TOKENS``
+    or more (or is not known)."""
+    _need(form in ("auto", "tokens", "chunks"), f"unknown form {form!r}")
+    if form != "tokens" and (form == "chunks" or not 0 < longest < LIGHTNING_CHUNK_TOKENS):
+        _need(qkv.is_cuda and qkv.dtype in _CODES and qkv.dim() == 2 and qkv.stride(1) == 1,
+              "qkv must be a CUDA [tokens, columns] tensor with unit column stride")
+        where = tuple(int(o) for o in offsets)
+        takes = bool(_fn("mxb_lightning_chunks_supported")(qkv.data_ptr(), qkv.stride(0), *where, dim, vdim, _CODES[qkv.dtype]))
+        _need(takes or form == "auto", "the chunked form takes bfloat16 heads of whole 16-byte pieces, up to 128 key channels")
+        if takes:
+            _check(decay, "decay", (torch.float32,), 1)
+            _check(state, "state", (torch.float32,), 4)
+            _need(decay.numel() == heads and state.shape[1:] == (heads, vdim, dim), "decay or state does not fit the heads")
+            for name, tensor in (("row_start", row_start), ("row_length", row_length), ("request_slots", request_slots)):
+                _check(tensor, name, (torch.int32,), 1)
+            rows = row_start.numel()
+            _need(row_length.numel() == rows and request_slots.numel() >= rows, "row lists differ in length")
+            _need(max(where[0] + heads * dim, where[1] + heads * dim, where[2] + heads * vdim) <= qkv.shape[1],
+                  "the column offsets reach beyond qkv")
+            out = torch.empty((qkv.shape[0], heads * vdim), dtype=torch.float32, device=qkv.device)
+            ranges = sorted((start, heads * width) for start, width in zip(where, (dim, dim, vdim)))
+            while len(ranges) > 1 and ranges[0][0] + ranges[0][1] == ranges[1][0]:    # neighbours are one range
+                ranges[:2] = [(ranges[0][0], ranges[0][1] + ranges[1][1])]
+            for start, width in ranges:
+                silu_columns_(qkv[:, start:start + width])
+            _call("mxb_lightning_chunks", qkv.data_ptr(), qkv.stride(0), *where, decay.data_ptr(), state.data_ptr(),
+                  state.stride(0), state.shape[0], row_start.data_ptr(), row_length.data_ptr(), request_slots.data_ptr(),
+                  out.data_ptr(), rows, heads, dim, vdim, _CODES[qkv.dtype], status_word(qkv.device).data_ptr(), _stream())
+            return out
     return _matrix_state(3, qkv, offsets, None, None, None, decay, None, state, row_start, row_length, request_slots,
                          heads, heads, dim, vdim, longest)
 
