@@ -140,6 +140,81 @@ __global__ void latent_heads_kernel(const T* __restrict__ q, long long ld_q, con
   }
 }
 
+// The same, eight bfloat16 values (16 bytes) a thread, for sizes that are whole pieces: a block takes 256 pieces of a
+// token's heads, so that a step of few tokens still has many blocks. A piece is unrotated, rotated or padding as a
+// whole; the partner of a rotated value lies in the same piece (interleaved) or in another whole piece.
+__global__ void __launch_bounds__(256)
+latent_heads_by8_kernel(const __nv_bfloat16* __restrict__ q, long long ld_q, const __nv_bfloat16* __restrict__ up,
+                        long long ld_up, const __nv_bfloat16* __restrict__ shared_part, long long ld_shared, int shared_off,
+                        __nv_bfloat16* __restrict__ q_heads, __nv_bfloat16* __restrict__ cache, const int* __restrict__ slots,
+                        const int* __restrict__ positions, const float* __restrict__ cos_table,
+                        const float* __restrict__ sin_table, int table_positions, int rotary_dim, int interleaved, int heads,
+                        int D, int R, int V, int hd, int page_tokens, int num_pages, int* status) {
+  chain_release();
+  const int t = blockIdx.x, pieces = hd / 8;
+  const int index = blockIdx.y * blockDim.x + threadIdx.x;
+  int pos = positions[t];
+  const bool reports = index == 0;
+  if (pos < 0 || (rotary_dim > 0 && pos >= table_positions)) {
+    if (reports) atomicOr(status, kStatusBadSlot);
+    pos = 0;
+  }
+  const int slot = slots != nullptr ? slots[t] : -1;
+  const bool writes = slot >= 0 && slot < num_pages * page_tokens;
+  if (slot >= num_pages * page_tokens && reports) atomicOr(status, kStatusBadSlot);
+  if (index >= heads * pieces) return;
+  const int h = index / pieces, i = (index - h * pieces) * 8;
+  const uint4 zero = make_uint4(0u, 0u, 0u, 0u);
+  auto load = [](const __nv_bfloat16* p) { return *reinterpret_cast<const uint4*>(p); };
+  const __nv_bfloat16* q_row = q + static_cast<long long>(t) * ld_q + static_cast<long long>(h) * (D + R);
+  uint4 query = i < D + R ? load(q_row + i) : zero, key = zero, value = zero;
+  if (writes) {
+    const __nv_bfloat16* up_row = up + static_cast<long long>(t) * ld_up;
+    if (i < D) key = load(up_row + static_cast<long long>(h) * D + i);
+    else if (i < D + R) key = load(shared_part + static_cast<long long>(t) * ld_shared + shared_off + i - D);
+    if (i < V) value = load(up_row + static_cast<long long>(heads) * D + static_cast<long long>(h) * V + i);
+  }
+  const int r = i - D;      // place in the rotated part
+  if (r >= 0 && r < rotary_dim) {
+    const int half = rotary_dim / 2;
+    const float* cos_row = cos_table + static_cast<long long>(pos) * half;
+    const float* sin_row = sin_table + static_cast<long long>(pos) * half;
+    uint32_t mine[4] = {query.x, query.y, query.z, query.w};
+    auto low = [](uint32_t w) { return __uint_as_float(w << 16); };
+    auto high = [](uint32_t w) { return __uint_as_float(w & 0xffff0000u); };
+    auto pack = [](float a, float b) {
+      const __nv_bfloat162 both = __floats2bfloat162_rn(a, b);
+      return *reinterpret_cast<const uint32_t*>(&both);
+    };
+    if (interleaved) {
+#pragma unroll
+      for (int w = 0; w < 4; ++w) {
+        const float c = cos_row[r / 2 + w], s = sin_row[r / 2 + w], a = low(mine[w]), b = high(mine[w]);
+        mine[w] = pack(a * c - b * s, b * c + a * s);
+      }
+    } else {
+      const bool first = r < half;
+      const uint4 partner = load(q_row + i + (first ? half : -half));
+      const uint32_t theirs[4] = {partner.x, partner.y, partner.z, partner.w};
+      const int pair = first ? r : r - half;
+      const float sign = first ? -1.0f : 1.0f;
+#pragma unroll
+      for (int w = 0; w < 4; ++w) {
+        const float c0 = cos_row[pair + 2 * w], c1 = cos_row[pair + 2 * w + 1];
+        const float s0 = sign * sin_row[pair + 2 * w], s1 = sign * sin_row[pair + 2 * w + 1];
+        mine[w] = pack(low(mine[w]) * c0 + low(theirs[w]) * s0, high(mine[w]) * c1 + high(theirs[w]) * s1);
+      }
+    }
+    query = make_uint4(mine[0], mine[1], mine[2], mine[3]);
+  }
+  *reinterpret_cast<uint4*>(q_heads + (static_cast<long long>(t) * heads + h) * hd + i) = query;
+  if (!writes) return;
+  const int page = slot / page_tokens, in_page = slot - page * page_tokens;
+  const long long at = ((static_cast<long long>(page) * 2 * heads + h) * page_tokens + in_page) * hd + i;
+  *reinterpret_cast<uint4*>(cache + at) = key;
+  *reinterpret_cast<uint4*>(cache + at + static_cast<long long>(heads) * page_tokens * hd) = value;
+}
+
 }  // namespace mxb
 
 using namespace mxb;
@@ -151,6 +226,17 @@ MXB_API int mxb_latent_heads(const void* q, long long ld_q, const void* up, long
                              int num_pages, int tokens, int dtype, int* status, cudaStream_t stream) {
   if (tokens <= 0) return 0;
   if (heads <= 0 || D + R > hd || V > hd || rotary_dim > R || rotary_dim % 2) return static_cast<int>(cudaErrorInvalidValue);
+  auto whole = [](const void* p, long long stride) { return (reinterpret_cast<uintptr_t>(p) & 15) == 0 && stride % 8 == 0; };
+  if (dtype == kBF16 && D % 8 == 0 && R % 8 == 0 && V % 8 == 0 && hd % 8 == 0 && rotary_dim % (interleaved ? 8 : 16) == 0 &&
+      shared_off % 8 == 0 && whole(q, ld_q) && whole(up, ld_up) && whole(shared_part, ld_shared) && whole(q_heads, 8) &&
+      whole(cache, 8)) {
+    latent_heads_by8_kernel<<<dim3(tokens, ceil_div(heads * (hd / 8), 256)), 256, 0, stream>>>(
+        static_cast<const __nv_bfloat16*>(q), ld_q, static_cast<const __nv_bfloat16*>(up), ld_up,
+        static_cast<const __nv_bfloat16*>(shared_part), ld_shared, shared_off, static_cast<__nv_bfloat16*>(q_heads),
+        static_cast<__nv_bfloat16*>(cache), slots, positions, cos_table, sin_table, table_positions, rotary_dim,
+        interleaved, heads, D, R, V, hd, page_tokens, num_pages, status);
+    return static_cast<int>(cudaGetLastError());
+  }
   if (dtype == kF32)
     latent_heads_kernel<float><<<tokens, 256, 0, stream>>>(
         static_cast<const float*>(q), ld_q, static_cast<const float*>(up), ld_up, static_cast<const float*>(shared_part),

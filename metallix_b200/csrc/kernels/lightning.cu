@@ -1,5 +1,6 @@
-// Lightning attention over portions of prompts, on the tensor cores: linear
-// attention whose decay per head is a constant, in chunks of 64 tokens. Per
+// Lightning attention: linear attention whose decay per head is a constant.
+//
+// Over portions of prompts, on the tensor cores in chunks of 64 tokens. Per
 // head, with g the decay and q, k, v past their silu (rounded to bfloat16, as
 // the token-by-token form in delta_rule.cu rounds them),
 //
@@ -24,6 +25,11 @@
 // the same queries and keys, and the exponentials of 64 tokens cost a block as
 // much time as its products. The next chunk's rows are on their way (cp.async)
 // while this one is worked on.
+//
+// Over single tokens (and a few) the state is what must be read and written:
+// lightning_step_kernel gives a value column to 8, 16 or 32 lanes with four key
+// channels each, a warp several columns whose loads are all on their way at
+// once, and walks over the row's tokens with the state in registers.
 #include "common.cuh"
 
 namespace mxb {
@@ -356,9 +362,133 @@ lightning_chunk_kernel(const __nv_bfloat16* __restrict__ qkv, long long ld, int 
   }
 }
 
+// Four neighbouring values as floats past their silu, rounded to their own type.
+__device__ __forceinline__ float4 ln_silu_four(const float* p) {
+  const float4 x = *reinterpret_cast<const float4*>(p);
+  return make_float4(x.x * sigmoid_of(x.x), x.y * sigmoid_of(x.y), x.z * sigmoid_of(x.z), x.w * sigmoid_of(x.w));
+}
+__device__ __forceinline__ float ln_silu_half(uint32_t bits) {
+  const float z = __uint_as_float(bits);
+  return to_float(from_float<__nv_bfloat16>(z * sigmoid_of(z)));
+}
+__device__ __forceinline__ float4 ln_silu_four(const __nv_bfloat16* p) {
+  const uint2 x = *reinterpret_cast<const uint2*>(p);
+  return make_float4(ln_silu_half(x.x << 16), ln_silu_half(x.x & 0xffff0000u), ln_silu_half(x.y << 16),
+                     ln_silu_half(x.y & 0xffff0000u));
+}
+
+// LANES lanes share a column (four of its key channels each), so a warp holds 32 / LANES columns side by side, kLnHeld of
+// each lane; a block is kLnStepWarps warps.
+constexpr int kLnHeld = 4, kLnStepWarps = 4;
+
+template <typename T, int LANES>
+__global__ void __launch_bounds__(kLnStepWarps * 32)
+lightning_step_kernel(const T* __restrict__ qkv, long long ld, int q_off, int k_off, int v_off,
+                      const float* __restrict__ decay, float* __restrict__ state, long long slot_stride, int num_slots,
+                      const int* __restrict__ row_start, const int* __restrict__ row_length,
+                      const int* __restrict__ request_slots, float* __restrict__ out, int heads, int dim, int vdim,
+                      int* status) {
+  constexpr int SIDE = 32 / LANES, COLUMNS = SIDE * kLnHeld;     // columns of a warp
+  const int row = blockIdx.x, head = blockIdx.y;
+  const int length = row_length[row], slot = request_slots[row], first = row_start[row];
+  if (length <= 0) return;   // a padding row owns no state
+  if (slot < 0 || slot >= num_slots) {
+    if (threadIdx.x == 0) atomicOr(status, kStatusBadSlot);
+    return;
+  }
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, side = lane / LANES, d = (lane % LANES) * 4;
+  const int column0 = (blockIdx.z * kLnStepWarps + warp) * COLUMNS + side;   // this lane's columns: column0 + c * SIDE
+  const bool channels = d < dim;
+  float* base = state + static_cast<long long>(slot) * slot_stride + static_cast<long long>(head) * vdim * dim + d;
+  float4 s[kLnHeld];
+#pragma unroll
+  for (int c = 0; c < kLnHeld; ++c) {
+    const int column = column0 + c * SIDE;
+    s[c] = channels && column < vdim ? *reinterpret_cast<const float4*>(base + static_cast<long long>(column) * dim)
+                                     : make_float4(0.0f, 0.0f, 0.0f, 0.0f);
+  }
+  const float g = decay[head];
+  for (int t = 0; t < length; ++t) {
+    const T* token = qkv + static_cast<long long>(first + t) * ld;
+    float4 q = make_float4(0.0f, 0.0f, 0.0f, 0.0f), k = q;
+    if (channels) {
+      q = ln_silu_four(token + q_off + head * dim + d);
+      k = ln_silu_four(token + k_off + head * dim + d);
+    }
+    float sums[kLnHeld];
+#pragma unroll
+    for (int c = 0; c < kLnHeld; ++c) {
+      const int column = column0 + c * SIDE;
+      float v = 0.0f;
+      if (column < vdim) {
+        v = to_float(token[v_off + head * vdim + column]);
+        v = to_float(from_float<T>(v * sigmoid_of(v)));
+      }
+      s[c].x = fmaf(k.x, v, g * s[c].x); s[c].y = fmaf(k.y, v, g * s[c].y);
+      s[c].z = fmaf(k.z, v, g * s[c].z); s[c].w = fmaf(k.w, v, g * s[c].w);
+      sums[c] = fmaf(q.x, s[c].x, fmaf(q.y, s[c].y, fmaf(q.z, s[c].z, q.w * s[c].w)));
+    }
+    // kLnHeld sums over LANES lanes: every exchange halves the sums a lane still adds up, then the lanes
+    static_assert(kLnHeld == 4, "the exchanges below are for four sums");
+    const bool upper = (lane & (LANES / 2)) != 0, odd = (lane & (LANES / 4)) != 0;
+    float a = upper ? sums[2] : sums[0], b = upper ? sums[3] : sums[1];
+    a += __shfl_xor_sync(0xffffffffu, upper ? sums[0] : sums[2], LANES / 2);
+    b += __shfl_xor_sync(0xffffffffu, upper ? sums[1] : sums[3], LANES / 2);
+    float sum = odd ? b : a;
+    sum += __shfl_xor_sync(0xffffffffu, odd ? a : b, LANES / 4);
+#pragma unroll
+    for (int offset = LANES / 8; offset > 0; offset >>= 1) sum += __shfl_xor_sync(0xffffffffu, sum, offset);
+    const int column = column0 + ((upper ? 2 : 0) + (odd ? 1 : 0)) * SIDE;
+    if (lane % (LANES / 4) == 0 && column < vdim)
+      out[static_cast<long long>(first + t) * (static_cast<long long>(heads) * vdim) + head * vdim + column] = sum;
+  }
+#pragma unroll
+  for (int c = 0; c < kLnHeld; ++c) {
+    const int column = column0 + c * SIDE;
+    if (channels && column < vdim) *reinterpret_cast<float4*>(base + static_cast<long long>(column) * dim) = s[c];
+  }
+}
+
 }  // namespace mxb
 
 using namespace mxb;
+
+// Whether the form for few tokens takes this layout: up to 128 key channels in whole groups of four, rows and state on
+// boundaries that four values make.
+MXB_API int mxb_lightning_steps_supported(const void* qkv, long long ld, int q_off, int k_off, const float* state,
+                                          long long slot_stride, int dim, int dtype) {
+  const int four = dtype == kBF16 ? 8 : 16;
+  return (dtype == kBF16 || dtype == kF32) && dim > 0 && dim <= 128 && dim % 4 == 0 && ld % 4 == 0 && q_off % 4 == 0 &&
+                 k_off % 4 == 0 && reinterpret_cast<uintptr_t>(qkv) % four == 0 && (reinterpret_cast<uintptr_t>(state) & 15) == 0 &&
+                 slot_stride % 4 == 0 ? 1 : 0;
+}
+
+// Operands as for mxb_lightning_chunks, of either type, q, k and v ahead of their silu.
+MXB_API int mxb_lightning_steps(const void* qkv, long long ld, int q_off, int k_off, int v_off, const float* decay,
+                                float* state, long long slot_stride, int num_slots, const int* row_start,
+                                const int* row_length, const int* request_slots, float* out, int rows, int heads, int dim,
+                                int vdim, int dtype, int* status, cudaStream_t stream) {
+  if (rows <= 0) return 0;
+  if (heads <= 0 || vdim <= 0 || !mxb_lightning_steps_supported(qkv, ld, q_off, k_off, state, slot_stride, dim, dtype))
+    return static_cast<int>(cudaErrorInvalidValue);
+  const int lanes = dim <= 32 ? 8 : (dim <= 64 ? 16 : 32);
+  const dim3 grid(rows, heads, ceil_div(vdim, kLnStepWarps * kLnHeld * (32 / lanes))), block(kLnStepWarps * 32);
+#define GO(T, LANES)                                                                                                    \
+  lightning_step_kernel<T, LANES><<<grid, block, 0, stream>>>(static_cast<const T*>(qkv), ld, q_off, k_off, v_off, decay, \
+                                                              state, slot_stride, num_slots, row_start, row_length,     \
+                                                              request_slots, out, heads, dim, vdim, status)
+  if (dtype == kBF16) {
+    if (lanes == 8) GO(__nv_bfloat16, 8);
+    else if (lanes == 16) GO(__nv_bfloat16, 16);
+    else GO(__nv_bfloat16, 32);
+  } else {
+    if (lanes == 8) GO(float, 8);
+    else if (lanes == 16) GO(float, 16);
+    else GO(float, 32);
+  }
+#undef GO
+  return static_cast<int>(cudaGetLastError());
+}
 
 // Whether the chunked form takes this layout: bfloat16 rows whose heads are whole 16-byte pieces, up to 128 key channels.
 MXB_API int mxb_lightning_chunks_supported(const void* qkv, long long ld, int q_off, int k_off, int v_off, int dim, int vdim,

@@ -60,6 +60,8 @@ _SIGNATURES = {
     "mxb_delta_rule": [_P, _L, _I, _I, _I, _P, _L, _I, _P, _L, _P, _P, _P, _I, _P, _L, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I,
                        _I, _I, _P, _P],
     "mxb_lightning_chunks_supported": [_P, _L, _I, _I, _I, _I, _I, _I],
+    "mxb_lightning_steps_supported": [_P, _L, _I, _I, _P, _L, _I, _I],
+    "mxb_lightning_steps": [_P, _L, _I, _I, _I, _P, _P, _L, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     "mxb_silu_columns": [_P, _L, _I, _I, _P],
     "mxb_lightning_chunks": [_P, _L, _I, _I, _I, _P, _P, _L, _I, _P, _P, _P, _P, _I, _I, _I, _I, _I, _P, _P],
     "mxb_add_cast": [_P, _P, _I, _P, _I, _L, _P],
@@ -1033,37 +1035,47 @@ def lightning_attention(qkv: torch.Tensor, offsets, decay: torch.Tensor, state: 
     itself takes it, so that these columns are used up); ``decay`` float32 ``[heads]``. Per head S <- decay S + k v^T, o = S^T q.
     ``state`` float32 ``[slots, heads, vdim, dim]`` is advanced in place; rows and
     slots as in ``delta_rule``. Returns float32 ``[tokens, heads * vdim]``. ``form``:
-    "tokens" walks token by token, "chunks" takes 64 tokens at a time on the
-    tensor cores (bfloat16, up to 128 key channels), "auto" the second where it
-    takes the layout and the longest row brings ``LIGHTNING_CHUNK_TOKENS``
-    or more (or is not known)."""
-    _need(form in ("auto", "tokens", "chunks"), f"unknown form {form!r}")
-    if form != "tokens" and (form == "chunks" or not 0 < longest < LIGHTNING_CHUNK_TOKENS):
-        _need(qkv.is_cuda and qkv.dtype in _CODES and qkv.dim() == 2 and qkv.stride(1) == 1,
-              "qkv must be a CUDA [tokens, columns] tensor with unit column stride")
-        where = tuple(int(o) for o in offsets)
-        takes = bool(_fn("mxb_lightning_chunks_supported")(qkv.data_ptr(), qkv.stride(0), *where, dim, vdim, _CODES[qkv.dtype]))
-        _need(takes or form == "auto", "the chunked form takes bfloat16 heads of whole 16-byte pieces, up to 128 key channels")
-        if takes:
-            _check(decay, "decay", (torch.float32,), 1)
-            _check(state, "state", (torch.float32,), 4)
-            _need(decay.numel() == heads and state.shape[1:] == (heads, vdim, dim), "decay or state does not fit the heads")
-            for name, tensor in (("row_start", row_start), ("row_length", row_length), ("request_slots", request_slots)):
-                _check(tensor, name, (torch.int32,), 1)
-            rows = row_start.numel()
-            _need(row_length.numel() == rows and request_slots.numel() >= rows, "row lists differ in length")
-            _need(max(where[0] + heads * dim, where[1] + heads * dim, where[2] + heads * vdim) <= qkv.shape[1],
-                  "the column offsets reach beyond qkv")
-            out = torch.empty((qkv.shape[0], heads * vdim), dtype=torch.float32, device=qkv.device)
+    "chunks" takes 64 tokens at a time on the tensor cores (bfloat16), "steps"
+    has every load of the state on its way at once (both up to 128 key channels
+    in whole vectors), "tokens" walks token by token through the kernel of the
+    other matrix-state recurrences; "auto" takes the first where the longest row
+    brings ``LIGHTNING_CHUNK_TOKENS`` or more (or is not known), else the second,
+    and the third where they do not take the layout."""
+    _need(form in ("auto", "tokens", "chunks", "steps"), f"unknown form {form!r}")
+    _need(qkv.is_cuda and qkv.dtype in _CODES and qkv.dim() == 2 and qkv.stride(1) == 1,
+          "qkv must be a CUDA [tokens, columns] tensor with unit column stride")
+    _check(decay, "decay", (torch.float32,), 1)
+    _check(state, "state", (torch.float32,), 4)
+    _need(decay.numel() == heads and state.shape[1:] == (heads, vdim, dim), "decay or state does not fit the heads")
+    where, code = tuple(int(o) for o in offsets), _CODES[qkv.dtype]
+    many = not 0 < longest < LIGHTNING_CHUNK_TOKENS
+    kernel = None
+    if form == "chunks" or (form == "auto" and many):
+        if _fn("mxb_lightning_chunks_supported")(qkv.data_ptr(), qkv.stride(0), *where, dim, vdim, code):
+            kernel = "mxb_lightning_chunks"
+    elif form == "steps" or form == "auto":
+        if _fn("mxb_lightning_steps_supported")(qkv.data_ptr(), qkv.stride(0), where[0], where[1], state.data_ptr(),
+                                                state.stride(0), dim, code):
+            kernel = "mxb_lightning_steps"
+    _need(kernel is not None or form in ("auto", "tokens"), f"the form {form!r} does not take this layout")
+    if kernel is not None:
+        for name, tensor in (("row_start", row_start), ("row_length", row_length), ("request_slots", request_slots)):
+            _check(tensor, name, (torch.int32,), 1)
+        rows = row_start.numel()
+        _need(row_length.numel() == rows and request_slots.numel() >= rows, "row lists differ in length")
+        _need(max(where[0] + heads * dim, where[1] + heads * dim, where[2] + heads * vdim) <= qkv.shape[1],
+              "the column offsets reach beyond qkv")
+        out = torch.empty((qkv.shape[0], heads * vdim), dtype=torch.float32, device=qkv.device)
+        if kernel == "mxb_lightning_chunks":
             ranges = sorted((start, heads * width) for start, width in zip(where, (dim, dim, vdim)))
             while len(ranges) > 1 and ranges[0][0] + ranges[0][1] == ranges[1][0]:    # neighbours are one range
                 ranges[:2] = [(ranges[0][0], ranges[0][1] + ranges[1][1])]
             for start, width in ranges:
                 silu_columns_(qkv[:, start:start + width])
-            _call("mxb_lightning_chunks", qkv.data_ptr(), qkv.stride(0), *where, decay.data_ptr(), state.data_ptr(),
-                  state.stride(0), state.shape[0], row_start.data_ptr(), row_length.data_ptr(), request_slots.data_ptr(),
-                  out.data_ptr(), rows, heads, dim, vdim, _CODES[qkv.dtype], status_word(qkv.device).data_ptr(), _stream())
-            return out
+        _call(kernel, qkv.data_ptr(), qkv.stride(0), *where, decay.data_ptr(), state.data_ptr(), state.stride(0),
+              state.shape[0], row_start.data_ptr(), row_length.data_ptr(), request_slots.data_ptr(), out.data_ptr(), rows,
+              heads, dim, vdim, code, status_word(qkv.device).data_ptr(), _stream())
+        return out
     return _matrix_state(3, qkv, offsets, None, None, None, decay, None, state, row_start, row_length, request_slots,
                          heads, heads, dim, vdim, longest)
 
