@@ -1008,6 +1008,8 @@ def test_a_key_at_either_side_of_a_windows_edge_and_of_the_last_kept_position(fo
     tensors = {name: rounded(value, torch.bfloat16) for name, value in tensors.items()}
     seen_at = {0: True, 15: True, 16: True, keep - 1: True, keep: False, 64: False, last - window: False,
                last - window + 1: True, last - 8: True, last - 1: True}
+    engine = Engine(MekuvikConfig.from_dict(raw), {k: torch.tensor(v, dtype=torch.float32) for k, v in tensors.items()},
+                    dtype=dtype, page_tokens=16, num_pages=16, max_requests=1)
     for early, seen in seen_at.items():
         ids = [int(t) for t in rng.integers(1, 60, size=last)]
         ids[early] = 62
@@ -1017,8 +1019,6 @@ def test_a_key_at_either_side_of_a_windows_edge_and_of_the_last_kept_position(fo
         tolerance = 2e-4 if dtype == "float32" else 3e-1
         assert (np.abs(want - other).max() > 8 * tolerance) == seen and (seen or np.abs(want - other).max() < 1e-9), early
         for sizes in ([last + 1], [last, 1], [100, 64, 36, 1], [3] * 66 + [2, 1]):
-            engine = Engine(MekuvikConfig.from_dict(raw), {k: torch.tensor(v, dtype=torch.float32) for k, v in tensors.items()},
-                            dtype=dtype, page_tokens=16, num_pages=16, max_requests=1)
             logits, at = None, 0
             for size in sizes:
                 logits = engine.step([StepEntry("a", ids[at:at + size], [size - 1])])
@@ -1027,6 +1027,7 @@ def test_a_key_at_either_side_of_a_windows_edge_and_of_the_last_kept_position(fo
             assert np.abs(logits[0].double().cpu().numpy() - want).max() < tolerance, (early, sizes)
             table = engine.manager.table(engine._ids["a"], 0)
             assert [page >= 0 for page in table[:2]] == [True, True] and table[4] < 0      # kept pages stay, others went back
+            engine.release("a")
 
 
 @gpu
